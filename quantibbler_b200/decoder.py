@@ -165,7 +165,215 @@ def _p(t) -> ctypes.c_void_p:
     return ctypes.c_void_p(t.data_ptr())
 
 
-class Decoder:
+class SlotDecoder:
+    """What every decoder here shares: a batch of sequence slots with device-resident token ids
+    and positions, batched greedy steps (eager or as a replayed CUDA graph), prompts fed in
+    portions, generation with the reference's control flow.
+
+    A subclass sets up ``torch``, ``ctx``, ``cfg`` (``vocab``, ``max_seq``, ``max_batch``,
+    ``prefill_min_tokens``, ``prefill_chunk``, ``serving``), ``token_ids``, ``positions``,
+    ``logits``, ``best_val``, ``best_idx``, ``h`` (hidden rows in front of the head), ``lm_head``
+    with ``head_width`` columns, ``v_loc`` and ``vocab_offset``, and provides ``step`` (one
+    batched step), ``_prefill_portion`` (the trunk over one portion of a prompt) and
+    ``_portion_hidden`` (final-normed hidden rows of the last portion)."""
+
+    tp_size, group = 1, None
+    keeps_state = False   # True: a step changes more than the cache row of its own position
+
+    def _setup_driver(self) -> None:
+        self.graph = None
+        self.kernels_per_step = None
+        self._host_positions = [0] * self.cfg.max_batch
+
+    # ------------------------------------------------------------------ head and sampling
+    def _head(self, hidden, n: int, logits) -> None:
+        """logits[:n] from ``n`` final-normed rows (a vocabulary shard under tensor parallelism)."""
+        tag = QK_BF16 if self.cfg.serving == "bfloat16" else QK_F32
+        check(_lib.lib().qk_lm_head(self.ctx.handle, _p(hidden), _p(self.lm_head), tag, n, self.v_loc,
+                                    self.head_width, self.v_loc, _p(logits)))
+
+    def _greedy(self, logits, n: int, best_val, best_idx) -> None:
+        """The first maximum of each row."""
+        check(_lib.lib().qk_argmax_first(self.ctx.handle, _p(logits), n, self.v_loc, self.v_loc,
+                                         self.vocab_offset, _p(best_val), _p(best_idx)))
+        if self.tp_size > 1:
+            self._gather_argmax(best_val, best_idx)
+
+    def prefill(self, tokens, seq: int = 0, first_position: int = 0, want=None):
+        """All of ``tokens`` (consecutive positions ``first_position ...`` of sequence slot ``seq``)
+        through the trunk in one pass per ``prefill_chunk`` positions: the batched form of the
+        reference's prompt loop (engine/mod.rs:1393-1413, one ``transformer`` call per prompt
+        token).  Appends what every position leaves in the cache or state and puts the greedy token
+        of the last position into ``best_idx[seq]``; ``advance()`` + ``step()`` then continue the
+        sequence.  Only the last position goes through the final norm and the head, and those at
+        the places ``want`` among ``tokens``, whose logits are then returned ([len(want), vocab],
+        on the device)."""
+        torch, cfg = self.torch, self.cfg
+        toks = [int(t) for t in tokens]
+        if not toks:
+            raise ValueError("prefill needs at least one token")
+        if not 0 <= seq < cfg.max_batch:
+            raise ValueError(f"sequence slot {seq} outside the batch of {cfg.max_batch}")
+        check_cache_capacity([first_position], len(toks), cfg.max_seq)
+        want = None if want is None else [int(w) for w in want]
+        if want and not 0 <= min(want) <= max(want) < len(toks):
+            raise ValueError(f"wanted places {min(want)}..{max(want)} outside the {len(toks)} tokens")
+        handle = self.ctx.stream
+        # (handles 0 and 1 are the legacy default stream, which torch wraps itself)
+        stream = torch.cuda.ExternalStream(handle) if handle > 2 else torch.cuda.default_stream()
+        stream.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(stream):
+            logits = None if want is None else torch.empty(len(want), self.v_loc, dtype=torch.float32,
+                                                           device=self.logits.device)
+            reserve = min(len(toks), cfg.prefill_chunk)
+            for c0 in range(0, len(toks), cfg.prefill_chunk):
+                part = toks[c0:c0 + cfg.prefill_chunk]
+                self._prefill_portion(part, seq, first_position + c0, reserve)
+                asked = [i for i, w in enumerate(want or []) if c0 <= w < c0 + len(part)]
+                for i in range(0, len(asked), 64):
+                    some = asked[i:i + 64]
+                    hidden = torch.zeros(len(some), self.head_width, dtype=torch.float32, device=logits.device)
+                    rows = torch.empty(len(some), self.v_loc, dtype=torch.float32, device=logits.device)
+                    self._portion_hidden([want[j] - c0 for j in some], hidden)
+                    self._head(hidden, len(some), rows)
+                    logits[torch.as_tensor(some, device=logits.device)] = rows
+            # the last position alone: final norm, head, greedy choice
+            self._portion_hidden([len(part) - 1], self.h[seq:seq + 1])
+            self._head(self.h[seq:seq + 1], 1, self.logits[seq:seq + 1])
+            self._greedy(self.logits[seq:seq + 1], 1, self.best_val[seq:seq + 1], self.best_idx[seq:seq + 1])
+            last = first_position + len(toks) - 1
+            self._reset_slot(seq, toks[-1], last)
+        stream.synchronize()
+        torch.cuda.current_stream().wait_stream(stream)
+        self._host_positions[seq] = last
+        self.ctx.synchronize()
+        return logits
+
+    def _reset_slot(self, seq: int, token: int, position: int) -> None:
+        self.token_ids[seq:seq + 1].fill_(token)
+        self.positions[seq:seq + 1].fill_(position)
+
+    def _step_inputs(self) -> list:
+        return [self.token_ids, self.positions]
+
+    def _make_idle(self) -> None:
+        """Make a step leave every cache and state alone (decoders with ``keeps_state``)."""
+
+    def _gather_argmax(self, best_val, best_idx) -> None:
+        """Vocabulary-parallel head: the first maximum over the ranks' shard winners."""
+        torch = self.torch
+        vals = [torch.empty_like(best_val) for _ in range(self.tp_size)]
+        idxs = [torch.empty_like(best_idx) for _ in range(self.tp_size)]
+        torch.distributed.all_gather(vals, best_val, group=self.group)
+        torch.distributed.all_gather(idxs, best_idx, group=self.group)
+        v = torch.stack(vals)              # [ranks, n]; shards are in vocabulary order,
+        win = torch.argmax(v, dim=0)       # and argmax returns the first maximum
+        best_idx.copy_(torch.stack(idxs).gather(0, win[None])[0])
+
+    def advance(self) -> None:
+        """Feed the greedy tokens back and move every sequence one position on."""
+        self.token_ids.copy_(self.best_idx)
+        self.positions.add_(1)
+
+    def capture(self) -> None:
+        """Record step() + advance() into a CUDA graph (after a few eager warm-up steps)."""
+        torch = self.torch
+        stream = torch.cuda.Stream()
+        stream.wait_stream(torch.cuda.current_stream())
+        saved = [t.clone() for t in self._step_inputs()]
+        if self.keeps_state:
+            self._make_idle()   # (the warm-up steps below must not move any sequence on)
+        with torch.cuda.stream(stream):
+            self.ctx.set_stream(stream.cuda_stream)
+            for _ in range(2):
+                self.step()
+        torch.cuda.current_stream().wait_stream(stream)
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        n0 = self.ctx.launch_count
+        with torch.cuda.graph(graph, stream=stream):  # the context already launches on `stream`
+            self.step()
+            self.advance()
+        self.kernels_per_step = self.ctx.launch_count - n0   # this library's kernels in the graph
+        for t, s in zip(self._step_inputs(), saved):
+            t.copy_(s)
+        torch.cuda.synchronize()
+        self.graph = graph
+
+    def start(self, token_ids, positions) -> None:
+        torch = self.torch
+        check_cache_capacity(positions, 1, self.cfg.max_seq)
+        self._host_positions = [int(p) for p in positions]
+        self.token_ids.copy_(torch.as_tensor(token_ids, dtype=torch.int32))
+        self.positions.copy_(torch.as_tensor(positions, dtype=torch.int32))
+
+    def decode(self, n_steps: int) -> np.ndarray:
+        """Greedy decode; returns the [n_steps, batch] generated ids."""
+        check_cache_capacity([p for p in self._host_positions if p is not None], n_steps, self.cfg.max_seq)
+        self._host_positions = [None if p is None else p + n_steps for p in self._host_positions]
+        out = []
+        for _ in range(n_steps):
+            if self.graph is not None:
+                self.graph.replay()
+            else:
+                self.step()
+                self.advance()
+            out.append(self.token_ids.clone())
+        self.torch.cuda.synchronize()
+        self.ctx.synchronize()   # also reports a device-side wait that gave up or a skipped token
+        return self.torch.stack(out).cpu().numpy()
+
+    def generate(self, prompt_tokens, max_tokens: int, eos_token_id: int | None = None) -> dict:
+        """Greedy generation for one sequence, with the control flow of the reference's
+        ``Engine::decode_start`` / ``push_token`` / ``decode_step`` / ``generate``
+        (engine/mod.rs:1377-1500): the prompt goes through the trunk one position at a time
+        over the device-resident KV cache, the first token is the argmax at the last prompt
+        position, EOS ends the generation without being part of it (finish ``"stop"``), and
+        the completion ends at ``max_tokens`` tokens (finish ``"length"``; as in the
+        reference the first token is kept even when ``max_tokens`` is 0).  ``prompt_ms`` is the
+        prefill span rounded up to a whole millisecond, at least 1.  Stop strings are text-side
+        (they need the tokenizer) and stay with the caller.
+        """
+        import math
+        import time
+        prompt = [int(t) for t in prompt_tokens]
+        if not prompt:
+            raise ValueError("prompt tokenized to zero tokens")
+        if self.cfg.max_batch != 1:
+            raise ValueError("generate serves one sequence: build the decoder with max_batch=1")
+        if len(prompt) + max(int(max_tokens), 1) > self.cfg.max_seq:
+            raise ValueError(f"prompt of {len(prompt)} tokens plus {max_tokens} new tokens does "
+                             f"not fit the KV cache of {self.cfg.max_seq} positions")
+        for tok in prompt:
+            if not 0 <= tok < self.cfg.vocab:
+                raise ValueError(f"token id {tok} out of range (vocab_size {self.cfg.vocab})")
+        started = time.perf_counter()
+        if len(prompt) >= self.cfg.prefill_min_tokens:
+            self.prefill(prompt, seq=0, first_position=0)   # the whole prompt in one pass
+        else:
+            for pos, tok in enumerate(prompt):
+                self.start([tok], [pos])
+                self.step()
+        self.ctx.synchronize()
+        prompt_ms = max(1, math.ceil((time.perf_counter() - started) * 1000.0))
+        out, finish = [], None
+        while finish is None:
+            nxt = int(self.best_idx[0].item())
+            if eos_token_id is not None and nxt == int(eos_token_id):
+                finish = "stop"
+                break
+            out.append(nxt)
+            if len(out) >= int(max_tokens):
+                finish = "length"
+                break
+            self.advance()
+            self.step()
+        self.ctx.synchronize()
+        return {"prompt_tokens": len(prompt), "completion_tokens": out, "finish": finish,
+                "prompt_ms": prompt_ms}
+
+
+class Decoder(SlotDecoder):
     """Batched greedy decode on one GPU (one tensor-parallel rank)."""
 
     def __init__(self, ctx: GpuContext, cfg: DecoderConfig, weights: dict | None, tp_rank: int = 0,
@@ -421,9 +629,8 @@ class Decoder:
                     "o": group([("o", 1)]),
                     "gu": group([("gu", 2), ("gate", 1), ("up", 1)]),
                     "down": group([("down", 1)])})
-        self.graph = None
-        self.kernels_per_step = None
-        self._host_positions = [0] * B
+        self.head_width = d
+        self._setup_driver()
 
     # ------------------------------------------------------------------ tensor parallel
     def _upload(self, ctx, layer: dict, name: str) -> PackedLayer:
@@ -578,13 +785,8 @@ class Decoder:
             self._all_reduce(self.delta_mlp)
             pending = 1
         self._norm(pending, self.final_norm, None, xa, xb)
-        head_tag = QK_BF16 if cfg.serving == "bfloat16" else QK_F32
-        check(lib.qk_lm_head(c, _p(self.h), _p(self.lm_head), head_tag, B, self.v_loc, d,
-                             self.v_loc, _p(self.logits)))
-        check(lib.qk_argmax_first(c, _p(self.logits), B, self.v_loc, self.v_loc, self.vocab_offset,
-                                  _p(self.best_val), _p(self.best_idx)))
-        if self.tp_size > 1:
-            self._gather_argmax(self.best_val, self.best_idx)
+        self._head(self.h, B, self.logits)
+        self._greedy(self.logits, B, self.best_val, self.best_idx)
 
     # ------------------------------------------------------------------ batched prefill
     def _prefill_buffers(self, n_tokens: int) -> dict:
@@ -623,200 +825,72 @@ class Decoder:
             for layer, dst in zip(layers, dsts):
                 layer.apply_device(src.data_ptr(), n_tokens, dst.data_ptr())
 
-    def prefill(self, tokens, seq: int = 0, first_position: int = 0) -> None:
-        """All of ``tokens`` (consecutive positions ``first_position ...`` of sequence slot ``seq``)
-        through the trunk in one pass per ``prefill_chunk`` positions: the batched form of the
-        reference's prompt loop (engine/mod.rs:1393-1413, one ``transformer`` call per prompt
-        token).  Appends the keys and values of every position to the cache and leaves the
-        greedy token of the last position in ``best_idx[seq]``; ``advance()`` + ``step()`` then
-        continue the sequence.  Only the last position goes through the final norm and the head."""
+    def _prefill_portion(self, part, seq: int, p0: int, reserve: int) -> None:
         torch, lib, c, cfg = self.torch, _lib.lib(), self.ctx.handle, self.cfg
-        toks = [int(t) for t in tokens]
-        if not toks:
-            raise ValueError("prefill needs at least one token")
-        if not 0 <= seq < cfg.max_batch:
-            raise ValueError(f"sequence slot {seq} outside the batch of {cfg.max_batch}")
-        check_cache_capacity([first_position], len(toks), cfg.max_seq)
         B, d, hd = cfg.max_batch, cfg.d_model, cfg.head_dim
-        handle = self.ctx.stream
-        # (handles 0 and 1 are the legacy default stream, which torch wraps itself)
-        stream = torch.cuda.ExternalStream(handle) if handle > 2 else torch.cuda.default_stream()
-        stream.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(stream):
-            for c0 in range(0, len(toks), cfg.prefill_chunk):
-                part = toks[c0:c0 + cfg.prefill_chunk]
-                T, p0 = len(part), first_position + c0
-                pf = self._prefill_buffers(min(len(toks), cfg.prefill_chunk))
-                pf["ids"][:T].copy_(torch.tensor(part, dtype=torch.int32), non_blocking=False)
-                pf["pos"][:T].copy_(torch.arange(p0, p0 + T, dtype=torch.int32))
-                pf["seq"][:T].fill_(seq)
-                check(lib.qk_embed(c, _p(self.embedding), self.emb_tag, _p(pf["ids"]), T, d, cfg.vocab,
-                                   _p(pf["x"])))
-                pending = None
-                for li in range(cfg.n_layers):
-                    in_w, post_w = self.norms[li]
-                    check(lib.qk_rmsnorm(c, _p(pf["x"]), pending, _p(in_w), T, d, cfg.rms_eps,
-                                         self.serving_tag, _p(pf["x"]), _p(pf["h"])))
-                    self._prefill_linears(li, ["q", "k", "v"], pf["h"], [pf["q"], pf["k"], pf["v"]], T)
-                    if self.qk_norms[li] is not None:
-                        for src, dst, wgt, heads in ((pf["q"], pf["qn"], self.qk_norms[li][0], self.h_loc),
-                                                     (pf["k"], pf["kn"], self.qk_norms[li][1], self.kv_loc)):
-                            check(lib.qk_rmsnorm(c, _p(src), None, _p(wgt), T * heads, hd, cfg.rms_eps,
-                                                 self.serving_tag, _p(src), _p(dst)))
-                    check(lib.qk_rope_cache(c, _p(pf["qn"]), _p(pf["kn"]), _p(pf["v"]), _p(self.cos_sin),
-                                            _p(pf["pos"]), _p(pf["seq"]), _p(self.cache_k[li]),
-                                            _p(self.cache_v[li]), self.kv_tag, T, self.h_loc,
-                                            self.kv_loc, hd, cfg.max_seq, B))
-                    check(lib.qk_prefill_attention(c, _p(pf["qn"]), _p(self.cache_k[li]),
-                                                   _p(self.cache_v[li]), self.kv_tag, seq, p0, T,
-                                                   self.h_loc, self.kv_loc, hd, cfg.max_seq,
-                                                   _p(pf["attn"])))
-                    self._prefill_linears(li, ["o"], pf["attn"], [pf["delta"]], T)
-                    if self.tp_size > 1:
-                        torch.distributed.all_reduce(pf["delta"][:T], group=self.group)
-                    check(lib.qk_rmsnorm(c, _p(pf["x"]), _p(pf["delta"]), _p(post_w), T, d, cfg.rms_eps,
-                                         self.serving_tag, _p(pf["x"]), _p(pf["h"])))
-                    self._prefill_linears(li, ["gate", "up"], pf["h"], [pf["g"], pf["u"]], T)
-                    if cfg.serving == "bfloat16" and T >= cfg.gemm_min_batch:
-                        apply_prefill_many_gated([self.layers[li]["down"]], pf["g"].data_ptr(), pf["u"].data_ptr(),
-                                                 T, [pf["delta"].data_ptr()])
-                    else:
-                        check(lib.qk_swiglu(c, _p(pf["g"]), _p(pf["u"]), T * self.ff_loc, _p(pf["a"])))
-                        self._prefill_linears(li, ["down"], pf["a"], [pf["delta"]], T)
-                    if self.tp_size > 1:
-                        torch.distributed.all_reduce(pf["delta"][:T], group=self.group)
-                    pending = _p(pf["delta"])
-            # the last position alone: final norm, head, greedy choice
-            last_x, last_delta = pf["x"][T - 1:T], pf["delta"][T - 1:T]
-            check(lib.qk_rmsnorm(c, _p(last_x), _p(last_delta) if pending is not None else None,
-                                 _p(self.final_norm), 1, d, cfg.rms_eps, self.serving_tag, _p(last_x),
-                                 _p(self.h[seq:seq + 1])))
-            head_tag = QK_BF16 if cfg.serving == "bfloat16" else QK_F32
-            check(lib.qk_lm_head(c, _p(self.h[seq:seq + 1]), _p(self.lm_head), head_tag, 1, self.v_loc, d,
-                                 self.v_loc, _p(self.logits[seq:seq + 1])))
-            check(lib.qk_argmax_first(c, _p(self.logits[seq:seq + 1]), 1, self.v_loc, self.v_loc,
-                                      self.vocab_offset, _p(self.best_val[seq:seq + 1]),
-                                      _p(self.best_idx[seq:seq + 1])))
+        T = len(part)
+        pf = self._prefill_buffers(reserve)
+        pf["ids"][:T].copy_(torch.tensor(part, dtype=torch.int32), non_blocking=False)
+        pf["pos"][:T].copy_(torch.arange(p0, p0 + T, dtype=torch.int32))
+        pf["seq"][:T].fill_(seq)
+        check(lib.qk_embed(c, _p(self.embedding), self.emb_tag, _p(pf["ids"]), T, d, cfg.vocab,
+                           _p(pf["x"])))
+        pending = None
+        for li in range(cfg.n_layers):
+            in_w, post_w = self.norms[li]
+            check(lib.qk_rmsnorm(c, _p(pf["x"]), pending, _p(in_w), T, d, cfg.rms_eps,
+                                 self.serving_tag, _p(pf["x"]), _p(pf["h"])))
+            self._prefill_linears(li, ["q", "k", "v"], pf["h"], [pf["q"], pf["k"], pf["v"]], T)
+            if self.qk_norms[li] is not None:
+                for src, dst, wgt, heads in ((pf["q"], pf["qn"], self.qk_norms[li][0], self.h_loc),
+                                             (pf["k"], pf["kn"], self.qk_norms[li][1], self.kv_loc)):
+                    check(lib.qk_rmsnorm(c, _p(src), None, _p(wgt), T * heads, hd, cfg.rms_eps,
+                                         self.serving_tag, _p(src), _p(dst)))
+            check(lib.qk_rope_cache(c, _p(pf["qn"]), _p(pf["kn"]), _p(pf["v"]), _p(self.cos_sin),
+                                    _p(pf["pos"]), _p(pf["seq"]), _p(self.cache_k[li]),
+                                    _p(self.cache_v[li]), self.kv_tag, T, self.h_loc,
+                                    self.kv_loc, hd, cfg.max_seq, B))
+            check(lib.qk_prefill_attention(c, _p(pf["qn"]), _p(self.cache_k[li]),
+                                           _p(self.cache_v[li]), self.kv_tag, seq, p0, T,
+                                           self.h_loc, self.kv_loc, hd, cfg.max_seq,
+                                           _p(pf["attn"])))
+            self._prefill_linears(li, ["o"], pf["attn"], [pf["delta"]], T)
             if self.tp_size > 1:
-                self._gather_argmax(self.best_val[seq:seq + 1], self.best_idx[seq:seq + 1])
-            last = first_position + len(toks) - 1
-            self.token_ids[seq:seq + 1].fill_(toks[-1])
-            self.positions[seq:seq + 1].fill_(last)
-            self.kv_len[seq:seq + 1].fill_(last + 1)
-        stream.synchronize()
-        torch.cuda.current_stream().wait_stream(stream)
-        self._host_positions[seq] = last
-        self.ctx.synchronize()
+                torch.distributed.all_reduce(pf["delta"][:T], group=self.group)
+            check(lib.qk_rmsnorm(c, _p(pf["x"]), _p(pf["delta"]), _p(post_w), T, d, cfg.rms_eps,
+                                 self.serving_tag, _p(pf["x"]), _p(pf["h"])))
+            self._prefill_linears(li, ["gate", "up"], pf["h"], [pf["g"], pf["u"]], T)
+            if cfg.serving == "bfloat16" and T >= cfg.gemm_min_batch:
+                apply_prefill_many_gated([self.layers[li]["down"]], pf["g"].data_ptr(), pf["u"].data_ptr(),
+                                         T, [pf["delta"].data_ptr()])
+            else:
+                check(lib.qk_swiglu(c, _p(pf["g"]), _p(pf["u"]), T * self.ff_loc, _p(pf["a"])))
+                self._prefill_linears(li, ["down"], pf["a"], [pf["delta"]], T)
+            if self.tp_size > 1:
+                torch.distributed.all_reduce(pf["delta"][:T], group=self.group)
+            pending = _p(pf["delta"])
 
-    def _gather_argmax(self, best_val, best_idx) -> None:
-        """Vocabulary-parallel head: the first maximum over the ranks' shard winners."""
-        torch = self.torch
-        vals = [torch.empty_like(best_val) for _ in range(self.tp_size)]
-        idxs = [torch.empty_like(best_idx) for _ in range(self.tp_size)]
-        torch.distributed.all_gather(vals, best_val, group=self.group)
-        torch.distributed.all_gather(idxs, best_idx, group=self.group)
-        v = torch.stack(vals)              # [ranks, n]; shards are in vocabulary order,
-        win = torch.argmax(v, dim=0)       # and argmax returns the first maximum
-        best_idx.copy_(torch.stack(idxs).gather(0, win[None])[0])
+    def _portion_hidden(self, rows, out) -> None:
+        cfg, pf = self.cfg, self._pf
+        if len(rows) == 1:
+            x, delta = pf["x"][rows[0]:rows[0] + 1], pf["delta"][rows[0]:rows[0] + 1]
+        else:
+            idx = self.torch.as_tensor(rows, device=out.device)
+            x, delta = pf["x"].index_select(0, idx), pf["delta"].index_select(0, idx)
+        check(_lib.lib().qk_rmsnorm(self.ctx.handle, _p(x), _p(delta), _p(self.final_norm), len(rows),
+                                    cfg.d_model, cfg.rms_eps, self.serving_tag, None, _p(out)))
+
+    def _reset_slot(self, seq: int, token: int, position: int) -> None:
+        super()._reset_slot(seq, token, position)
+        self.kv_len[seq:seq + 1].fill_(position + 1)
 
     def advance(self) -> None:
-        """Feed the greedy tokens back and move every sequence one position on."""
-        self.token_ids.copy_(self.best_idx)
-        self.positions.add_(1)
+        super().advance()
         self.kv_len.add_(1)
 
-    def capture(self) -> None:
-        """Record step() + advance() into a CUDA graph (after a few eager warm-up steps)."""
-        torch = self.torch
-        stream = torch.cuda.Stream()
-        stream.wait_stream(torch.cuda.current_stream())
-        saved = [t.clone() for t in (self.token_ids, self.positions, self.kv_len)]
-        with torch.cuda.stream(stream):
-            self.ctx.set_stream(stream.cuda_stream)
-            for _ in range(2):
-                self.step()
-        torch.cuda.current_stream().wait_stream(stream)
-        torch.cuda.synchronize()
-        graph = torch.cuda.CUDAGraph()
-        n0 = self.ctx.launch_count
-        with torch.cuda.graph(graph, stream=stream):  # the context already launches on `stream`
-            self.step()
-            self.advance()
-        self.kernels_per_step = self.ctx.launch_count - n0   # this library's kernels in the graph
-        for t, s in zip((self.token_ids, self.positions, self.kv_len), saved):
-            t.copy_(s)
-        torch.cuda.synchronize()
-        self.graph = graph
+    def _step_inputs(self) -> list:
+        return [self.token_ids, self.positions, self.kv_len]
 
     def start(self, token_ids, positions) -> None:
-        torch = self.torch
-        check_cache_capacity(positions, 1, self.cfg.max_seq)
-        self._host_positions = [int(p) for p in positions]
-        self.token_ids.copy_(torch.as_tensor(token_ids, dtype=torch.int32))
-        self.positions.copy_(torch.as_tensor(positions, dtype=torch.int32))
+        super().start(token_ids, positions)
         self.kv_len.copy_(self.positions + 1)
-
-    def decode(self, n_steps: int) -> np.ndarray:
-        """Greedy decode; returns the [n_steps, batch] generated ids."""
-        check_cache_capacity(self._host_positions, n_steps, self.cfg.max_seq)
-        self._host_positions = [p + n_steps for p in self._host_positions]
-        out = []
-        for _ in range(n_steps):
-            if self.graph is not None:
-                self.graph.replay()
-            else:
-                self.step()
-                self.advance()
-            out.append(self.token_ids.clone())
-        self.torch.cuda.synchronize()
-        self.ctx.synchronize()   # also reports a device-side wait that gave up or a skipped token
-        return self.torch.stack(out).cpu().numpy()
-
-    def generate(self, prompt_tokens, max_tokens: int, eos_token_id: int | None = None) -> dict:
-        """Greedy generation for one sequence, with the control flow of the reference's
-        ``Engine::decode_start`` / ``push_token`` / ``decode_step`` / ``generate``
-        (engine/mod.rs:1377-1500): the prompt goes through the trunk one position at a time
-        over the device-resident KV cache, the first token is the argmax at the last prompt
-        position, EOS ends the generation without being part of it (finish ``"stop"``), and
-        the completion ends at ``max_tokens`` tokens (finish ``"length"``; as in the
-        reference the first token is kept even when ``max_tokens`` is 0).  ``prompt_ms`` is the
-        prefill span rounded up to a whole millisecond, at least 1.  Stop strings are text-side
-        (they need the tokenizer) and stay with the caller.
-        """
-        import math
-        import time
-        prompt = [int(t) for t in prompt_tokens]
-        if not prompt:
-            raise ValueError("prompt tokenized to zero tokens")
-        if self.cfg.max_batch != 1:
-            raise ValueError("generate serves one sequence: build the decoder with max_batch=1")
-        if len(prompt) + max(int(max_tokens), 1) > self.cfg.max_seq:
-            raise ValueError(f"prompt of {len(prompt)} tokens plus {max_tokens} new tokens does "
-                             f"not fit the KV cache of {self.cfg.max_seq} positions")
-        for tok in prompt:
-            if not 0 <= tok < self.cfg.vocab:
-                raise ValueError(f"token id {tok} out of range (vocab_size {self.cfg.vocab})")
-        started = time.perf_counter()
-        if len(prompt) >= self.cfg.prefill_min_tokens:
-            self.prefill(prompt, seq=0, first_position=0)   # the whole prompt in one pass
-        else:
-            for pos, tok in enumerate(prompt):
-                self.start([tok], [pos])
-                self.step()
-        self.ctx.synchronize()
-        prompt_ms = max(1, math.ceil((time.perf_counter() - started) * 1000.0))
-        out, finish = [], None
-        while finish is None:
-            nxt = int(self.best_idx[0].item())
-            if eos_token_id is not None and nxt == int(eos_token_id):
-                finish = "stop"
-                break
-            out.append(nxt)
-            if len(out) >= int(max_tokens):
-                finish = "length"
-                break
-            self.advance()
-            self.step()
-        self.ctx.synchronize()
-        return {"prompt_tokens": len(prompt), "completion_tokens": out, "finish": finish,
-                "prompt_ms": prompt_ms}
