@@ -556,6 +556,156 @@ qk_status qk_argmax_first(qk_ctx *ctx, const float *logits, size_t n_tokens, siz
                           size_t logits_stride, int32_t index_base, float *out_val,
                           int32_t *out_idx);
 
+/* ------------------------------------------------------------------ layered decoders
+ * Building blocks of decoders whose linears are dense (bfloat16 or float32 weights) and whose
+ * layers mix windowed latent attention with gated-delta-rule recurrences.  No reference
+ * counterpart.  All of them only launch kernels on the context's stream; device memory,
+ * including scratch, belongs to the caller.
+ *
+ * Every call works on `tokens` rows.  Row t is one token: positions[t] is its position in its
+ * sequence (negative: the row is idle; it changes no cache and no state), slots[t] the cache and
+ * state slot of that sequence. */
+
+/* How a dense linear forms its input vector from what it is given. */
+enum {
+    QK_INPUT_PLAIN = 0,   /* x */
+    QK_INPUT_NORM = 1,    /* h = x + pending; x_out = h; the input is norm(h) */
+    QK_INPUT_CONCAT = 2,  /* h as above; the input is [h ; second], each half k/2 entries */
+    QK_INPUT_GATED = 3,   /* x in groups of `group`: x / rms(group) * norm_weight * silu(gate) */
+};
+enum { QK_NORM_NONE = 0, QK_NORM_LAYER = 1, QK_NORM_RMS = 2 };
+enum { QK_ACT_RELU = 0, QK_ACT_SILU = 1, QK_ACT_GELU_TANH = 2 };
+/* What a dense linear does with its result v[t][n]. */
+enum {
+    QK_OUTPUT_STORE = 0,     /* out = v */
+    QK_OUTPUT_RESIDUAL = 1,  /* residual += v * out_scale (null: 1); out, when given, = the new residual */
+    QK_OUTPUT_GLU = 2,       /* rows come in blocks of 32 gate rows and 32 up rows: out = act(gate) * up */
+    QK_OUTPUT_SIDE = 3,      /* out = act(v) * side[ids[t]][side_offset + n] */
+};
+/* RMS norm of a latent and its append to a ring cache: the row of position p of a slot is
+ * cache[slot][p mod ring][stride] (entries from width on are written as zeros). */
+typedef struct {
+    const float *src;       /* null: nothing is appended; row t at src + t * src_stride */
+    size_t src_stride, width;
+    const float *weight;
+    float eps;
+    int32_t cache_dtype;
+    void *cache;
+    size_t ring, stride;
+} qk_latent_append;
+typedef struct {
+    size_t tokens;
+    const int32_t *positions, *slots, *ids;  /* per row; ids only for QK_OUTPUT_SIDE */
+    size_t vocab;                            /* rows of `side`: ids are clamped to it */
+    /* input: rows of `width` values; the weight rows have k >= width columns, k a multiple of 8 */
+    int32_t input, x_dtype;                  /* x_dtype QK_BF16 only with QK_INPUT_PLAIN */
+    const void *x;
+    size_t x_stride, width, k;
+    const float *pending;                    /* null: nothing pending */
+    size_t pending_stride;
+    const float *pending_weight;             /* pending value = y / rms(y) * pending_weight */
+    float pending_eps;
+    float *x_out;                            /* row stride x_stride; not x itself; null: not stored */
+    const float *second;                     /* QK_INPUT_CONCAT, row stride x_stride */
+    int32_t norm;
+    float norm_eps;
+    const float *norm_weight;
+    const float *gate;                       /* QK_INPUT_GATED */
+    size_t gate_stride, group;
+    qk_latent_append append;                 /* done beside the linear, with any input */
+    /* weights [rows][w_stride]; columns past width are zero */
+    int32_t w_dtype;
+    const void *w;
+    size_t rows, w_stride;
+    /* output */
+    int32_t output, activation, out_dtype;
+    void *out;
+    size_t out_stride;
+    float *residual;
+    size_t residual_stride;
+    const float *out_scale;
+    const void *side;
+    int32_t side_dtype;
+    size_t side_stride, side_offset;
+    /* scratch for the input rows of the matrix forms: tokens * k * (2 or 4) bytes */
+    void *scratch;
+    size_t scratch_bytes;
+} qk_dense_call;
+/* One dense linear.  Up to QK_DENSE_VECTOR_TOKENS rows (qk_dense_form says which form a shape
+ * takes) run as one launch that forms the input in every block; more rows as a launch for the
+ * input (none for a plain input of the weights' dtype) and a matrix product. */
+qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *call);
+enum { QK_FORM_VECTOR = 0, QK_FORM_SKINNY = 1, QK_FORM_TCGEN05 = 2, QK_FORM_F32 = 3 };
+int32_t qk_dense_form(size_t tokens, size_t k, int32_t w_dtype);
+/* Only the input rows: out [tokens][k] in out_dtype (stride k). */
+qk_status qk_dense_input(qk_ctx *ctx, const qk_dense_call *call);
+
+/* x[t] = table[ids[t]] * scale + sinusoid(positions[t]): entry 2i is sin(p f_i), 2i+1 cos(p f_i),
+ * f_i = inv_freq[i] (float64); inv_freq null: no positions.  Idle rows are zero.  x_copy, when
+ * given, gets the same rows. */
+qk_status qk_embed_scaled(qk_ctx *ctx, const void *table, int32_t table_dtype, size_t table_stride,
+                          const int32_t *ids, const int32_t *positions, size_t tokens, size_t width,
+                          size_t vocab, float scale, const double *inv_freq, float *x, float *x_copy,
+                          size_t x_stride);
+
+/* Gated delta rule.  proj holds, per row (stride proj_stride): q [kv_heads*dim] k [kv_heads*dim]
+ * v [heads*vdim], and at beta_offset / decay_offset the two per-head projections.  conv_q/k/v
+ * [channels][taps] float32.  Rows of one sequence portion are consecutive; segment s is rows
+ * seg_first[s] .. + seg_len[s] - 1.  conv_state [slots][taps][channels] (ring by position),
+ * state [slots][heads][vdim][dim] float32 (per output channel the dim values it is read from).
+ * A portion that starts at position 0 starts from zero. */
+typedef struct {
+    size_t tokens, segments;
+    const int32_t *positions, *slots;        /* per row */
+    const int32_t *seg_first, *seg_len;      /* per segment, on the device */
+    const int32_t *seg_row;                  /* per row: its place in its segment */
+    size_t heads, kv_heads, dim, vdim, taps;
+    const float *proj;
+    size_t proj_stride, beta_offset, decay_offset;
+    const float *conv_q, *conv_k, *conv_v, *a_log, *dt_bias;
+    float unit_eps;
+    float *conv_state, *state;
+    float *qkv;                              /* scratch [tokens][2*kv_heads*dim + heads*vdim] */
+    float *gates;                            /* scratch [tokens][heads][4] */
+    float *out;                              /* [tokens][heads*vdim], stride out_stride */
+    size_t out_stride;
+} qk_delta_call;
+qk_status qk_delta(qk_ctx *ctx, const qk_delta_call *call);
+
+/* Windowed attention over a latent ring cache (qk_latent_append).  q [tokens][heads][dim_stride]
+ * float32; uk [heads*dim_stride][kv_stride] and uv [heads*vdim_stride][kv_stride] in w_dtype.
+ * A row at position p sees positions max(0, p - window + 1) .. p; every one of them must still
+ * be in the ring.  out [tokens][heads*vdim], stride out_stride. */
+typedef struct {
+    size_t tokens;
+    const int32_t *positions, *slots;
+    size_t heads, dim, dim_stride, vdim, vdim_stride, kv_rank, kv_stride;
+    size_t window, ring, n_slots;
+    float scale;
+    const void *q;                           /* float32; bfloat16 in the expanded form */
+    int32_t q_dtype;
+    size_t q_stride;
+    int32_t w_dtype;                         /* weights and cache */
+    const void *uk, *uv, *cache;
+    size_t n_splits;
+    float *scratch;                          /* qk_latent_scratch() bytes */
+    void *out;
+    int32_t out_dtype;
+    size_t out_stride;
+} qk_latent_call;
+/* Absorbed form, any mix of rows: scores of W_uk^T q against the cached latents. */
+qk_status qk_latent_attention(qk_ctx *ctx, const qk_latent_call *call);
+size_t qk_latent_scratch(size_t tokens, size_t heads, size_t kv_stride, size_t n_splits);
+/* Rows first .. first + count - 1 (positions) of one slot's ring, gathered into consecutive rows. */
+qk_status qk_latent_gather(qk_ctx *ctx, const void *cache, int32_t dtype, size_t ring, size_t stride,
+                           size_t slot, size_t first, size_t count, void *out);
+/* Expanded form, one sequence portion at positions first_position .. + tokens - 1, bfloat16:
+ * kv [keys][kv_row] holds k (heads*dim_stride) and v (heads*vdim_stride) of positions key0 .. */
+qk_status qk_window_attention(qk_ctx *ctx, const void *q, size_t q_stride, const void *kv, size_t kv_row,
+                              size_t key0, size_t n_keys, size_t first_position, size_t tokens, size_t heads,
+                              size_t dim_stride, size_t vdim, size_t vdim_stride, size_t window, float scale,
+                              void *out, size_t out_stride);
+
 /* Which GEMV kernel qk_layer_apply and the group calls use: 0 = sign-select SIMT, 1 = bit-sliced
  * INT8 tensor-core (default; many instances per launch run in the persistent streaming form),
  * 3 = the same without the split-k form, 5 = the same with one block per instance instead of

@@ -153,6 +153,19 @@ _SIGNATURES = {
     "qk_gpu_sage_quantize": (c_int32, [c_void_p, c_void_p, c_void_p, c_size_t, c_void_p, c_size_t,
                                        c_void_p, c_size_t, c_size_t, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_void_p, c_void_p, c_void_p]),
+    "qk_dense": (c_int32, [c_void_p, c_void_p]),
+    "qk_dense_form": (c_int32, [c_size_t, c_size_t, c_int32]),
+    "qk_dense_input": (c_int32, [c_void_p, c_void_p]),
+    "qk_embed_scaled": (c_int32, [c_void_p, c_void_p, c_int32, c_size_t, c_void_p, c_void_p, c_size_t, c_size_t,
+                                  c_size_t, c_float, c_void_p, c_void_p, c_void_p, c_size_t]),
+    "qk_delta": (c_int32, [c_void_p, c_void_p]),
+    "qk_latent_attention": (c_int32, [c_void_p, c_void_p]),
+    "qk_latent_scratch": (c_size_t, [c_size_t, c_size_t, c_size_t, c_size_t]),
+    "qk_latent_gather": (c_int32, [c_void_p, c_void_p, c_int32, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t,
+                                   c_void_p]),
+    "qk_window_attention": (c_int32, [c_void_p, c_void_p, c_size_t, c_void_p, c_size_t, c_size_t, c_size_t, c_size_t,
+                                      c_size_t, c_size_t, c_size_t, c_size_t, c_size_t, c_size_t, c_float, c_void_p,
+                                      c_size_t]),
     "qk_set_wait_limit": (ctypes.c_uint32, [c_void_p, ctypes.c_uint32]),
     "qk_set_dependent_launch": (c_int32, [c_void_p, c_int32]),
 }

@@ -1,0 +1,996 @@
+// Dense linears y = W x with bfloat16 or float32 weights, in four forms:
+//   * vector (up to kVectorTokens rows): one launch; every block forms the input vectors itself
+//     (norm, pending residual, gate - see qk_dense_dev.cuh) and its warps stream weight rows;
+//   * skinny (bfloat16, up to kSkinnyTokens rows): mma.sync, the weights on the M side and read
+//     once, straight from global memory into fragments, the rows on the N side;
+//   * tcgen05 (bfloat16, more rows): TMA-fed tcgen05.mma with the accumulators in tensor memory;
+//   * float32 (more rows, float32 weights): plain float32 multiply-adds, no reduced-precision
+//     matrix mode.
+// The matrix forms take their input rows from a kernel that runs the same device function as
+// the vector form.  All forms share the epilogues.
+#include <cuda.h>  // CUtensorMap types only; the encoder is fetched through the runtime
+
+#include <algorithm>
+
+#include "qk_dense_dev.cuh"
+#include "qk_umma.cuh"
+
+namespace {
+
+constexpr int kVecThreads = 256, kVecWarps = kVecThreads / 32;
+constexpr int kVectorTokens = 4;
+constexpr int kSkinnyTokens = 64;
+constexpr size_t kVecSmemMax = 200 * 1024;
+
+// ------------------------------------------------------------------ vector form
+template <typename W> struct VecTraits;
+template <> struct VecTraits<uint16_t> {
+    static constexpr uint32_t kPer = 8, kStep = 32 * 8;  // entries per lane and per warp step
+    // A lane reads entries 8l .. 8l+7 of a 256-entry step as two 16-byte pieces: the first
+    // halves of all lanes lie side by side, then the second halves, so that a warp's reads hit
+    // every bank once.
+    __device__ static uint32_t place(uint32_t i) {
+        return (i & ~255u) | ((i & 4u) << 5) | ((i & 248u) >> 1) | (i & 3u);
+    }
+};
+template <> struct VecTraits<float> {
+    static constexpr uint32_t kPer = 4, kStep = 32 * 4;
+    __device__ static uint32_t place(uint32_t i) { return i; }
+};
+
+__device__ __forceinline__ uint4 load_weights16(const void *p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
+                 : "l"(p));
+    return v;
+}
+
+template <typename W, int NT>
+__device__ __forceinline__ void vec_fma(float (&acc)[NT], const uint4 &w, const float *xs, uint32_t pitch,
+                                        uint32_t at, uint32_t lane) {
+    if constexpr (sizeof(W) == 2) {
+        const uint32_t u[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            const float *p = xs + t * pitch + at + lane * 4;
+            const float4 a = *reinterpret_cast<const float4 *>(p);
+            const float4 b = *reinterpret_cast<const float4 *>(p + 128);
+            const float v[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                acc[t] = fmaf(__uint_as_float(u[e] << 16), v[2 * e], acc[t]);
+                acc[t] = fmaf(__uint_as_float(u[e] & 0xffff0000u), v[2 * e + 1], acc[t]);
+            }
+        }
+    } else {
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            const float4 a = *reinterpret_cast<const float4 *>(xs + t * pitch + at + lane * 4);
+            acc[t] = fmaf(__uint_as_float(w.x), a.x, acc[t]);
+            acc[t] = fmaf(__uint_as_float(w.y), a.y, acc[t]);
+            acc[t] = fmaf(__uint_as_float(w.z), a.z, acc[t]);
+            acc[t] = fmaf(__uint_as_float(w.w), a.w, acc[t]);
+        }
+    }
+}
+
+// A warp (or `ksplit` warps that share out the k range) owns R weight rows; with a gated pair,
+// R / 2 gate rows and their up rows.
+template <typename W, int NT, int R>
+__global__ void __launch_bounds__(kVecThreads)
+dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint32_t rows, uint32_t w_stride,
+                    uint32_t n_tokens, uint32_t ksplit) {
+    using T = VecTraits<W>;
+    constexpr int U = R >= 4 ? 2 : 4;  // steps in flight
+    constexpr int HR = R >= 2 ? R / 2 : 1;
+    qk::pdl_launch();
+    extern __shared__ __align__(16) float xs[];  // [NT][pitch]
+    __shared__ float red[kVecWarps];
+    __shared__ float part_sum[kVecWarps][R * NT];
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const uint32_t k = in.k, pitch = (k + T::kStep - 1) / T::kStep * T::kStep, steps = pitch / T::kStep;
+    const uint32_t group = (blockIdx.x * kVecWarps + warp) / ksplit, part = warp % ksplit;
+    const bool pair = out.kind == QK_OUTPUT_GLU;
+    const W *row[R];
+    uint32_t r0 = group * R;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        uint32_t n;
+        if (pair) n = pair_row(group * HR + r % HR) + (r >= HR ? 32 : 0);
+        else n = r0 + r;
+        row[r] = w + (size_t)min(n, rows - 1) * w_stride + lane * T::kPer;
+    }
+    uint4 cur[U][R];
+    auto fetch = [&](uint32_t s, uint4 (&dst)[R]) {
+        const bool live = s < steps && s * T::kStep + lane * T::kPer < k;
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+            dst[r] = live ? load_weights16(row[r] + (size_t)s * T::kStep) : make_uint4(0, 0, 0, 0);
+    };
+    // weights depend on no other kernel: the first ones are requested before the dependency wait
+#pragma unroll
+    for (int u = 0; u < U; ++u) fetch(part + u * ksplit, cur[u]);
+    qk::pdl_wait();
+#pragma unroll 1
+    for (uint32_t t = 0; t < (uint32_t)NT; ++t) {
+        float *dst = xs + t * pitch;
+        if (t < n_tokens) {
+            build_input(in, t, blockIdx.x == 0, [&](uint32_t i) -> float & { return dst[T::place(i)]; }, red);
+        }
+        // what lies between k and the pitch meets zero weights; it must only be finite
+        for (uint32_t i = (t < n_tokens ? k : 0) + threadIdx.x; i < pitch; i += kVecThreads) dst[T::place(i)] = 0.f;
+    }
+    __syncthreads();
+    float acc[R][NT];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+        for (int t = 0; t < NT; ++t) acc[r][t] = 0.f;
+    for (uint32_t s = part; s < steps; s += U * ksplit) {
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            uint4 now[R];
+#pragma unroll
+            for (int r = 0; r < R; ++r) now[r] = cur[u][r];
+            const uint32_t at = s + u * ksplit;
+            fetch(at + U * ksplit, cur[u]);
+            if (at < steps) {
+#pragma unroll
+                for (int r = 0; r < R; ++r) vec_fma<W, NT>(acc[r], now[r], xs, pitch, at * T::kStep, lane);
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+            float a = acc[r][t];
+            for (int off = 16; off > 0; off >>= 1) a += __shfl_xor_sync(0xffffffffu, a, off);
+            acc[r][t] = a;
+        }
+    if (ksplit > 1) {
+        if (lane == 0) {
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+#pragma unroll
+                for (int t = 0; t < NT; ++t) part_sum[warp][r * NT + t] = acc[r][t];
+        }
+        __syncthreads();
+        if (part == 0) {
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+#pragma unroll
+                for (int t = 0; t < NT; ++t)
+                    for (uint32_t p = 1; p < ksplit; ++p) acc[r][t] += part_sum[warp + p][r * NT + t];
+        }
+    }
+    if (part == 0) {
+        if (pair) {
+            if constexpr (R >= 2) {
+#pragma unroll
+                for (int r = 0; r < R / 2; ++r)
+#pragma unroll
+                    for (int t = 0; t < NT; ++t) {
+                        const uint32_t j = group * (R / 2) + r;
+                        if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && j < rows / 2)
+                            finish_pair(out, t, j, acc[r][t], acc[r + R / 2][t]);
+                    }
+            }
+        } else {
+#pragma unroll
+            for (int r = 0; r < R; ++r)
+#pragma unroll
+                for (int t = 0; t < NT; ++t)
+                    if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && r0 + r < rows)
+                        finish(out, t, r0 + r, acc[r][t]);
+        }
+    }
+    if (in.append.src && blockIdx.x == gridDim.x - 1)
+        for (uint32_t t = 0; t < n_tokens; ++t) append_latent(in, t, red);
+}
+
+// ------------------------------------------------------------------ input rows of the matrix forms
+template <typename A>
+__global__ void __launch_bounds__(256)
+dense_input_kernel(InputArgs in, A *__restrict__ dst) {
+    qk::pdl_launch();
+    qk::pdl_wait();
+    extern __shared__ __align__(16) float row_smem[];
+    __shared__ float red[8];
+    const uint32_t t = blockIdx.x;
+    if (dst) {
+        build_input(in, t, true, [&](uint32_t i) -> float & { return row_smem[i]; }, red);
+        A *o = dst + (size_t)t * in.k;
+        if constexpr (sizeof(A) == 2) {
+            for (uint32_t i = threadIdx.x * 2; i < in.k; i += 512) {  // (k is a multiple of 8)
+                const uint32_t lo = float_to_bf16_bits(row_smem[i]), hi = float_to_bf16_bits(row_smem[i + 1]);
+                *reinterpret_cast<uint32_t *>(o + i) = lo | (hi << 16);
+            }
+        } else {
+            for (uint32_t i = threadIdx.x; i < in.k; i += 256) o[i] = row_smem[i];
+        }
+    }
+    if (in.append.src) append_latent(in, t, red);
+}
+
+// ------------------------------------------------------------------ skinny form
+__device__ __forceinline__ void sk_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
+                                       uint32_t b0, uint32_t b1) {
+    asm volatile(
+        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
+        "{%0,%1,%2,%3};"
+        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void sk_copy16(void *smem, const void *gmem, uint32_t bytes) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)),
+                 "l"(gmem), "r"(bytes)
+                 : "memory");
+}
+constexpr int kSkWarps = 8, kSkPitch = 96;  // bf16 entries per staged row: 64 k + 32 pad
+
+// A warp owns two tiles of 16 weight rows (32 consecutive rows, or 16 gate rows and their up
+// rows) and every ksplit-th chunk of 64 k; the staged x chunks of all ksplit parts are shared by
+// the block.  k order inside a 32-wide group as in the LM head's kernel: one 16-byte load feeds
+// two MMAs on either operand.
+template <int NT>
+__global__ void __launch_bounds__(kSkWarps * 32)
+dense_skinny_kernel(const uint16_t *__restrict__ x, uint32_t x_stride, uint32_t k,
+                    const uint16_t *__restrict__ w, uint32_t rows, uint32_t w_stride, uint32_t n_tokens,
+                    uint32_t ksplit, OutputArgs out) {
+    qk::pdl_launch();
+    extern __shared__ __align__(16) uint8_t sk_smem[];
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane >> 2, t = lane & 3;
+    const uint32_t part = warp % ksplit, tile = (blockIdx.x * kSkWarps + warp) / ksplit;
+    const bool pair = out.kind == QK_OUTPUT_GLU;
+    uint32_t first[2];
+    if (pair) {
+        first[0] = pair_row(tile * 16);
+        first[1] = first[0] + 32;
+    } else {
+        first[0] = tile * 32;
+        first[1] = first[0] + 16;
+    }
+    const uint16_t *row[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+        row[i] = w + (size_t)min(first[i / 2] + g + (i % 2) * 8, rows - 1) * w_stride + 8 * t;
+    const uint32_t chunks = (k + 63) / 64, rounds = (chunks + ksplit - 1) / ksplit;
+    auto fetch = [&](uint32_t round, uint4 (&dst)[4][2]) {
+        const uint32_t c = round * ksplit + part;
+#pragma unroll
+        for (int gi = 0; gi < 2; ++gi) {
+            const uint32_t col = c * 64 + gi * 32;
+            const bool live = c < chunks && col + 8 * t < k;
+#pragma unroll
+            for (int i = 0; i < 4; ++i) dst[i][gi] = live ? load_weights16(row[i] + col) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    const uint32_t buf_elems = ksplit * 8 * NT * kSkPitch;
+    uint16_t *stage_base = reinterpret_cast<uint16_t *>(sk_smem);
+    auto stage = [&](uint32_t round, uint32_t buf) {
+        for (uint32_t idx = threadIdx.x; idx < ksplit * 8 * NT * 8; idx += kSkWarps * 32) {
+            const uint32_t piece = idx % 8, tok = (idx / 8) % (8 * NT), p = idx / (8 * 8 * NT);
+            const uint32_t col = (round * ksplit + p) * 64 + piece * 8;
+            const bool live = tok < n_tokens && col < k;
+            sk_copy16(stage_base + buf * buf_elems + (p * 8 * NT + tok) * kSkPitch + piece * 8,
+                      x + (live ? (size_t)tok * x_stride + col : 0), live ? 16u : 0u);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    float acc[2][NT][4];
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) acc[m][nt][0] = acc[m][nt][1] = acc[m][nt][2] = acc[m][nt][3] = 0.f;
+    uint4 nxt[4][2];
+    fetch(0, nxt);
+    qk::pdl_wait();
+    stage(0, 0);
+    for (uint32_t c = 0; c < rounds; ++c) {
+        uint4 cur[4][2];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) cur[i][0] = nxt[i][0], cur[i][1] = nxt[i][1];
+        fetch(c + 1, nxt);
+        if (c + 1 < rounds) {
+            stage(c + 1, (c + 1) & 1);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
+        }
+        __syncthreads();
+        const uint16_t *xb = stage_base + (c & 1) * buf_elems + part * 8 * NT * kSkPitch;
+#pragma unroll
+        for (int gi = 0; gi < 2; ++gi)
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) {
+                const uint4 b = *reinterpret_cast<const uint4 *>(xb + (8 * nt + g) * kSkPitch + gi * 32 + 8 * t);
+#pragma unroll
+                for (int m = 0; m < 2; ++m) {
+                    const uint4 lo = cur[2 * m][gi], hi = cur[2 * m + 1][gi];
+                    sk_mma(acc[m][nt], lo.x, hi.x, lo.y, hi.y, b.x, b.y);
+                    sk_mma(acc[m][nt], lo.z, hi.z, lo.w, hi.w, b.z, b.w);
+                }
+            }
+        __syncthreads();
+    }
+    if (ksplit > 1) {
+        // the parts' sums, part 0 first: [warp][value][lane]
+        float *sums = reinterpret_cast<float *>(sk_smem);
+        constexpr int kVals = 2 * NT * 4;
+        if (part != 0) {
+#pragma unroll
+            for (int m = 0; m < 2; ++m)
+#pragma unroll
+                for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e)
+                        sums[((size_t)warp * kVals + (m * NT + nt) * 4 + e) * 32 + lane] = acc[m][nt][e];
+        }
+        __syncthreads();
+        if (part == 0) {
+            for (uint32_t p = 1; p < ksplit; ++p)
+#pragma unroll
+                for (int m = 0; m < 2; ++m)
+#pragma unroll
+                    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e)
+                            acc[m][nt][e] += sums[((size_t)(warp + p) * kVals + (m * NT + nt) * 4 + e) * 32 + lane];
+        }
+    }
+    if (part != 0) return;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const uint32_t tok = 8 * nt + 2 * t + (e & 1), r = g + (e >> 1) * 8;
+            if (tok >= n_tokens) continue;
+            if (pair) {
+                if (tile * 16 + r < rows / 2) finish_pair(out, tok, tile * 16 + r, acc[0][nt][e], acc[1][nt][e]);
+            } else {
+                if (first[0] + r < rows) finish(out, tok, first[0] + r, acc[0][nt][e]);
+                if (first[1] + r < rows) finish(out, tok, first[1] + r, acc[1][nt][e]);
+            }
+        }
+}
+
+// ------------------------------------------------------------------ float32 form
+constexpr int kFTile = 64, kFK = 16;
+__global__ void __launch_bounds__(256)
+dense_f32_kernel(const float *__restrict__ x, uint32_t x_stride, uint32_t k, const float *__restrict__ w,
+                 uint32_t rows, uint32_t w_stride, uint32_t n_tokens, OutputArgs out) {
+    qk::pdl_launch();
+    qk::pdl_wait();
+    __shared__ float xt[kFK][kFTile + 1], wt[kFK][kFTile + 1];
+    const uint32_t tx = threadIdx.x % 16, ty = threadIdx.x / 16;
+    const uint32_t t0 = blockIdx.y * kFTile, n0 = blockIdx.x * kFTile;
+    float acc[4][4] = {};
+    for (uint32_t k0 = 0; k0 < k; k0 += kFK) {
+        for (uint32_t i = threadIdx.x; i < kFTile * kFK; i += 256) {
+            const uint32_t kk = i % kFK, r = i / kFK;
+            const bool in_k = k0 + kk < k;
+            xt[kk][r] = in_k && t0 + r < n_tokens ? x[(size_t)(t0 + r) * x_stride + k0 + kk] : 0.f;
+            wt[kk][r] = in_k && n0 + r < rows ? w[(size_t)(n0 + r) * w_stride + k0 + kk] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int kk = 0; kk < kFK; ++kk) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) a[i] = xt[kk][ty + 16 * i], b[i] = wt[kk][tx + 16 * i];
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const uint32_t t = t0 + ty + 16 * i;
+        if (t >= n_tokens) continue;
+        if (out.kind == QK_OUTPUT_GLU) {  // one block of 32 gate rows and 32 up rows per tile
+#pragma unroll
+            for (int j = 0; j < 2; ++j) {
+                const uint32_t o = blockIdx.x * 32 + tx + 16 * j;
+                if (o < rows / 2) finish_pair(out, t, o, acc[i][j], acc[i][j + 2]);
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (n0 + tx + 16 * j < rows) finish(out, t, n0 + tx + 16 * j, acc[i][j]);
+        }
+    }
+}
+
+// ------------------------------------------------------------------ tcgen05 form
+// D[128 rows of x][BN weight rows]: x on the M side (an accumulator lane is a token, so that an
+// epilogue thread holds consecutive outputs of one token), W on the N side; both K-major tiles of
+// 64 k brought in by TMA with the 128-byte swizzle.  One persistent CTA per SM walks over the
+// tiles (token tiles fastest: neighbouring CTAs share the weight tile in L2).  Warp 0 issues the
+// copies, warp 1 the MMAs, warps 2..5 run the epilogue of one of two tensor-memory accumulators
+// while the next tile is multiplied into the other.  Every wait is bounded; a CTA that gives up
+// drains its copies and products in flight before it frees tensor memory.
+constexpr int kTcM = 128, kTcK = 64, kTcThreads = 192, kTcEpiWarps = 4;
+constexpr uint32_t kTcWaitDefault = 1u << 22;
+template <int BN> struct TcShape {
+    static constexpr uint32_t kABytes = kTcM * kTcK * 2, kBBytes = BN * kTcK * 2, kStage = kABytes + kBBytes;
+    static constexpr int kStages = BN == 256 ? 4 : BN == 128 ? 6 : 8;
+    static constexpr uint32_t kTmemCols = 2 * BN;
+    static constexpr size_t kSmem = 1024 + kStages * kStage + (2 * kStages + 5) * 8 + 32;
+};
+struct TcArgs {
+    uint32_t n_tokens, rows, k_chunks, m_tiles, tiles, wait_limit;
+    int *error;
+};
+__device__ __forceinline__ uint32_t tc_idesc(uint32_t bn) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((bn >> 3) << 17) | ((uint32_t)(kTcM >> 4) << 24);
+}
+__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap *map, uint32_t x, uint32_t y,
+                                            uint64_t *bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::
+            "r"(dst), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar))
+        : "memory");
+}
+__device__ __forceinline__ bool tc_epilogue_vote(bool ok) {
+    uint32_t all;
+    asm volatile(
+        "{\n .reg .pred p, q;\n setp.ne.b32 p, %1, 0;\n"
+        " barrier.cta.red.and.pred q, 1, %2, p;\n selp.u32 %0, 1, 0, q;\n}"
+        : "=r"(all)
+        : "r"((uint32_t)ok), "r"(kTcEpiWarps * 32)
+        : "memory");
+    return all != 0;
+}
+
+// Thirty-two consecutive outputs n0 .. of token t.  `vec`: rows are 16-byte aligned.
+__device__ __forceinline__ void tc_store32(const OutputArgs &o, uint32_t t, uint32_t n0, uint32_t limit,
+                                           float (&v)[32], bool vec) {
+    if (n0 >= limit) return;
+    if (!vec || n0 + 32 > limit) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (n0 + j < limit) {
+                if (o.kind == QK_OUTPUT_GLU) put(o.out, o.out_bf16, (size_t)t * o.out_stride + n0 + j, v[j]);
+                else finish(o, t, n0 + j, v[j]);
+            }
+        return;
+    }
+    if (o.kind == QK_OUTPUT_RESIDUAL) {
+        float *r = o.residual + (size_t)t * o.residual_stride + n0;
+#pragma unroll
+        for (int j = 0; j < 32; j += 4) {
+            const float4 old = *reinterpret_cast<const float4 *>(r + j);
+            float4 s = make_float4(1.f, 1.f, 1.f, 1.f);
+            if (o.scale) s = *reinterpret_cast<const float4 *>(o.scale + n0 + j);
+            v[j] = old.x + v[j] * s.x;
+            v[j + 1] = old.y + v[j + 1] * s.y;
+            v[j + 2] = old.z + v[j + 2] * s.z;
+            v[j + 3] = old.w + v[j + 3] * s.w;
+            *reinterpret_cast<float4 *>(r + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+        }
+        if (!o.out) return;
+    } else if (o.kind == QK_OUTPUT_SIDE) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] = activate(o.act, v[j]) * side_value(o, t, n0 + j);
+    }
+    if (o.out_bf16) {
+        uint16_t *p = static_cast<uint16_t *>(o.out) + (size_t)t * o.out_stride + n0;
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) {
+            uint32_t u[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+                u[e] = (uint32_t)float_to_bf16_bits(v[j + 2 * e]) |
+                       ((uint32_t)float_to_bf16_bits(v[j + 2 * e + 1]) << 16);
+            *reinterpret_cast<uint4 *>(p + j) = make_uint4(u[0], u[1], u[2], u[3]);
+        }
+    } else {
+        float *p = static_cast<float *>(o.out) + (size_t)t * o.out_stride + n0;
+#pragma unroll
+        for (int j = 0; j < 32; j += 4)
+            *reinterpret_cast<float4 *>(p + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+    }
+}
+
+template <int BN>
+__global__ void __launch_bounds__(kTcThreads, 1)
+dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, TcArgs g,
+                OutputArgs out, int vec) {
+    using S = TcShape<BN>;
+    qk::pdl_launch();
+    extern __shared__ __align__(1024) uint8_t tc_smem[];
+    uint8_t *tiles = reinterpret_cast<uint8_t *>(((uintptr_t)tc_smem + 1023) & ~(uintptr_t)1023);
+    uint64_t *full = reinterpret_cast<uint64_t *>(tiles + S::kStages * S::kStage);
+    uint64_t *empty = full + S::kStages;
+    uint64_t *acc_full = empty + S::kStages;
+    uint64_t *acc_empty = acc_full + 2;
+    uint64_t *drain = acc_empty + 2;
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(drain + 1);
+    volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+    volatile int *never = reinterpret_cast<volatile int *>(tmem_slot + 2);
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < S::kStages; ++s) {
+            mbar_init(&full[s], 1);
+            mbar_init(&empty[s], 1);
+        }
+        for (int a = 0; a < 2; ++a) {
+            mbar_init(&acc_full[a], 1);
+            mbar_init(&acc_empty[a], kTcEpiWarps);
+        }
+        mbar_init(drain, 1);
+        *abort_flag = 0;
+        *never = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&x_map) : "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&w_map) : "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)),
+                     "r"(S::kTmemCols)
+                     : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    qk::pdl_wait();
+    const uint32_t tmem_base = *tmem_slot;
+
+    if (warp == 0) {
+        uint32_t gc = 0;
+        bool dead = false;
+        for (uint32_t tile = blockIdx.x; tile < g.tiles && !dead; tile += gridDim.x) {
+            const uint32_t t0 = (tile % g.m_tiles) * kTcM, n0 = (tile / g.m_tiles) * BN;
+            for (uint32_t kc = 0; kc < g.k_chunks; ++kc, ++gc) {
+                const uint32_t s = gc % S::kStages;
+                if (!mbar_wait(&empty[s], ((gc / S::kStages) & 1) ^ 1, abort_flag, g.wait_limit)) {
+                    dead = true;
+                    break;
+                }
+                if (lane == 0) {
+                    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(&full[s])),
+                                 "r"(S::kStage)
+                                 : "memory");
+                    const uint32_t a = smem_u32(tiles + s * S::kStage);
+                    tma_load_2d(a, &x_map, kc * kTcK, t0, &full[s]);
+                    tma_load_2d(a + S::kABytes, &w_map, kc * kTcK, n0, &full[s]);
+                }
+                __syncwarp();
+            }
+        }
+        if (dead) {
+            *abort_flag = 1;
+            // the copies still in flight
+            for (uint32_t i = gc > (uint32_t)S::kStages ? gc - S::kStages : 0; i < gc; ++i)
+                (void)mbar_wait(&full[i % S::kStages], (i / S::kStages) & 1, never, g.wait_limit);
+        } else if (*abort_flag) {
+            for (uint32_t i = gc > (uint32_t)S::kStages ? gc - S::kStages : 0; i < gc; ++i)
+                (void)mbar_wait(&full[i % S::kStages], (i / S::kStages) & 1, never, g.wait_limit);
+        }
+    } else if (warp == 1) {
+        const uint32_t idesc = tc_idesc(BN);
+        uint32_t gc = 0, seg = 0;
+        bool dead = false;
+        for (uint32_t tile = blockIdx.x; tile < g.tiles && !dead; tile += gridDim.x, ++seg) {
+            const uint32_t acc = seg & 1;
+            if (!mbar_wait(&acc_empty[acc], ((seg >> 1) & 1) ^ 1, abort_flag, g.wait_limit)) {
+                dead = true;
+                break;
+            }
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t d_tmem = tmem_base + acc * BN;
+            for (uint32_t kc = 0; kc < g.k_chunks; ++kc, ++gc) {
+                const uint32_t s = gc % S::kStages;
+                if (!mbar_wait(&full[s], (gc / S::kStages) & 1, abort_flag, g.wait_limit)) {
+                    dead = true;
+                    break;
+                }
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                if (lane == 0) {
+                    const uint32_t a_addr = smem_u32(tiles + s * S::kStage), b_addr = a_addr + S::kABytes;
+#pragma unroll
+                    for (int k = 0; k < kTcK / 16; ++k) {
+                        const uint64_t ad = umma_desc(a_addr + k * 32), bd = umma_desc(b_addr + k * 32);
+                        const uint32_t accumulate = (kc != 0 || k != 0) ? 1u : 0u;
+                        asm volatile(
+                            "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
+                            " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}" ::"r"(d_tmem),
+                            "l"(ad), "l"(bd), "r"(idesc), "r"(accumulate)
+                            : "memory");
+                    }
+                    umma_commit(&empty[s]);
+                }
+                __syncwarp();
+            }
+            if (!dead && lane == 0) umma_commit(&acc_full[acc]);
+            __syncwarp();
+        }
+        if (dead) {
+            *abort_flag = 1;
+            if (lane == 0) umma_commit(drain);  // the products still in flight
+            __syncwarp();
+            (void)mbar_wait(drain, 0, never, g.wait_limit);
+        }
+    } else {
+        const uint32_t quarter = warp % 4;
+        uint32_t seg = 0;
+        for (uint32_t tile = blockIdx.x; tile < g.tiles; tile += gridDim.x, ++seg) {
+            const uint32_t acc = seg & 1;
+            const uint32_t t = (tile % g.m_tiles) * kTcM + quarter * 32 + lane, n0 = (tile / g.m_tiles) * BN;
+            if (!tc_epilogue_vote(mbar_wait(&acc_full[acc], (seg >> 1) & 1, abort_flag, g.wait_limit))) {
+                *abort_flag = 1;
+                break;
+            }
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const uint32_t lane_addr = tmem_base + acc * BN + ((quarter * 32) << 16);
+            if (out.kind == QK_OUTPUT_GLU) {
+                for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += 64) {  // warp-uniform
+                    uint32_t a[32], b[32];
+                    tmem_ld32(lane_addr + c, a);
+                    tmem_ld32(lane_addr + c + 32, b);
+                    tmem_ld_wait();
+                    float v[32];
+#pragma unroll
+                    for (int j = 0; j < 32; ++j)
+                        v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
+                    if (t < g.n_tokens) tc_store32(out, t, (n0 + c) / 2, g.rows / 2, v, vec != 0);
+                }
+            } else {
+                for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += 32) {
+                    uint32_t a[32];
+                    tmem_ld32(lane_addr + c, a);
+                    tmem_ld_wait();
+                    float v[32];
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(a[j]);
+                    if (t < g.n_tokens) tc_store32(out, t, n0 + c, g.rows, v, vec != 0);
+                }
+            }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&acc_empty[acc]);
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1)
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(S::kTmemCols)
+                     : "memory");
+    if (threadIdx.x == 0 && *abort_flag) atomicOr(g.error, 1);
+}
+
+typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
+                                  const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
+                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+
+// rows x k bfloat16 entries, `stride` entries from row to row; boxes of 64 k x box_rows.
+qk_status encode_map(const void *base, size_t rows, size_t k, size_t stride, uint32_t box_rows, CUtensorMap *out) {
+    static EncodeTiledFn fn = nullptr;
+    if (!fn) {
+        void *sym = nullptr;
+        cudaDriverEntryPointQueryResult qres;
+        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres);
+        if (e != cudaSuccess || qres != cudaDriverEntryPointSuccess || !sym)
+            return qk::fail(QK_ERR_CUDA, "cuTensorMapEncodeTiled is not available: %s", cudaGetErrorString(e));
+        fn = (EncodeTiledFn)sym;
+    }
+    const cuuint64_t dims[2] = {k, rows};
+    const cuuint64_t strides[1] = {stride * 2};
+    const cuuint32_t box[2] = {(cuuint32_t)kTcK, box_rows};
+    const cuuint32_t estr[2] = {1, 1};
+    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return qk::fail(QK_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d", (int)r);
+    return QK_OK;
+}
+
+// Weight rows per tile: the width whose number of waves over the SMs costs least.
+int pick_tile(size_t m_tiles, size_t rows, size_t sms) {
+    int best = 64;
+    size_t best_cost = ~(size_t)0;
+    for (int bn : {256, 128, 64}) {
+        const size_t waves = qk::ceil_div(m_tiles * qk::ceil_div(rows, bn), sms);
+        const size_t cost = waves * (bn + 48);  // (48: what a tile costs whatever its width)
+        if (cost < best_cost) best = bn, best_cost = cost;
+    }
+    return best;
+}
+
+template <int BN>
+qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out,
+                    int vec) {
+    using S = TcShape<BN>;
+    CUtensorMap xm, wm;
+    qk_status st;
+    if ((st = encode_map(x, d.tokens, d.k, x_stride, kTcM, &xm)) != QK_OK) return st;
+    if ((st = encode_map(d.w, d.rows, d.k, d.w_stride, BN, &wm)) != QK_OK) return st;
+    TcArgs g{};
+    g.n_tokens = (uint32_t)d.tokens;
+    g.rows = (uint32_t)d.rows;
+    g.k_chunks = (uint32_t)qk::ceil_div(d.k, kTcK);
+    g.m_tiles = (uint32_t)qk::ceil_div(d.tokens, kTcM);
+    g.tiles = g.m_tiles * (uint32_t)qk::ceil_div(d.rows, BN);
+    g.wait_limit = c->wait_limit ? c->wait_limit : kTcWaitDefault;
+    g.error = (int *)c->d_err.ptr;
+    QK_CUDA(cudaFuncSetAttribute(dense_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
+    (void)qk::launch_pdl(c->pdl, dense_tc_kernel<BN>, dim3(std::min(g.tiles, (uint32_t)c->sm_count)),
+                         dim3(kTcThreads), S::kSmem, c->stream, xm, wm, g, out, vec);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    c->err_armed = true;
+    return QK_OK;
+}
+
+template <int NT>
+qk_status launch_skinny(qk_ctx *c, const uint16_t *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out) {
+    const bool pair = d.output == QK_OUTPUT_GLU;
+    const size_t tiles = pair ? qk::ceil_div(d.rows / 2, 16) : qk::ceil_div(d.rows, 32);
+    const size_t chunks = qk::ceil_div(d.k, 64);
+    uint32_t ks = 1;  // warps that share out a row tile's k range: enough blocks to fill the SMs
+    while (ks < kSkWarps && qk::ceil_div(tiles * ks, kSkWarps) < (size_t)c->sm_count && ks * 2 <= chunks) ks *= 2;
+    const size_t stage = 2 * (size_t)ks * 8 * NT * kSkPitch * 2;
+    const size_t sums = (size_t)kSkWarps * 2 * NT * 4 * 32 * 4;
+    const size_t smem = std::max(stage, ks > 1 ? sums : (size_t)0);
+    QK_CUDA(cudaFuncSetAttribute(dense_skinny_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    (void)qk::launch_pdl(c->pdl, dense_skinny_kernel<NT>, dim3((unsigned)qk::ceil_div(tiles * ks, kSkWarps)),
+                         dim3(kSkWarps * 32), smem, c->stream, x, (uint32_t)x_stride, (uint32_t)d.k,
+                         (const uint16_t *)d.w, (uint32_t)d.rows, (uint32_t)d.w_stride, (uint32_t)d.tokens, ks, out);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    return QK_OK;
+}
+
+template <typename W, int NT, int R>
+qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
+                          size_t n_tokens, uint32_t ks) {
+    const size_t step = VecTraits<W>::kStep;
+    const size_t smem = NT * qk::ceil_div(d.k, step) * step * 4;
+    const size_t groups = d.output == QK_OUTPUT_GLU ? qk::ceil_div(d.rows / 2, R / 2 ? R / 2 : 1)
+                                                    : qk::ceil_div(d.rows, R);
+    QK_CUDA(cudaFuncSetAttribute(dense_vector_kernel<W, NT, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 (int)std::max(smem, (size_t)48 * 1024)));
+    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>, dim3((unsigned)qk::ceil_div(groups * ks, kVecWarps)),
+                         dim3(kVecThreads), smem, c->stream, in, out, (const W *)d.w, (uint32_t)d.rows,
+                         (uint32_t)d.w_stride, (uint32_t)n_tokens, ks);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    return QK_OK;
+}
+template <typename W, int NT>
+qk_status launch_vector(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
+                        size_t n_tokens) {
+    // rows per warp and warps per row group: about two blocks per SM or more
+    const size_t want = 2 * (size_t)c->sm_count * kVecWarps, steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
+    const bool pair = d.output == QK_OUTPUT_GLU;
+    if (d.rows / 4 >= want) return launch_vector_r<W, NT, 4>(c, in, out, d, n_tokens, 1);
+    if (d.rows / 2 >= want || pair) {
+        uint32_t ks = 1;
+        while (ks < kVecWarps && d.rows / 2 * ks < want && ks * 4 <= steps) ks *= 2;
+        return launch_vector_r<W, NT, 2>(c, in, out, d, n_tokens, ks);
+    }
+    uint32_t ks = 1;
+    while (ks < kVecWarps && d.rows * ks < want && ks * 4 <= steps) ks *= 2;
+    return launch_vector_r<W, NT, 1>(c, in, out, d, n_tokens, ks);
+}
+
+InputArgs input_args(const qk_dense_call &d) {
+    InputArgs a{};
+    a.x = (const float *)d.x;
+    a.pending = d.pending;
+    a.pending_weight = d.pending_weight;
+    a.second = d.second;
+    a.norm_weight = d.norm_weight;
+    a.gate = d.gate;
+    a.x_out = d.x_out;
+    a.positions = d.positions;
+    a.slots = d.slots;
+    a.x_stride = (uint32_t)d.x_stride;
+    a.pending_stride = (uint32_t)d.pending_stride;
+    a.gate_stride = (uint32_t)d.gate_stride;
+    a.width = (uint32_t)d.width;
+    a.k = (uint32_t)d.k;
+    a.group = (uint32_t)d.group;
+    a.pending_eps = d.pending_eps;
+    a.norm_eps = d.norm_eps;
+    a.kind = d.input;
+    a.norm = d.norm;
+    a.append = AppendArgs{d.append.src, d.append.weight, d.append.cache, (uint32_t)d.append.src_stride,
+                          (uint32_t)d.append.width, (uint32_t)d.append.ring, (uint32_t)d.append.stride, d.append.eps,
+                          d.append.cache_dtype == QK_BF16};
+    return a;
+}
+OutputArgs output_args(const qk_dense_call &d) {
+    OutputArgs o{};
+    o.out = d.out;
+    o.residual = d.residual;
+    o.scale = d.out_scale;
+    o.side = d.side;
+    o.ids = d.ids;
+    o.out_stride = (uint32_t)d.out_stride;
+    o.residual_stride = (uint32_t)d.residual_stride;
+    o.side_stride = (uint32_t)d.side_stride;
+    o.side_offset = (uint32_t)d.side_offset;
+    o.vocab = (uint32_t)d.vocab;
+    o.kind = d.output;
+    o.act = d.activation;
+    o.out_bf16 = d.out_dtype == QK_BF16;
+    o.side_bf16 = d.side_dtype == QK_BF16;
+    return o;
+}
+void advance(InputArgs &a, OutputArgs &o, size_t t) {  // the same call from row t on
+    a.x += t * a.x_stride;
+    if (a.pending) a.pending += t * a.pending_stride;
+    if (a.second) a.second += t * a.x_stride;
+    if (a.gate) a.gate += t * a.gate_stride;
+    if (a.x_out) a.x_out += t * a.x_stride;
+    if (a.positions) a.positions += t;
+    if (a.slots) a.slots += t;
+    if (a.append.src) a.append.src += t * a.append.src_stride;
+    if (o.out) o.out = (uint8_t *)o.out + t * o.out_stride * (o.out_bf16 ? 2 : 4);
+    if (o.residual) o.residual += t * o.residual_stride;
+    if (o.ids) o.ids += t;
+}
+
+qk_status validate(const qk_dense_call *d, bool with_weights) {
+    if (!d || !d->x) return qk::fail(QK_ERR_VALUE, "qk_dense: null argument");
+    if (d->k == 0 || d->k % 8 || d->width > d->k || d->width == 0)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: %zu input columns for vectors of %zu (a multiple of 8 is needed)",
+                        d->k, d->width);
+    if (d->input < QK_INPUT_PLAIN || d->input > QK_INPUT_GATED)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: unknown input kind %d", d->input);
+    if (d->x_dtype == QK_BF16 && d->input != QK_INPUT_PLAIN)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: bfloat16 input rows must be plain");
+    if (d->x_dtype != QK_BF16 && d->x_dtype != QK_F32)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: input dtype must be float32 or bfloat16, got tag %d", d->x_dtype);
+    if (d->input == QK_INPUT_CONCAT && (!d->second || d->k % 2 || d->width > d->k / 2))
+        return qk::fail(QK_ERR_VALUE, "qk_dense: a concatenated input needs a second vector and two equal halves");
+    if (d->input == QK_INPUT_GATED &&
+        (!d->gate || !d->norm_weight || d->group == 0 || d->width % d->group))
+        return qk::fail(QK_ERR_VALUE, "qk_dense: a gated input needs a gate and whole groups");
+    if (d->norm != QK_NORM_NONE && !d->norm_weight && d->input != QK_INPUT_PLAIN)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: a norm needs its weight");
+    if (d->x_out && d->x_out == d->x) return qk::fail(QK_ERR_VALUE, "qk_dense: x_out must be another buffer than x");
+    if (d->pending && !d->pending_weight) return qk::fail(QK_ERR_VALUE, "qk_dense: a pending residual needs its weight");
+    if (d->append.src && (!d->append.cache || !d->positions || !d->slots || d->append.ring == 0 ||
+                          d->append.width > d->append.stride))
+        return qk::fail(QK_ERR_VALUE, "qk_dense: an append needs a cache, positions and slots");
+    if (d->input != QK_INPUT_PLAIN && d->k * 4 > kVecSmemMax)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: an input vector of %zu entries does not fit shared memory", d->k);
+    if (!with_weights) return QK_OK;
+    if (!d->w || d->rows == 0 || d->w_stride < d->k || d->w_stride % 8)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: %zu weight rows of stride %zu for %zu columns", d->rows, d->w_stride,
+                        d->k);
+    if (d->w_dtype != QK_F32 && d->w_dtype != QK_BF16)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: weight dtype must be float32 or bfloat16, got tag %d", d->w_dtype);
+    if (d->output < QK_OUTPUT_STORE || d->output > QK_OUTPUT_SIDE)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: unknown output kind %d", d->output);
+    if (d->output == QK_OUTPUT_RESIDUAL ? !d->residual : !d->out)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: no output buffer");
+    if (d->output == QK_OUTPUT_GLU && d->rows % 64)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: gated pairs come in blocks of 64 rows, got %zu", d->rows);
+    if (d->output == QK_OUTPUT_SIDE && (!d->side || !d->ids || d->vocab == 0))
+        return qk::fail(QK_ERR_VALUE, "qk_dense: a side product needs its table and token ids");
+    return QK_OK;
+}
+
+template <typename A>
+qk_status launch_input(qk_ctx *c, const InputArgs &in, size_t tokens, A *dst) {
+    const size_t smem = dst ? (size_t)in.k * 4 : 0;
+    if (smem > kVecSmemMax) return qk::fail(QK_ERR_VALUE, "qk_dense: an input vector of %u entries does not fit shared memory", in.k);
+    QK_CUDA(cudaFuncSetAttribute(dense_input_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 (int)std::max(smem, (size_t)48 * 1024)));
+    (void)qk::launch_pdl(c->pdl, dense_input_kernel<A>, dim3((unsigned)tokens), dim3(256), smem, c->stream, in, dst);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    return QK_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+int32_t qk_dense_form(size_t tokens, size_t k, int32_t w_dtype) {
+    if (tokens <= (size_t)kVectorTokens && k * 4 <= kVecSmemMax) return QK_FORM_VECTOR;
+    if (w_dtype == QK_F32) return QK_FORM_F32;
+    return tokens <= (size_t)kSkinnyTokens ? QK_FORM_SKINNY : QK_FORM_TCGEN05;
+}
+
+qk_status qk_dense_input(qk_ctx *ctx, const qk_dense_call *d) {
+    qk_ctx *c;
+    qk_status st = qk::resolve_ctx(ctx, &c);
+    if (st != QK_OK) return st;
+    QK_CUDA(cudaSetDevice(c->device));
+    if ((st = validate(d, false)) != QK_OK) return st;
+    if (d->tokens == 0) return QK_OK;
+    if (d->x_dtype != QK_F32) return qk::fail(QK_ERR_VALUE, "qk_dense_input: the rows must be float32");
+    const InputArgs in = input_args(*d);
+    return d->out_dtype == QK_BF16 ? launch_input<uint16_t>(c, in, d->tokens, (uint16_t *)d->out)
+                                   : launch_input<float>(c, in, d->tokens, (float *)d->out);
+}
+
+qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
+    qk_ctx *c;
+    qk_status st = qk::resolve_ctx(ctx, &c);
+    if (st != QK_OK) return st;
+    QK_CUDA(cudaSetDevice(c->device));
+    if ((st = validate(d, true)) != QK_OK) return st;
+    if (d->tokens == 0) return QK_OK;
+    const bool bf16 = d->w_dtype == QK_BF16;
+    const int32_t form = qk_dense_form(d->tokens, d->k, d->w_dtype);
+    InputArgs in = input_args(*d);
+    OutputArgs out = output_args(*d);
+    if (form == QK_FORM_VECTOR && d->x_dtype == QK_F32) {
+        // as many rows per launch as fit shared memory
+        for (size_t t = 0; t < d->tokens;) {
+            const size_t left = d->tokens - t;
+            const int nt = left >= 3 && d->k * 16 <= kVecSmemMax ? 4 : left >= 2 && d->k * 8 <= kVecSmemMax ? 2 : 1;
+            const size_t n = std::min(left, (size_t)nt);
+            if (bf16)
+                st = nt == 4 ? launch_vector<uint16_t, 4>(c, in, out, *d, n)
+                     : nt == 2 ? launch_vector<uint16_t, 2>(c, in, out, *d, n)
+                               : launch_vector<uint16_t, 1>(c, in, out, *d, n);
+            else
+                st = nt == 4 ? launch_vector<float, 4>(c, in, out, *d, n)
+                     : nt == 2 ? launch_vector<float, 2>(c, in, out, *d, n)
+                               : launch_vector<float, 1>(c, in, out, *d, n);
+            if (st != QK_OK) return st;
+            advance(in, out, n);
+            t += n;
+        }
+        return QK_OK;
+    }
+    // the input rows in the weights' dtype
+    const void *rows = d->x;
+    size_t stride = d->x_stride;
+    const bool direct = d->input == QK_INPUT_PLAIN && d->x_dtype == d->w_dtype && d->x_stride >= d->k &&
+                        d->x_stride % 8 == 0 && ((uintptr_t)d->x & 15) == 0;
+    if (d->x_dtype == QK_BF16 && !direct)
+        return qk::fail(QK_ERR_VALUE, "qk_dense: bfloat16 rows of stride %zu cannot feed %zu columns", d->x_stride, d->k);
+    if (!direct) {
+        const size_t need = d->tokens * d->k * (bf16 ? 2 : 4);
+        if (!d->scratch || d->scratch_bytes < need)
+            return qk::fail(QK_ERR_VALUE, "qk_dense: %zu bytes of scratch are needed, %zu given", need,
+                            d->scratch_bytes);
+        st = bf16 ? launch_input<uint16_t>(c, in, d->tokens, (uint16_t *)d->scratch)
+                  : launch_input<float>(c, in, d->tokens, (float *)d->scratch);
+        if (st != QK_OK) return st;
+        rows = d->scratch;
+        stride = d->k;
+    } else if (d->append.src) {
+        if ((st = launch_input<float>(c, in, d->tokens, nullptr)) != QK_OK) return st;
+    }
+    if (!bf16) {
+        dim3 grid((unsigned)qk::ceil_div(d->rows, kFTile), (unsigned)qk::ceil_div(d->tokens, kFTile));
+        (void)qk::launch_pdl(c->pdl, dense_f32_kernel, grid, dim3(256), 0, c->stream, (const float *)rows,
+                             (uint32_t)stride, (uint32_t)d->k, (const float *)d->w, (uint32_t)d->rows,
+                             (uint32_t)d->w_stride, (uint32_t)d->tokens, out);
+        QK_CUDA(cudaGetLastError());
+        c->launches++;
+        return QK_OK;
+    }
+    if (d->tokens <= (size_t)kSkinnyTokens) {
+        const uint16_t *x = (const uint16_t *)rows;
+        if (d->tokens <= 8) return launch_skinny<1>(c, x, stride, *d, out);
+        if (d->tokens <= 16) return launch_skinny<2>(c, x, stride, *d, out);
+        if (d->tokens <= 32) return launch_skinny<4>(c, x, stride, *d, out);
+        return launch_skinny<8>(c, x, stride, *d, out);
+    }
+    if ((st = qk::error_word(c)) != QK_OK) return st;
+    const int per16 = d->out_dtype == QK_BF16 ? 8 : 4;
+    const int vec = (!d->out || (((uintptr_t)d->out & 15) == 0 && d->out_stride % per16 == 0)) &&
+                    (!d->residual || (((uintptr_t)d->residual & 15) == 0 && d->residual_stride % 4 == 0)) &&
+                    ((uintptr_t)d->out_scale & 15) == 0;
+    switch (pick_tile(qk::ceil_div(d->tokens, kTcM), d->rows, (size_t)c->sm_count)) {
+        case 256: return launch_tc<256>(c, rows, stride, *d, out, vec);
+        case 128: return launch_tc<128>(c, rows, stride, *d, out, vec);
+        default: return launch_tc<64>(c, rows, stride, *d, out, vec);
+    }
+}
+
+}  // extern "C"
