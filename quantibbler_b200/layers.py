@@ -1,0 +1,405 @@
+"""Building blocks of layered decoders: dense linears with their fused inputs and outputs, and the
+mixers (windowed latent attention, gated delta rule), each with the cache or state it keeps per
+sequence slot.
+
+A mixer takes the residual stream of a ``Rows`` workspace and adds its result to it; everything
+it does is a C-ABI call that only launches kernels, so a step can be captured in a CUDA graph.
+Sizes and constants are parameters: nothing here belongs to one design.
+"""
+
+from __future__ import annotations
+
+import ctypes
+from ctypes import c_float, c_int32, c_size_t, c_void_p
+from dataclasses import dataclass
+
+from . import _lib
+from ._lib import QK_BF16, QK_F32, check
+
+IN_PLAIN, IN_NORM, IN_CONCAT, IN_GATED = range(4)
+NORM_NONE, NORM_LAYER, NORM_RMS = range(3)
+ACTIVATIONS = {"relu": 0, "silu": 1, "gelu_tanh": 2}
+OUT_STORE, OUT_RESIDUAL, OUT_GLU, OUT_SIDE = range(4)
+FORM_VECTOR = 0
+
+
+def _struct(name, fields):
+    return type(name, (ctypes.Structure,), {"_fields_": fields})
+
+
+_P, _Z, _I, _F = c_void_p, c_size_t, c_int32, c_float
+LatentAppend = _struct("LatentAppend", [
+    ("src", _P), ("src_stride", _Z), ("width", _Z), ("weight", _P), ("eps", _F), ("cache_dtype", _I),
+    ("cache", _P), ("ring", _Z), ("stride", _Z)])
+DenseCall = _struct("DenseCall", [
+    ("tokens", _Z), ("positions", _P), ("slots", _P), ("ids", _P), ("vocab", _Z),
+    ("input", _I), ("x_dtype", _I), ("x", _P), ("x_stride", _Z), ("width", _Z), ("k", _Z),
+    ("pending", _P), ("pending_stride", _Z), ("pending_weight", _P), ("pending_eps", _F), ("x_out", _P),
+    ("second", _P), ("norm", _I), ("norm_eps", _F), ("norm_weight", _P), ("gate", _P), ("gate_stride", _Z),
+    ("group", _Z), ("append", LatentAppend),
+    ("w_dtype", _I), ("w", _P), ("rows", _Z), ("w_stride", _Z),
+    ("output", _I), ("activation", _I), ("out_dtype", _I), ("out", _P), ("out_stride", _Z),
+    ("residual", _P), ("residual_stride", _Z), ("out_scale", _P), ("side", _P), ("side_dtype", _I),
+    ("side_stride", _Z), ("side_offset", _Z), ("scratch", _P), ("scratch_bytes", _Z)])
+DeltaCall = _struct("DeltaCall", [
+    ("tokens", _Z), ("segments", _Z), ("positions", _P), ("slots", _P), ("seg_first", _P), ("seg_len", _P),
+    ("seg_row", _P), ("heads", _Z), ("kv_heads", _Z), ("dim", _Z), ("vdim", _Z), ("taps", _Z), ("proj", _P),
+    ("proj_stride", _Z), ("beta_offset", _Z), ("decay_offset", _Z), ("conv_q", _P), ("conv_k", _P), ("conv_v", _P),
+    ("a_log", _P), ("dt_bias", _P), ("unit_eps", _F), ("conv_state", _P), ("state", _P), ("qkv", _P), ("gates", _P),
+    ("out", _P), ("out_stride", _Z)])
+LatentCall = _struct("LatentCall", [
+    ("tokens", _Z), ("positions", _P), ("slots", _P), ("heads", _Z), ("dim", _Z), ("dim_stride", _Z), ("vdim", _Z),
+    ("vdim_stride", _Z), ("kv_rank", _Z), ("kv_stride", _Z), ("window", _Z), ("ring", _Z), ("n_slots", _Z),
+    ("scale", _F), ("q", _P), ("q_dtype", _I), ("q_stride", _Z), ("w_dtype", _I), ("uk", _P), ("uv", _P),
+    ("cache", _P), ("n_splits", _Z), ("scratch", _P), ("out", _P), ("out_dtype", _I), ("out_stride", _Z)])
+
+
+def up_to(n: int, multiple: int) -> int:
+    return -(-int(n) // multiple) * multiple
+
+
+def padded(n: int) -> int:
+    """Row strides: a whole number of 64-entry pieces, the matrix kernels' k step."""
+    return up_to(n, 64)
+
+
+@dataclass
+class Linear:
+    """Weight rows on the device, columns padded with zeros to ``k``."""
+    w: object
+    rows: int
+    width: int
+    k: int
+
+
+class Weights:
+    """Packs a model's tensors for the kernels: ``dtype`` is the dtype of the linears."""
+
+    def __init__(self, torch, device, serving: str):
+        self.torch, self.device = torch, device
+        self.dtype = torch.float32 if serving == "float32" else torch.bfloat16
+        self.tag = QK_F32 if serving == "float32" else QK_BF16
+
+    def to(self, t, dtype=None):
+        return t.to(self.device, dtype or self.dtype).contiguous()
+
+    def vector(self, t):
+        return self.to(t, self.torch.float32)
+
+    def matrix(self, *mats) -> Linear:
+        """The matrices' rows one after the other (they share their input)."""
+        width = mats[0].shape[1]
+        k = padded(width)
+        rows = sum(m.shape[0] for m in mats)
+        w = self.torch.zeros(rows, k, dtype=self.dtype, device=self.device)
+        w[:, :width] = self.torch.cat([self.to(m) for m in mats])
+        return Linear(w, rows, width, k)
+
+    def heads(self, mat, heads: int, size: int, stride: int):
+        """Head-major rows with every head's rows padded to ``stride``."""
+        m = self.to(mat).reshape(heads, size, mat.shape[1])
+        out = self.torch.zeros(heads, stride, mat.shape[1], dtype=self.dtype, device=self.device)
+        out[:, :size] = m
+        return out.reshape(heads * stride, mat.shape[1])
+
+    def halves(self, mat, width: int) -> Linear:
+        """A matrix over [x ; y], each half's columns padded on their own."""
+        half = padded(width)
+        m = self.to(mat)
+        w = self.torch.zeros(m.shape[0], 2 * half, dtype=self.dtype, device=self.device)
+        w[:, :width] = m[:, :width]
+        w[:, half:half + width] = m[:, width:]
+        return Linear(w, m.shape[0], width, 2 * half)
+
+    def gated_pair(self, gate, up) -> Linear:
+        """Blocks of 32 gate rows and their 32 up rows, so that a kernel that has one has both."""
+        ff, width = gate.shape
+        k, blocks = padded(width), up_to(ff, 32) // 32
+        w = self.torch.zeros(blocks, 2, 32, k, dtype=self.dtype, device=self.device)
+        for which, m in enumerate((gate, up)):
+            full = self.torch.zeros(blocks * 32, width, dtype=self.dtype, device=self.device)
+            full[:ff] = self.to(m)
+            w[:, which, :, :width] = full.reshape(blocks, 32, width)
+        return Linear(w, blocks * 64, width, k)
+
+
+class Rows:
+    """Activation buffers and row descriptions for up to ``cap`` rows at a time.
+
+    The residual stream alternates between ``x`` and ``x2``; ``pending`` is a result that the next
+    norm still has to add to it.  ``act`` holds the dtype of what only matrix products read:
+    float32 where the vector form takes the rows, else the linears' dtype."""
+
+    def __init__(self, torch, device, cap: int, stride: int, weights: Weights, vector: bool):
+        self.torch, self.device, self.cap, self.stride = torch, device, cap, stride
+        i32 = dict(dtype=torch.int32, device=device)
+        self.ids, self.slots = torch.zeros(cap, **i32), torch.arange(cap, **i32)
+        self.positions = torch.zeros(cap, **i32)
+        self.seg_first, self.seg_len = torch.arange(cap, **i32), torch.ones(cap, **i32)
+        self.seg_row = torch.zeros(cap, **i32)
+        self.n = self.segments = cap
+        self.portion = None            # (slot, first position) when the rows are one portion
+        self.act = torch.float32 if vector else weights.dtype
+        self.act_tag = QK_F32 if self.act == torch.float32 else QK_BF16
+        self.weights = weights
+        self._buffers, self.split_floats = {}, {}
+        self.x, self.x2 = self.f32("x", stride), self.f32("x2", stride)
+        self.pending = None            # (buffer, weight, eps)
+
+    def f32(self, name: str, width: int):
+        return self.buffer(name, width, self.torch.float32)
+
+    def buffer(self, name: str, width: int, dtype=None, rows: int | None = None):
+        """A zeroed buffer of ``cap`` rows, shared by every layer that asks for the same one."""
+        dtype = dtype or self.act
+        key = (name, int(width), dtype, rows)
+        if key not in self._buffers:
+            self._buffers[key] = self.torch.zeros(rows or self.cap, int(width), dtype=dtype, device=self.device)
+        return self._buffers[key]
+
+    def call(self, lin: Linear, **fields) -> DenseCall:
+        d = DenseCall(tokens=self.n, positions=self.positions.data_ptr(), slots=self.slots.data_ptr(),
+                      ids=self.ids.data_ptr(), x_dtype=QK_F32, width=lin.width, k=lin.k,
+                      w_dtype=self.weights.tag, w=lin.w.data_ptr(), rows=lin.rows, w_stride=lin.k,
+                      out_dtype=QK_F32)
+        for name, value in fields.items():
+            if hasattr(value, "data_ptr"):
+                value = value.data_ptr()
+            setattr(d, name, value)
+        return d
+
+    def dense(self, ctx, lin: Linear, **fields) -> None:
+        d = self.call(lin, **fields)
+        plain = d.input == IN_PLAIN and d.x_dtype == self.weights.tag
+        if not plain and _lib.lib().qk_dense_form(self.n, lin.k, self.weights.tag) != FORM_VECTOR:
+            scratch = self.buffer("input", lin.k, self.weights.dtype)
+            d.scratch, d.scratch_bytes = scratch.data_ptr(), scratch.numel() * scratch.element_size()
+        check(_lib.lib().qk_dense(ctx.handle, ctypes.byref(d)))
+
+    def stream_fields(self, norm: int, norm_weight, eps: float) -> dict:
+        """Input fields of a linear behind a norm of the residual stream; takes ``pending`` in."""
+        f = dict(input=IN_NORM, x=self.x, x_stride=self.stride, norm=norm, norm_weight=norm_weight, norm_eps=eps)
+        if self.pending is not None:
+            y, weight, peps = self.pending
+            f.update(pending=y, pending_stride=y.shape[1], pending_weight=weight, pending_eps=peps, x_out=self.x2)
+        return f
+
+    def settle(self) -> None:
+        """After a linear with ``stream_fields``: the stream is where it has been written."""
+        if self.pending is not None:
+            self.x, self.x2 = self.x2, self.x
+            self.pending = None
+
+    def residual_fields(self, scale) -> dict:
+        """Output fields of a linear that adds to the stream; bfloat16 rows also keep a copy for
+        the plain linear that may follow."""
+        f = dict(output=OUT_RESIDUAL, residual=self.x, residual_stride=self.stride, out_scale=scale)
+        if self.act != self.torch.float32:
+            f.update(out=self.buffer("stream", self.stride), out_stride=self.stride, out_dtype=self.act_tag)
+        return f
+
+    def stream_rows(self):
+        """The stream as a plain input (after ``residual_fields``): (buffer, dtype tag)."""
+        if self.act != self.torch.float32:
+            return self.buffer("stream", self.stride), self.act_tag
+        return self.x, QK_F32
+
+
+class RingCache:
+    """The last ``rows`` latents of every slot: position p of a slot lies in row p mod rows."""
+
+    def __init__(self, torch, device, slots: int, rows: int, stride: int, dtype):
+        self.rows, self.stride = int(rows), int(stride)
+        self.data = torch.zeros(slots, self.rows, self.stride, dtype=dtype, device=device)
+
+
+class RecurrentState:
+    """Per slot: the heads' float32 state matrices and the convolution's last inputs.  A portion
+    that starts at position 0 starts from zero, so a slot needs no clearing between sequences."""
+
+    def __init__(self, torch, device, slots: int, heads: int, dim: int, vdim: int, taps: int, channels: int):
+        f32 = dict(dtype=torch.float32, device=device)
+        self.matrix = torch.zeros(slots, heads, vdim, dim, **f32)
+        self.conv = torch.zeros(slots, taps, channels, **f32)
+
+
+class LatentAttention:
+    """Latent attention without positions under a sliding window (None: no window).
+
+    Portions of more than ``absorbed_rows`` rows (bfloat16, head sizes up to 256) expand the
+    window's latents into keys and values by a matrix product; everything else works on the
+    latents themselves."""
+
+    absorbed_rows = 16
+
+    def __init__(self, weights: Weights, tensors: dict, *, heads: int, dim: int, vdim: int, kv_rank: int,
+                 q_rank: int, scale: float, window: int | None, eps: float):
+        self.heads, self.dim, self.vdim, self.kv_rank, self.q_rank = heads, dim, vdim, kv_rank, q_rank
+        self.scale, self.window, self.eps, self.weights = float(scale), window, float(eps), weights
+        self.dim_stride, self.vdim_stride, self.kv_stride = up_to(dim, 16), up_to(vdim, 16), padded(kv_rank)
+        t, w = tensors, weights
+        self.down = w.matrix(t["dq"], t["dkv"])
+        self.q_norm, self.kv_norm = w.vector(t["dq.norm"]), w.vector(t["dkv.norm"])
+        self.uq = w.matrix(w.heads(t["uq"], heads, dim, self.dim_stride))
+        self.ukv = w.matrix(w.heads(t["uk"], heads, dim, self.dim_stride),
+                            w.heads(t["uv"], heads, vdim, self.vdim_stride))
+        self.out = w.matrix(t["o"])
+        self.expands = w.tag == QK_BF16 and max(self.dim_stride, self.vdim_stride) <= 256
+
+    def make_state(self, torch, device, slots: int, max_seq: int, portion: int) -> RingCache:
+        # a portion is appended before its first row is read, so the ring holds a window beside it
+        window = min(self.window or max_seq, max_seq)
+        return RingCache(torch, device, slots, min(window - 1 + portion, max(max_seq, window)), self.kv_stride,
+                         self.weights.dtype)
+
+    def n_splits(self, rows: int, window: int) -> int:
+        """Key splits of the absorbed form: about two blocks per SM, 32 keys or more each."""
+        groups = -(-self.heads // 16) if self.weights.tag == QK_BF16 else self.heads
+        return max(1, min(64, 296 // max(1, rows * groups), -(-window // 32)))
+
+    def _split_floats(self, rows: Rows, window: int) -> int:
+        """Scratch of the absorbed form for any number of rows it may get in this workspace."""
+        key = (self.heads, self.kv_stride, window)
+        if key not in rows.split_floats:
+            most = min(rows.cap, self.absorbed_rows) if self.expands and rows.portion is not None else rows.cap
+            rows.split_floats[key] = max(_lib.lib().qk_latent_scratch(
+                m, self.heads, self.kv_stride, self.n_splits(m, window)) for m in range(1, most + 1)) // 4
+        return rows.split_floats[key]
+
+    def forward(self, ctx, rows: Rows, norm: int, norm_weight, norm_eps: float, scale, state: RingCache,
+                max_seq: int) -> None:
+        lib, n = _lib.lib(), rows.n
+        window = min(self.window or max_seq, max_seq, state.rows)
+        lat_stride = up_to(self.q_rank + self.kv_rank, 4)
+        lat = rows.f32("latents", lat_stride)
+        rows.dense(ctx, self.down, **rows.stream_fields(norm, norm_weight, norm_eps), out=lat, out_stride=lat_stride)
+        rows.settle()
+        expanded = self.expands and rows.portion is not None and n > self.absorbed_rows
+        q_stride = padded(self.heads * self.dim_stride)
+        q = rows.buffer("query", q_stride, self.weights.dtype if expanded else rows.torch.float32)
+        append = LatentAppend(src=lat.data_ptr() + 4 * self.q_rank, src_stride=lat_stride, width=self.kv_rank,
+                              weight=self.kv_norm.data_ptr(), eps=self.eps, cache_dtype=self.weights.tag,
+                              cache=state.data.data_ptr(), ring=state.rows, stride=state.stride)
+        rows.dense(ctx, self.uq, input=IN_NORM, x=lat, x_stride=lat_stride, norm=NORM_RMS, norm_weight=self.q_norm,
+                   norm_eps=self.eps, append=append, out=q, out_stride=q_stride,
+                   out_dtype=self.weights.tag if expanded else QK_F32)
+        o_stride = padded(self.heads * self.vdim)
+        att = rows.buffer("attention", o_stride)
+        if expanded:
+            self._expanded(ctx, rows, q, q_stride, att, o_stride, state, window)
+        else:
+            splits = self.n_splits(n, window)
+            scratch = rows.buffer("splits", self._split_floats(rows, window), rows.torch.float32, rows=1)
+            c = LatentCall(
+                tokens=n, positions=rows.positions.data_ptr(), slots=rows.slots.data_ptr(), heads=self.heads,
+                dim=self.dim, dim_stride=self.dim_stride, vdim=self.vdim, vdim_stride=self.vdim_stride,
+                kv_rank=self.kv_rank, kv_stride=self.kv_stride, window=window, ring=state.rows,
+                n_slots=state.data.shape[0], scale=self.scale, q=q.data_ptr(), q_dtype=QK_F32, q_stride=q_stride,
+                w_dtype=self.weights.tag, uk=self.ukv.w.data_ptr(),
+                uv=self.ukv.w[self.heads * self.dim_stride:].data_ptr(), cache=state.data.data_ptr(),
+                n_splits=splits, scratch=scratch.data_ptr(), out=att.data_ptr(), out_dtype=rows.act_tag,
+                out_stride=o_stride)
+            check(lib.qk_latent_attention(ctx.handle, ctypes.byref(c)))
+        rows.dense(ctx, self.out, input=IN_PLAIN, x=att, x_dtype=rows.act_tag, x_stride=o_stride,
+                   **rows.residual_fields(scale))
+
+    def _expanded(self, ctx, rows: Rows, q, q_stride, att, o_stride, state: RingCache, window: int) -> None:
+        lib = _lib.lib()
+        slot, p0 = rows.portion
+        first = max(0, p0 - window + 1)
+        keys = p0 + rows.n - first
+        kv_row = padded(self.ukv.rows)
+        lat = rows.buffer("window", self.kv_stride, self.weights.dtype, rows=state.rows)
+        kv = rows.buffer("keys", kv_row, self.weights.dtype, rows=state.rows)
+        check(lib.qk_latent_gather(ctx.handle, c_void_p(state.data.data_ptr()), self.weights.tag, state.rows,
+                                   state.stride, slot, first, keys, c_void_p(lat.data_ptr())))
+        d = rows.call(self.ukv, tokens=keys, input=IN_PLAIN, x=lat, x_dtype=self.weights.tag, x_stride=self.kv_stride,
+                      out=kv, out_stride=kv_row, out_dtype=self.weights.tag)
+        check(lib.qk_dense(ctx.handle, ctypes.byref(d)))
+        check(lib.qk_window_attention(ctx.handle, c_void_p(q.data_ptr()), q_stride, c_void_p(kv.data_ptr()), kv_row,
+                                      first, keys, p0, rows.n, self.heads, self.dim_stride, self.vdim,
+                                      self.vdim_stride, window, self.scale, c_void_p(att.data_ptr()), o_stride))
+
+
+class GatedDelta:
+    """Gated delta rule with short causal convolutions and one decay per head."""
+
+    def __init__(self, weights: Weights, tensors: dict, *, heads: int, kv_heads: int, dim: int, vdim: int, taps: int,
+                 eps: float, unit_eps: float):
+        self.heads, self.kv_heads, self.dim, self.vdim, self.taps = heads, kv_heads, dim, vdim, taps
+        self.eps, self.unit_eps = float(eps), float(unit_eps)
+        t, w = tensors, weights
+        self.proj = w.matrix(t["q"], t["k"], t["v"], t["g"], t["b"], t["a"])
+        self.channels = 2 * kv_heads * dim + heads * vdim
+        self.gate_at = self.channels
+        self.beta_at = self.gate_at + heads * vdim
+        self.decay_at = self.beta_at + heads
+        self.conv = [w.vector(t[n + ".conv"]) for n in ("q", "k", "v")]
+        self.a_log, self.dt_bias, self.norm = w.vector(t["A_log"]), w.vector(t["dt_bias"]), w.vector(t["norm"])
+        self.out = w.matrix(t["o"])
+
+    def make_state(self, torch, device, slots: int, max_seq: int, portion: int) -> RecurrentState:
+        return RecurrentState(torch, device, slots, self.heads, self.dim, self.vdim, self.taps, self.channels)
+
+    def forward(self, ctx, rows: Rows, norm: int, norm_weight, norm_eps: float, scale, state: RecurrentState,
+                max_seq: int) -> None:
+        stride = up_to(self.proj.rows, 8)
+        proj = rows.f32("projections", stride)
+        rows.dense(ctx, self.proj, **rows.stream_fields(norm, norm_weight, norm_eps), out=proj, out_stride=stride)
+        rows.settle()
+        o_stride = padded(self.heads * self.vdim)
+        out = rows.f32("readout", o_stride)
+        qkv, gates = rows.f32("qkv", self.channels), rows.f32("gates", self.heads * 4)
+        c = DeltaCall(tokens=rows.n, segments=rows.segments, positions=rows.positions.data_ptr(),
+                      slots=rows.slots.data_ptr(), seg_first=rows.seg_first.data_ptr(),
+                      seg_len=rows.seg_len.data_ptr(), seg_row=rows.seg_row.data_ptr(), heads=self.heads,
+                      kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, taps=self.taps, proj=proj.data_ptr(),
+                      proj_stride=stride, beta_offset=self.beta_at, decay_offset=self.decay_at,
+                      conv_q=self.conv[0].data_ptr(), conv_k=self.conv[1].data_ptr(), conv_v=self.conv[2].data_ptr(),
+                      a_log=self.a_log.data_ptr(), dt_bias=self.dt_bias.data_ptr(), unit_eps=self.unit_eps,
+                      conv_state=state.conv.data_ptr(), state=state.matrix.data_ptr(), qkv=qkv.data_ptr(),
+                      gates=gates.data_ptr(), out=out.data_ptr(), out_stride=o_stride)
+        check(_lib.lib().qk_delta(ctx.handle, ctypes.byref(c)))
+        rows.dense(ctx, self.out, input=IN_GATED, x=out, x_stride=o_stride, gate=proj.data_ptr() + 4 * self.gate_at,
+                   gate_stride=stride, group=self.vdim, norm_weight=self.norm, norm_eps=self.eps,
+                   **rows.residual_fields(scale))
+
+
+class GatedMlp:
+    """W_down (act(W_gate h) * (W_up h))."""
+
+    def __init__(self, weights: Weights, tensors: dict, *, activation: str):
+        self.pair = weights.gated_pair(tensors["gate"], tensors["up"])
+        self.down = weights.matrix(tensors["down"])
+        self.act = ACTIVATIONS[activation]
+
+    def forward(self, ctx, rows: Rows, norm: int, norm_weight, norm_eps: float, scale) -> None:
+        stride = self.down.k
+        ff = rows.buffer("ff", stride)
+        rows.dense(ctx, self.pair, **rows.stream_fields(norm, norm_weight, norm_eps), output=OUT_GLU,
+                   activation=self.act, out=ff, out_stride=stride, out_dtype=rows.act_tag)
+        rows.settle()
+        rows.dense(ctx, self.down, input=IN_PLAIN, x=ff, x_dtype=rows.act_tag, x_stride=stride,
+                   **rows.residual_fields(scale))
+
+
+class TokenSide:
+    """Per-layer token input: norm(W_proj (gelu(W_gate x) * e)) is left pending on the stream, e
+    being ``dim`` columns of the token's row of ``table`` from ``offset`` on."""
+
+    def __init__(self, weights: Weights, tensors: dict, table, *, dim: int, offset: int, eps: float):
+        self.gate, self.proj = weights.matrix(tensors["gate"]), weights.matrix(tensors["proj"])
+        self.norm, self.table, self.dim, self.offset, self.eps = (weights.vector(tensors["norm"]), table, dim, offset,
+                                                                  float(eps))
+
+    def forward(self, ctx, rows: Rows) -> None:
+        x, tag = rows.stream_rows()
+        s = rows.buffer("side", self.proj.k)
+        rows.dense(ctx, self.gate, input=IN_PLAIN, x=x, x_dtype=tag, x_stride=rows.stride, output=OUT_SIDE,
+                   activation=ACTIVATIONS["gelu_tanh"], side=self.table, side_dtype=rows.weights.tag,
+                   side_stride=self.table.shape[1], side_offset=self.offset, vocab=self.table.shape[0], out=s,
+                   out_stride=self.proj.k, out_dtype=rows.act_tag)
+        y = rows.f32("side result", rows.stride)
+        rows.dense(ctx, self.proj, input=IN_PLAIN, x=s, x_dtype=rows.act_tag, x_stride=self.proj.k, out=y,
+                   out_stride=rows.stride)
+        rows.pending = (y, self.norm, self.eps)
