@@ -22,6 +22,7 @@ kernels are Rust and no Rust toolchain exists on this image.
 from __future__ import annotations
 
 import argparse
+import ctypes
 import json
 import os
 import statistics
@@ -624,6 +625,306 @@ def run_attention(args, local_rank: int) -> None:
         "gpu_launches": int(launches), "clocks": clocks}))
 
 
+LAYERED_SIZES = {
+    # width, heads, latent rank, query rank, window, ff, delta heads / key heads, side dim
+    "2048": dict(width=2048, heads=16, kv_rank=512, q_rank=768, window=2048, ff=8192, dheads=16, dkv=8, side=128),
+    "4096": dict(width=4096, heads=32, kv_rank=512, q_rank=1536, window=4096, ff=14336, dheads=32, dkv=16, side=256),
+}
+LAYERED_VOCAB, LAYERED_RUNS = 32768, 8
+
+
+def layered_config(size: str) -> dict:
+    """A Vogizen config with the layer sizes of a real model: attention and delta layers in turn,
+    a feed-forward on every second one, the first two layers looped, eight layer runs."""
+    z = LAYERED_SIZES[size]
+    att = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+           "mixer": {"heads": z["heads"], "dim": 128, "vdim": 128, "kv_rank": z["kv_rank"], "q_rank": z["q_rank"],
+                     "scale": 128 ** -0.5, "mask": {"size": z["window"]}}}
+    rec = {"type": "delta", "mlp": None,
+           "mixer": {"heads": z["dheads"], "kv_heads": z["dkv"], "dim": 128, "vdim": 128, "conv": 4}}
+    return {"architecture": "Vogizen", "width": z["width"], "vocab": LAYERED_VOCAB, "norm": {"eps": 1e-5},
+            "embedding": {"scale": z["width"] ** 0.5}, "token_side": {"dim": z["side"]},
+            "loop": {"start": 0, "stop": 2, "times": 2}, "layers": [att, rec] * 3}
+
+
+def layered_tensors(config: dict, seed: int = 0) -> dict:
+    import torch
+    from quantibbler_b200 import vogizen
+    gen = torch.Generator(device="cuda").manual_seed(seed)
+    out = {}
+    for name, shape in vogizen.shapes(config).items():
+        t = torch.randn(shape, device="cuda", generator=gen)
+        if name.endswith(("A_log", "dt_bias")):
+            t = t * 0.1 - 1.0
+        elif len(shape) == 1:
+            t = 1.0 + 0.1 * t
+        else:
+            t = t / shape[-1] ** 0.5
+        out[name] = t.to(torch.bfloat16)
+    return out
+
+
+def graph_ms(ctx, calls, repeats: int = 10) -> float:
+    """Device time per call of a captured sequence of library calls (CUDA events around replays)."""
+    import torch
+    stream = torch.cuda.Stream()
+    torch.cuda.synchronize()
+    ctx.set_stream(stream.cuda_stream)
+    with torch.cuda.stream(stream):
+        for f in calls:
+            f()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph, stream=stream):
+        for f in calls:
+            f()
+    for _ in range(3):
+        graph.replay()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(repeats):
+        graph.replay()
+    b.record()
+    torch.cuda.synchronize()
+    ctx.synchronize()
+    return a.elapsed_time(b) / repeats / len(calls)
+
+
+def timed_prompt(dec, n: int, vocab: int) -> float:
+    """ms of one prompt of n tokens (third run), CUDA events on the decoder's stream."""
+    import torch
+    prompt = torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(3)).tolist()
+    handle = dec.ctx.stream
+    stream = torch.cuda.ExternalStream(handle) if handle > 2 else torch.cuda.default_stream()
+    for _ in range(3):
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        a.record(stream)
+        dec.prefill(prompt, seq=0, first_position=0)
+        b.record(stream)
+        torch.cuda.synchronize()
+    return a.elapsed_time(b)
+
+
+def timed_decode(dec, context: int, steps: int, warmup: int) -> float:
+    """ms per step of the captured batched step at the given context."""
+    import torch
+    B = dec.cfg.max_batch
+    dec.start(torch.randint(0, dec.cfg.vocab, (B,)).tolist(), [context] * B)
+    dec.capture()
+    for _ in range(max(warmup, 3)):
+        dec.graph.replay()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    a.record()
+    for _ in range(steps):
+        dec.graph.replay()
+    b.record()
+    torch.cuda.synchronize()
+    dec.ctx.synchronize()
+    return a.elapsed_time(b) / steps
+
+
+def layered_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
+    """The design's kernels one at a time: captured sequences over the layers' own weights (more
+    than L2 holds), against the roofline that bounds each."""
+    import torch
+    from quantibbler_b200 import layers as L
+    hbm, tc = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    out = {}
+    lays = dec.layers
+
+    def note(name, ms, bytes_=None, flops=None, peak_flops=None):
+        e = {"us": ms * 1e3}
+        if bytes_ is not None:
+            e.update(bound="hbm", gbs=bytes_ / ms / 1e6, frac=bytes_ / ms / 1e6 / hbm)
+        else:
+            e.update(bound="tensor" if peak_flops is None else "float32", tflops=flops / ms / 1e9,
+                     frac=flops / ms / 1e9 / (peak_flops or tc))
+        out[name] = e
+
+    att = [x for x in lays if isinstance(x.mixer, L.LatentAttention)]
+    rec = [x for x in lays if isinstance(x.mixer, L.GatedDelta)]
+    states = {id(layer): st for layer, _, st in dec.runs}
+
+    for T in (1, 64, tokens):
+        vector = T <= dec.cfg.vector_rows
+        rows = L.Rows(torch, dec.device, T, dec.stride, dec.weights, vector=vector)
+        rows.positions.copy_(torch.arange(T) + dec.bench_context)
+        x = torch.randn(T, 1 << 15, device="cuda").to(rows.act)
+        o = torch.zeros(T, 1 << 15, device="cuda")
+        for name, lins, kind in (("delta projections", [x_.mixer.proj for x_ in rec], L.OUT_STORE),
+                                 ("gate, up", [x_.mlp.pair for x_ in att], L.OUT_GLU),
+                                 ("down", [x_.mlp.down for x_ in att], L.OUT_STORE),
+                                 ("output of the mixer", [x_.mixer.out for x_ in lays], L.OUT_STORE)):
+            calls = []
+            for m in lins:
+                f = dict(input=L.IN_PLAIN, x=x, x_dtype=rows.act_tag, x_stride=1 << 15, output=kind, out=o,
+                         out_stride=1 << 15)
+                calls.append(lambda m=m, f=f: rows.dense(ctx, m, **f))
+            ms = graph_ms(ctx, calls * 4)
+            if T == tokens:
+                note(f"{name}, {T} rows", ms, flops=2.0 * T * lins[0].rows * lins[0].width)
+            else:
+                note(f"{name}, {T} rows", ms, bytes_=2.0 * lins[0].rows * lins[0].width)
+        # the mixers' own kernels: everything of a mixer but its linears
+        if T == tokens:
+            rows.portion = (0, 0)
+            rows.positions.copy_(torch.arange(T))
+            rows.segments = 1
+            rows.seg_first[:1].fill_(0)
+            rows.seg_len[:1].fill_(T)
+            rows.seg_row.copy_(torch.arange(T))
+            rows.slots.fill_(0)
+        elif T > dec.cfg.max_batch:
+            rows.slots.fill_(0)   # (rows of one slot: only the time counts)
+        real = rows.dense
+        skip = lambda *a, **k: None
+        rows.dense = skip
+        m = rec[0].mixer
+        ms = graph_ms(ctx, [lambda x_=x_: x_.mixer.forward(ctx, rows, 0, x_.norm1, 1e-5, None, states[id(x_)], 1 << 20)
+                            for x_ in rec] * 4)
+        if T == tokens:
+            note(f"delta rule (convolution and recurrence), {T} rows", ms,
+                 flops=6.0 * T * m.heads * m.dim * m.vdim, peak_flops=148 * 128 * 2 * 1.965e-3)
+        else:
+            note(f"delta rule (convolution and recurrence), {T} rows", ms, bytes_=8.0 * T * m.heads * m.dim * m.vdim)
+        m = att[0].mixer
+        ms = graph_ms(ctx, [lambda x_=x_: x_.mixer.forward(ctx, rows, 0, x_.norm1, 1e-5, None, states[id(x_)], 1 << 20)
+                            for x_ in att] * 4)
+        if T == tokens:
+            pairs = sum(min(i + 1, m.window) for i in range(T))
+            note(f"window attention (with gather and expansion), {T} rows", ms,
+                 flops=2.0 * m.heads * (m.dim + m.vdim) * (pairs + T * m.kv_rank))
+        else:
+            keys = min(m.window, dec.bench_context + 1)
+            note(f"latent attention, {T} rows", ms,
+                 bytes_=2.0 * (T * keys * m.kv_rank + m.heads * (m.dim + m.vdim) * m.kv_rank))
+        rows.dense = real
+    return out
+
+
+def closest_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
+    """The like kernels of the factorized Llama-shaped decoder, timed the same way."""
+    import torch
+    from quantibbler_b200.gpu import apply_prefill_many
+    hbm, tc = peaks["hbm_gbs"], peaks["bf16_tflops"]
+    out = {}
+    for name in ("q", "gate", "down", "o"):
+        lays = [x[name] for x in dec.layers]
+        d = lays[0]
+        x = torch.randn(tokens, d.din, device="cuda")
+        y = torch.zeros(tokens, d.dout, device="cuda")
+        bits = d.r * (d.din + d.dout) / 8
+        for T in (64, tokens):
+            calls = [lambda m=m: apply_prefill_many([m], x.data_ptr(), T, [y.data_ptr()]) for m in lays]
+            ms = graph_ms(ctx, calls * 4)
+            if T == tokens:
+                fl = 2.0 * T * d.r * (d.din + d.dout)
+                out[f"{name}, {T} rows"] = {"us": ms * 1e3, "bound": "tensor", "tflops": fl / ms / 1e9,
+                                            "frac": fl / ms / 1e9 / tc}
+            else:
+                out[f"{name}, {T} rows"] = {"us": ms * 1e3, "bound": "hbm", "gbs": bits / ms / 1e6,
+                                            "frac": bits / ms / 1e6 / hbm}
+    for name, parts in (("qkv", "qkv"), ("gu", ("gate", "up")), ("o", "o"), ("down", ("down",))):
+        if name in dec.plans[0]:
+            ms = graph_ms(ctx, [p[name].apply for p in dec.plans] * 4)
+            bits = sum(dec.layers[0][n].r * (dec.layers[0][n].din + dec.layers[0][n].dout) / 8 for n in parts)
+            out[f"{name}, 1 row"] = {"us": ms * 1e3, "bound": "hbm", "gbs": bits / ms / 1e6, "frac": bits / ms / 1e6 / hbm}
+    cfg, lib = dec.cfg, _qk_lib()
+    P = lambda t: ctypes.c_void_p(t.data_ptr())
+    H, KV, hd = dec.h_loc, dec.kv_loc, cfg.head_dim
+    q, o = torch.randn(tokens, H * hd, device="cuda"), torch.zeros(tokens, H * hd, device="cuda")
+    ms = graph_ms(ctx, [lambda i=i: lib.qk_prefill_attention(
+        ctx.handle, P(q), P(dec.cache_k[i]), P(dec.cache_v[i]), dec.kv_tag, 0, 0, tokens, H, KV, hd, cfg.max_seq, P(o))
+        for i in range(cfg.n_layers)])
+    fl = 4.0 * H * hd * tokens * (tokens + 1) / 2
+    out[f"prefill attention, {tokens} rows"] = {"us": ms * 1e3, "bound": "tensor", "tflops": fl / ms / 1e9,
+                                                "frac": fl / ms / 1e9 / tc}
+    dec.kv_len.fill_(dec.bench_context)
+    ms = graph_ms(ctx, [lambda i=i: lib.qk_decode_attention(
+        ctx.handle, P(q), P(dec.cache_k[i]), P(dec.cache_v[i]), dec.kv_tag, P(dec.kv_len), 1, H, KV, hd, cfg.max_seq,
+        dec.n_splits, P(dec.att_scratch), P(o)) for i in range(cfg.n_layers)] * 4)
+    by = 4.0 * KV * hd * dec.bench_context
+    out["decode attention, 1 row"] = {"us": ms * 1e3, "bound": "hbm", "gbs": by / ms / 1e6, "frac": by / ms / 1e6 / hbm}
+    return out
+
+
+def _qk_lib():
+    from quantibbler_b200 import _lib
+    return _lib.lib()
+
+
+def run_layered(args, local_rank: int) -> None:
+    """Prefill and decode throughput of the Vogizen design at the layer sizes of real models (random
+    weights) beside the factorized Llama-shaped decoder with the same width, heads, feed-forward,
+    vocabulary and number of layer runs."""
+    import torch
+
+    from quantibbler_b200 import vogizen
+    from quantibbler_b200.decoder import Decoder, DecoderConfig, random_model
+    from quantibbler_b200.gpu import GpuContext
+    from quantibbler_b200.layered import LayeredDecoder
+    torch.cuda.set_device(local_rank)
+    ctx = GpuContext.init_at(local_rank)
+    peaks_path = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    peaks = json.load(open(peaks_path)) if os.path.exists(peaks_path) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    tokens, context = args.tokens, args.context
+    sizes, launches = {}, 0
+    with ClockSampler(local_rank) as clocks:
+        for size in args.layered_sizes.split(","):
+            z = LAYERED_SIZES[size]
+            config = layered_config(size)
+            tensors = layered_tensors(config)
+            res = {"layer_runs": LAYERED_RUNS, "vocab": LAYERED_VOCAB, **z}
+            for name in ("vogizen", "closest"):
+                r = {}
+                for batch in (1, 64):
+                    if name == "vogizen":
+                        dec = LayeredDecoder(ctx, vogizen.parse(config, max_seq=context + 4096, max_batch=batch), tensors)
+                        for _, _, st in dec.runs:
+                            for t in vars(st).values():
+                                if isinstance(t, torch.Tensor):
+                                    t.normal_(std=0.1)
+                    else:
+                        ranks = {k: max(64, int(v * z["width"] / 4096) // 2 * 2) for k, v in C4_RANKS.items()}
+                        cfg = DecoderConfig(n_layers=LAYERED_RUNS, d_model=z["width"], n_heads=z["heads"],
+                                            n_kv_heads=max(1, z["heads"] // 4), head_dim=128, d_ff=z["ff"],
+                                            vocab=LAYERED_VOCAB, serving="bfloat16", max_seq=context + 4096,
+                                            max_batch=batch)
+                        dec = Decoder(ctx, cfg, random_model(cfg, ranks, device_tables=True))
+                    dec.bench_context = context
+                    if batch == 1:
+                        ms = timed_prompt(dec, tokens, LAYERED_VOCAB)
+                        r["prefill"] = {"tokens": tokens, "ms": ms, "tok_s": tokens / ms * 1e3}
+                    ms = timed_decode(dec, context, args.steps, args.warmup)
+                    launches += dec.kernels_per_step * args.steps
+                    r[f"decode_batch{batch}"] = {"context": context, "ms_per_step": ms, "tok_s": batch / ms * 1e3,
+                                                 "kernels_per_step": dec.kernels_per_step}
+                    if batch == 1 and args.layered_kernels:
+                        dec.graph = None
+                        r["kernels"] = (layered_kernels if name == "vogizen" else closest_kernels)(
+                            ctx, dec, tokens, peaks)
+                    dec.graph = None
+                    del dec
+                    ctx.set_stream(None)
+                    torch.cuda.empty_cache()
+                res[name] = r
+            sizes[size] = res
+            print(f"width {size}: {json.dumps(res)}", file=sys.stderr, flush=True)
+            del tensors
+    head = sizes[args.layered_sizes.split(",")[-1]]["vogizen"]
+    print(json.dumps({
+        "metric": "layered_decode_tok_s", "value": head["decode_batch1"]["tok_s"], "unit": "tok/s", "n_gpus": 1,
+        "steps": args.steps, "warmup": max(args.warmup, 3), "ms_per_step": head["decode_batch1"]["ms_per_step"],
+        "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+        "config": {"workload": "Vogizen layers at real sizes, random weights, beside the factorized Llama-shaped "
+                               "decoder of equal width, heads, feed-forward, vocabulary and layer runs",
+                   "global_batch": 1, "seq_len": context,
+                   "l2_policy": "weights larger than L2, streamed every step", "sizes": sizes},
+        "gpu_launches": launches, "clocks": clocks.summary()}), flush=True)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -638,8 +939,10 @@ def main() -> None:
                     help="sub-groups of the host-buffer pipeline (0: HostLayerGroup's own choice)")
     ap.add_argument("--e2e-applies", type=int, default=296,
                     help="layers of the one-call-per-layer leg (0 switches both end-to-end legs off)")
-    ap.add_argument("--workload", default="gemv", choices=["gemv", "decode", "prefill", "attention"])
+    ap.add_argument("--workload", default="gemv", choices=["gemv", "decode", "prefill", "attention", "layered"])
     ap.add_argument("--tokens", type=int, default=2048)
+    ap.add_argument("--layered-sizes", default="2048,4096", help="layered workload: widths, with commas between them")
+    ap.add_argument("--layered-kernels", type=int, default=1, help="layered workload: also time the kernels one by one")
     ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "llama2-7b-layer"])
     ap.add_argument("--batch", type=int, default=1)
     ap.add_argument("--context", type=int, default=2048)
@@ -678,6 +981,10 @@ def main() -> None:
     if args.workload == "attention":
         if rank == 0:
             run_attention(args, local_rank)
+        return
+    if args.workload == "layered":
+        if rank == 0:
+            run_layered(args, local_rank)
         return
     if args.workload == "prefill":
         if rank == 0:

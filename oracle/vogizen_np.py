@@ -11,6 +11,29 @@ from __future__ import annotations
 import numpy as np
 
 
+_operand = None   # rounding of the linears' inputs while ``rounded_operands`` is in force
+
+
+class rounded_operands:
+    """with rounded_operands(fn): every linear reads fn(its input), the rest stays exact - what a
+    16-bit matrix product does at the least, hence a measure of a model's sensitivity to it."""
+
+    def __init__(self, fn):
+        self.fn = fn
+
+    def __enter__(self):
+        global _operand
+        _operand = self.fn
+
+    def __exit__(self, *exc):
+        global _operand
+        _operand = None
+
+
+def linear(h, w):
+    return (h if _operand is None else _operand(h).astype(h.dtype)) @ w.T
+
+
 def sigmoid(z):
     return 1.0 / (1.0 + np.exp(-z))
 
@@ -58,10 +81,10 @@ def causal_conv(x, taps):
 def latent_attention(h, m, w, eps, return_weights=False):
     """Windowed latent attention without positions; ``w`` holds the mixer's tensors."""
     T, H, dim, vdim = len(h), m["heads"], m["dim"], m["vdim"]
-    q = (rms_norm(h @ w["dq"].T, w["dq.norm"], eps) @ w["uq"].T).reshape(T, H, dim)
-    c = rms_norm(h @ w["dkv"].T, w["dkv.norm"], eps)
-    k = (c @ w["uk"].T).reshape(T, H, dim)
-    v = (c @ w["uv"].T).reshape(T, H, vdim)
+    q = linear(rms_norm(linear(h, w["dq"]), w["dq.norm"], eps), w["uq"]).reshape(T, H, dim)
+    c = rms_norm(linear(h, w["dkv"]), w["dkv.norm"], eps)
+    k = linear(c, w["uk"]).reshape(T, H, dim)
+    v = linear(c, w["uv"]).reshape(T, H, vdim)
     back = np.arange(T)[:, None] - np.arange(T)[None, :]
     seen = (back >= 0) & (back < m["mask"]["size"])
     out = np.zeros((T, H, vdim), h.dtype)
@@ -72,7 +95,7 @@ def latent_attention(h, m, w, eps, return_weights=False):
         p /= p.sum(axis=1, keepdims=True)
         probs.append(p)
         out[:, a] = p @ v[:, a]
-    y = out.reshape(T, H * vdim) @ w["o"].T
+    y = linear(out.reshape(T, H * vdim), w["o"])
     return (y, np.stack(probs)) if return_weights else y
 
 
@@ -92,7 +115,7 @@ def delta_mixer(h, m, w, eps):
     T, H, KV, dim, vdim = len(h), m["heads"], m["kv_heads"], m["dim"], m["vdim"]
 
     def branch(name, heads, size):
-        return silu(causal_conv(h @ w[name].T, w[name + ".conv"])).reshape(T, heads, size)
+        return silu(causal_conv(linear(h, w[name]), w[name + ".conv"])).reshape(T, heads, size)
 
     def unit(x):
         return x / np.sqrt((x ** 2).sum(axis=-1, keepdims=True) + 1e-6)
@@ -100,24 +123,24 @@ def delta_mixer(h, m, w, eps):
     q = unit(branch("q", KV, dim)) * dim ** -0.5
     k = unit(branch("k", KV, dim))
     v = branch("v", H, vdim)
-    beta = sigmoid(h @ w["b"].T)
-    decay = np.exp(-np.exp(w["A_log"]) * softplus(h @ w["a"].T + w["dt_bias"]))
-    gate = silu(h @ w["g"].T).reshape(T, H, vdim)
+    beta = sigmoid(linear(h, w["b"]))
+    decay = np.exp(-np.exp(w["A_log"]) * softplus(linear(h, w["a"]) + w["dt_bias"]))
+    gate = silu(linear(h, w["g"])).reshape(T, H, vdim)
     out = np.zeros((T, H, vdim), h.dtype)
     for a in range(H):
         src = a // (H // KV)
         out[:, a], _ = delta_rule(q[:, src], k[:, src], v[:, a], beta[:, a], decay[:, a])
     y = rms_norm(out, w["norm"], eps) * gate
-    return y.reshape(T, H * vdim) @ w["o"].T
+    return linear(y.reshape(T, H * vdim), w["o"])
 
 
 def relu_mlp(h, w):
-    return (np.maximum(h @ w["gate"].T, 0.0) * (h @ w["up"].T)) @ w["down"].T
+    return linear(np.maximum(linear(h, w["gate"]), 0.0) * linear(h, w["up"]), w["down"])
 
 
 def token_side(x, rows, w, eps):
     """``rows`` [T, dim]: this layer's part of the tokens' side embedding."""
-    y = (gelu_tanh(x @ w["gate"].T) * rows) @ w["proj"].T
+    y = linear(gelu_tanh(linear(x, w["gate"])) * rows, w["proj"])
     return x + rms_norm(y, w["norm"], eps)
 
 
@@ -149,7 +172,7 @@ def forward(cfg, weights, tokens, ft=np.float64, per_layer=None):
         layer = cfg["layers"][i]
         w = part(f"l{i}.")
         if starts_pass:
-            x = np.concatenate([x, x0], axis=1) @ W["loop.in"].T
+            x = linear(np.concatenate([x, x0], axis=1), W["loop.in"])
         mixed = MIXERS[layer["type"]](layer_norm(x, w["norm1"], eps), layer["mixer"], part(f"l{i}.mix."), eps)
         x = x + mixed * w["ls1"]
         if layer["mlp"] is not None:
@@ -159,4 +182,4 @@ def forward(cfg, weights, tokens, ft=np.float64, per_layer=None):
             x = token_side(x, W["side.embed"][tokens, i * dim:(i + 1) * dim], part(f"l{i}.side."), eps)
         if per_layer is not None:
             per_layer.append(x)
-    return layer_norm(x, W["final.norm"], eps) @ W["embed"].T
+    return linear(layer_norm(x, W["final.norm"], eps), W["embed"])
