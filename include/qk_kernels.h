@@ -635,7 +635,7 @@ typedef struct {
  * takes) run as one launch that forms the input in every block; more rows as a launch for the
  * input (none for a plain input of the weights' dtype) and a matrix product. */
 qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *call);
-enum { QK_FORM_VECTOR = 0, QK_FORM_SKINNY = 1, QK_FORM_TCGEN05 = 2, QK_FORM_F32 = 3 };
+enum { QK_FORM_VECTOR = 0, QK_FORM_NARROW = 1, QK_FORM_TCGEN05 = 2, QK_FORM_F32 = 3 };
 int32_t qk_dense_form(size_t tokens, size_t k, int32_t w_dtype);
 /* Only the input rows: out [tokens][k] in out_dtype (stride k). */
 qk_status qk_dense_input(qk_ctx *ctx, const qk_dense_call *call);
@@ -666,7 +666,7 @@ typedef struct {
     float unit_eps;
     float *conv_state, *state;
     float *qkv;                              /* scratch [tokens][2*kv_heads*dim + heads*vdim] */
-    float *gates;                            /* scratch [tokens][heads][4] */
+    float *gates;                            /* scratch [tokens rounded up to 8][heads][20] */
     float *out;                              /* [tokens][heads*vdim], stride out_stride */
     size_t out_stride;
 } qk_delta_call;

@@ -8,6 +8,8 @@
 // through all tokens of a sequence portion while the next tokens' k, q and v arrive by cp.async.
 // Both dot products of a token read the OLD state, so that only one reduction lies between two
 // tokens: S^T k after the decay is g (S_old^T k), and o = g (S_old^T q) + (k . q) u.
+#include <algorithm>
+
 #include "qk_dense_dev.cuh"
 
 namespace {
@@ -50,86 +52,6 @@ struct DeltaArgs {
     float unit_eps;
 };
 
-// Convolution and silu of channel c (of q | k | v, as the projection lays them out) at row t.
-__device__ __forceinline__ float conv_silu(const DeltaArgs &a, uint32_t t, int pos, uint32_t in_seg, uint32_t slot,
-                                           const float *__restrict__ taps, uint32_t c) {
-    float y = 0.f;
-    for (uint32_t back = 0; back < a.taps; ++back) {
-        float v = 0.f;
-        if (in_seg >= back) v = a.proj[(size_t)(t - back) * a.proj_stride + c];
-        else if (pos >= (int)back)
-            v = a.conv_state[((size_t)slot * a.taps + (uint32_t)(pos - (int)back) % a.taps) * a.channels + c];
-        y = fmaf(taps[a.taps - 1 - back], v, y);
-    }
-    return silu_f(y);
-}
-
-constexpr int kPrepThreads = 256, kMaxLane = 16;  // dim up to 32 * kMaxLane
-__global__ void __launch_bounds__(kPrepThreads)
-delta_inputs_kernel(DeltaArgs a) {
-    qk::pdl_launch();
-    qk::pdl_wait();
-    extern __shared__ float kq[];  // [kv heads of this block]
-    const uint32_t t = blockIdx.x, warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-    const int pos = a.positions[t];
-    if (pos < 0) return;
-    const uint32_t in_seg = (uint32_t)a.seg_row[t], slot = (uint32_t)a.slots[t];
-    const uint32_t n_local = (a.kv_heads - blockIdx.y + gridDim.y - 1) / gridDim.y;  // kv heads y, y + parts, ..
-    const uint32_t ratio = a.heads / a.kv_heads, key0 = a.kv_heads * a.dim, val0 = 2 * key0;
-    float *row = a.qkv + (size_t)t * a.channels;
-    for (uint32_t i = warp; i < n_local; i += kPrepThreads / 32) {
-        const uint32_t c0 = (blockIdx.y + i * gridDim.y) * a.dim;
-        float q[kMaxLane], k[kMaxLane], sq = 0.f, sk = 0.f;
-#pragma unroll
-        for (int j = 0; j < kMaxLane; ++j) {
-            const uint32_t d = lane + 32 * j;
-            q[j] = k[j] = 0.f;
-            if (d < a.dim) {
-                q[j] = conv_silu(a, t, pos, in_seg, slot, a.conv_q + (size_t)(c0 + d) * a.taps, c0 + d);
-                k[j] = conv_silu(a, t, pos, in_seg, slot, a.conv_k + (size_t)(c0 + d) * a.taps, key0 + c0 + d);
-            }
-            sq += q[j] * q[j];
-            sk += k[j] * k[j];
-        }
-        for (int off = 16; off > 0; off >>= 1) {
-            sq += __shfl_xor_sync(0xffffffffu, sq, off);
-            sk += __shfl_xor_sync(0xffffffffu, sk, off);
-        }
-        const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)a.dim));
-        const float ik = 1.0f / sqrtf(sk + a.unit_eps);
-        float dot = 0.f;
-#pragma unroll
-        for (int j = 0; j < kMaxLane; ++j) {
-            const uint32_t d = lane + 32 * j;
-            const float qv = q[j] * iq, kv = k[j] * ik;
-            if (d < a.dim) {
-                row[c0 + d] = qv;
-                row[key0 + c0 + d] = kv;
-            }
-            dot += qv * kv;
-        }
-        for (int off = 16; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
-        if (lane == 0) kq[i] = dot;
-    }
-    // values: the channels of the heads that belong to these kv heads
-    const uint32_t per = ratio * a.vdim;
-    for (uint32_t i = threadIdx.x; i < n_local * per; i += kPrepThreads) {
-        const uint32_t c = (blockIdx.y + i / per * gridDim.y) * per + i % per;
-        row[val0 + c] = conv_silu(a, t, pos, in_seg, slot, a.conv_v + (size_t)c * a.taps, val0 + c);
-    }
-    __syncthreads();
-    const float *pr = a.proj + (size_t)t * a.proj_stride;
-    for (uint32_t i = threadIdx.x; i < n_local * ratio; i += kPrepThreads) {
-        const uint32_t h = (blockIdx.y + i / ratio * gridDim.y) * ratio + i % ratio;
-        const float z = pr[a.decay_offset + h] + a.dt_bias[h];
-        const float sp = z > 20.f ? z : log1pf(expf(z));
-        float *g = a.gates + ((size_t)t * a.heads + h) * 4;
-        g[0] = sigmoid_f(pr[a.beta_offset + h]);
-        g[1] = expf(-expf(a.a_log[h]) * sp);
-        g[2] = kq[i / ratio];
-    }
-}
-
 // ------------------------------------------------------------------ delta rule: the recurrence
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack2(float a, float b) {
@@ -157,6 +79,19 @@ __device__ __forceinline__ void copy_async4(float *smem, const float *gmem) {
 __device__ __forceinline__ void copy_async16(float *smem, const float *gmem) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem)
                  : "memory");
+}
+
+// The convolution's last taps - 1 inputs of a segment (their readers, the inputs kernel, have
+// finished), shared out over the blocks of a segment (grid x and y).
+__device__ __forceinline__ void keep_conv_inputs(const DeltaArgs &a, uint32_t slot, int pos0, uint32_t first,
+                                                 uint32_t len, uint32_t threads) {
+    const uint32_t keep = min(a.taps - 1, len);
+    const uint32_t n_blocks = gridDim.x * gridDim.y, block = blockIdx.y * gridDim.x + blockIdx.x;
+    for (uint32_t i = block * threads + threadIdx.x; i < keep * a.channels; i += n_blocks * threads) {
+        const uint32_t back = i / a.channels, c = i % a.channels, r = len - 1 - back;
+        a.conv_state[((size_t)slot * a.taps + (uint32_t)(pos0 + (int)r) % a.taps) * a.channels + c] =
+            a.proj[(size_t)(first + r) * a.proj_stride + c];
+    }
 }
 
 constexpr int kScanThreads = 128, kScanCols = kScanThreads / 8;  // columns per block
@@ -301,14 +236,357 @@ delta_scan_kernel(DeltaArgs a, int vec) {
             }
         }
     }
-    // the convolution's last taps - 1 inputs (their readers, the inputs kernel, have finished)
-    const uint32_t keep = min(a.taps - 1, len);
-    const uint32_t n_blocks = gridDim.x * gridDim.y, block = blockIdx.y * gridDim.x + blockIdx.x;
-    for (uint32_t i = block * kScanThreads + threadIdx.x; i < keep * a.channels; i += n_blocks * kScanThreads) {
-        const uint32_t back = i / a.channels, c = i % a.channels, r = len - 1 - back;
-        a.conv_state[((size_t)slot * a.taps + (uint32_t)(pos0 + (int)r) % a.taps) * a.channels + c] =
-            a.proj[(size_t)(first + r) * a.proj_stride + c];
+    keep_conv_inputs(a, slot, pos0, first, len, kScanThreads);
+}
+
+// ------------------------------------------------------------------ delta rule: a portion, eight tokens at a time
+// For eight tokens from a state S0 on, with P_t = g_1 .. g_t and R_ti = g_i+1 .. g_t:
+//   u_t = beta_t (v_t - P_t S0^T k_t - sum_{i<t} R_ti (k_i . k_t) u_i)
+//   o_t = P_t S0^T q_t + sum_{i<=t} R_ti (k_i . q_t) u_i
+//   S8  = P_8 S0 + sum_i R_8i k_i u_i^T
+// so all sixteen products with the state are independent, and only an 8 x 8 triangular solve of
+// scalars per column is sequential.  The scalars depend on the head alone: the inputs kernel
+// writes them once, 20 floats per token: beta R (k . k) [8], R (k . q) [8], beta, beta P, P, R_8.
+constexpr int kMini = 8, kCoef = 20;
+
+// A block takes kTok rows and one key head with the heads it serves.  Thread per channel: convolution
+// and silu of the rows from one window of loads (kTaps bounds the taps), then a warp per row for
+// the unit norms, then the scalars.  kTok = 8: rows of one portion, kCoef scalars per row and
+// head; kTok = 1: any row, {beta, g, k . q} per row and head.
+template <int kTaps, int kTok>
+__global__ void __launch_bounds__(256)
+delta_inputs_kernel(DeltaArgs a, uint32_t n_tokens) {
+    qk::pdl_launch();
+    extern __shared__ float ci_smem[];  // q, k [kTok][dim + 1], then products, then [ratio][kTok][2] gates
+    const uint32_t t0 = blockIdx.x * kTok, kvh = blockIdx.y, pitch = a.dim + 1, ratio = a.heads / a.kv_heads;
+    float *qs = ci_smem, *ks = qs + kTok * pitch, *prod = ks + kTok * pitch, *gate = prod + 2 * kTok * kTok;
+    const uint32_t n = min((uint32_t)kTok, n_tokens - t0), warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    qk::pdl_wait();
+    const int pos = a.positions[t0];
+    if (pos < 0) return;
+    const int in_seg = a.seg_row[t0];
+    const uint32_t slot = (uint32_t)a.slots[t0], key0 = a.kv_heads * a.dim, per = ratio * a.vdim;
+    for (uint32_t c = threadIdx.x; c < 2 * a.dim + per; c += 256) {
+        const uint32_t which = c < a.dim ? 0 : c < 2 * a.dim ? 1 : 2;
+        const uint32_t in = which == 0 ? c : which == 1 ? c - a.dim : c - 2 * a.dim;   // place in this head's part
+        const uint32_t own = which == 2 ? kvh * per + in : kvh * a.dim + in;          // row of the taps
+        const uint32_t ch = which == 0 ? own : which == 1 ? key0 + own : 2 * key0 + own;
+        const float *taps = (which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v) + (size_t)own * a.taps;
+        float w[kTaps], x[kTaps - 1 + kTok];
+#pragma unroll
+        for (int j = 0; j < kTaps - 1 + kTok; ++j) {
+            const int r = j - (kTaps - 1), p = pos + r;  // row t0 + r at position p
+            const bool row = r < (int)n && r >= -in_seg, kept = r < -in_seg && p >= 0 && -r < (int)a.taps;
+            const float *src = row ? a.proj + (size_t)((int)t0 + r) * a.proj_stride + ch
+                                   : a.conv_state + ((size_t)slot * a.taps + (uint32_t)(kept ? p : 0) % a.taps) * a.channels + ch;
+            x[j] = row || kept ? *src : 0.f;
+        }
+#pragma unroll
+        for (int j = 0; j < kTaps; ++j) w[j] = j < (int)a.taps ? taps[a.taps - 1 - j] : 0.f;   // w[j]: j tokens back
+#pragma unroll
+        for (int t = 0; t < kTok; ++t) {
+            float y = 0.f;
+#pragma unroll
+            for (int j = 0; j < kTaps; ++j) y = fmaf(w[j], x[kTaps - 1 + t - j], y);
+            y = silu_f(y);
+            if (which == 2) {
+                if (t < (int)n) a.qkv[(size_t)(t0 + t) * a.channels + ch] = y;
+            } else {
+                (which == 0 ? qs : ks)[t * pitch + in] = t < (int)n ? y : 0.f;
+            }
+        }
     }
+    for (uint32_t i = threadIdx.x; i < ratio * kTok; i += 256) {
+        const uint32_t h = kvh * ratio + i / kTok, t = i % kTok;
+        float beta = 0.f, g = 1.f;
+        if (t < n) {
+            const float *pr = a.proj + (size_t)(t0 + t) * a.proj_stride;
+            const float z = pr[a.decay_offset + h] + a.dt_bias[h];
+            beta = sigmoid_f(pr[a.beta_offset + h]);
+            g = expf(-expf(a.a_log[h]) * (z > 20.f ? z : log1pf(expf(z))));
+        }
+        gate[2 * i] = beta;
+        gate[2 * i + 1] = g;
+    }
+    __syncthreads();
+    if (warp < (uint32_t)kTok) {   // unit vectors: warp = row
+        float sq = 0.f, sk = 0.f;
+        for (uint32_t d = lane; d < a.dim; d += 32) {
+            sq += qs[warp * pitch + d] * qs[warp * pitch + d];
+            sk += ks[warp * pitch + d] * ks[warp * pitch + d];
+        }
+        for (int off = 16; off > 0; off >>= 1) {
+            sq += __shfl_xor_sync(0xffffffffu, sq, off);
+            sk += __shfl_xor_sync(0xffffffffu, sk, off);
+        }
+        const float iq = 1.0f / sqrtf(sq + a.unit_eps) * (1.0f / sqrtf((float)a.dim));
+        const float ik = 1.0f / sqrtf(sk + a.unit_eps);
+        float *row = a.qkv + (size_t)(t0 + warp) * a.channels + kvh * a.dim;
+        float dot = 0.f;
+        for (uint32_t d = lane; d < a.dim; d += 32) {
+            const float q = qs[warp * pitch + d] * iq, k = ks[warp * pitch + d] * ik;
+            qs[warp * pitch + d] = q;
+            ks[warp * pitch + d] = k;
+            dot += q * k;
+            if (warp < n) {
+                row[d] = q;
+                row[key0 + d] = k;
+            }
+        }
+        if constexpr (kTok == 1) {
+            for (int off = 16; off > 0; off >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, off);
+            for (uint32_t r = lane; r < ratio; r += 32) {
+                float *dst = a.gates + ((size_t)t0 * a.heads + kvh * ratio + r) * 4;
+                dst[0] = gate[2 * r];
+                dst[1] = gate[2 * r + 1];
+                dst[2] = dot;
+            }
+        }
+    }
+    if constexpr (kTok == 1) return;
+    __syncthreads();
+    {   // k_i . k_t and k_i . q_t: two threads per product
+        const uint32_t pair = threadIdx.x / 2, half = threadIdx.x % 2, t = pair / kTok % kTok, i = pair % kTok;
+        const float *x = (pair < kTok * kTok ? ks : qs) + t * pitch, *y = ks + i * pitch;
+        float v = 0.f;
+        for (uint32_t d = half; d < a.dim; d += 2) v = fmaf(x[d], y[d], v);
+        v += __shfl_xor_sync(0xffffffffu, v, 1);
+        if (half == 0 && pair < 2 * kTok * kTok) prod[pair] = v;
+    }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x; i < ratio * kTok; i += 256) {
+        const uint32_t r = i / kTok, t = i % kTok;
+        const float *g = gate + r * kTok * 2;
+        float *dst = a.gates + (((size_t)blockIdx.x * a.heads + kvh * ratio + r) * kTok + t) * kCoef;
+        const float beta = g[2 * t];
+        float decay = 1.f;  // R_ti, from i = t downwards
+        for (int j = kTok - 1; j >= 0; --j) {
+            float kk = 0.f, kq = 0.f;
+            if (j <= (int)t) {
+                if (j < (int)t) {
+                    decay *= g[2 * (j + 1) + 1];
+                    kk = beta * decay * prod[t * kTok + j];
+                }
+                kq = decay * prod[kTok * kTok + t * kTok + j];
+            }
+            dst[j] = kk;
+            dst[kTok + j] = kq;
+        }
+        const float from_start = decay * g[1];  // (R_t0 g_0)
+        float to_end = 1.f;
+        for (uint32_t j = t + 1; j < (uint32_t)kTok; ++j) to_end *= g[2 * j + 1];
+        dst[16] = beta;
+        dst[17] = beta * from_start;
+        dst[18] = from_start;
+        dst[19] = to_end;
+    }
+}
+
+// Values j = 0 .. 31 of every lane -> the sum over the lanes of value `lane`, in each lane.
+__device__ __forceinline__ float scatter_sum(float (&v)[32], uint32_t lane) {
+#pragma unroll
+    for (int half = 16; half > 0; half >>= 1) {
+        const bool up = (lane & half) != 0;
+#pragma unroll
+        for (int j = 0; j < half; ++j) {
+            const float send = up ? v[j] : v[j + half], keep = up ? v[j + half] : v[j];
+            v[j] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+        }
+    }
+    return v[0];
+}
+
+constexpr int kChunkWarps = 4, kChunkCols = 4;  // columns per warp
+template <int kE> struct ChunkShape {
+    static constexpr int kDim = 32 * kE, kStages = kE > 4 ? 3 : 4, kCols = kChunkWarps * kChunkCols;
+    static constexpr int kFloats = 2 * kMini * kDim + kMini * kCols + kMini * kCoef;  // per stage
+    static constexpr size_t kSmem = ((size_t)kStages * kFloats + kChunkWarps * kMini * kChunkCols) * 4;
+};
+// kE: state entries per lane and column (dim <= 32 * kE): entry e of lane l is 128 (e / 4) + 4 l + e % 4
+// (kE = 2: 2 l + e).  A warp owns four columns of one head.
+template <int kE>
+__global__ void __launch_bounds__(kChunkWarps * 32)
+delta_chunk_scan_kernel(DeltaArgs a, uint32_t n_tokens, int vec) {
+    using S = ChunkShape<kE>;
+    constexpr int kPairs = kE / 2, kPiece = kE < 4 ? 2 : 4;
+    qk::pdl_launch();
+    qk::pdl_wait();
+    extern __shared__ __align__(16) float cs_smem[];
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32, h = blockIdx.y;
+    const int pos0 = a.positions[0];
+    if (pos0 < 0) return;
+    const uint32_t slot = (uint32_t)a.slots[0], kvh = h / (a.heads / a.kv_heads), key0 = a.kv_heads * a.dim;
+    const uint32_t col0 = blockIdx.x * S::kCols, n_chunks = (n_tokens + kMini - 1) / kMini;
+    float *us = cs_smem + S::kStages * S::kFloats + warp * kMini * kChunkCols;
+    if (a.dim < (uint32_t)S::kDim) {  // entries past dim stay zero
+        for (uint32_t i = threadIdx.x; i < S::kStages * S::kFloats; i += kChunkWarps * 32) cs_smem[i] = 0.f;
+        __syncthreads();
+    }
+    auto stage = [&](uint32_t chunk) {
+        if (chunk < n_chunks) {
+            float *q = cs_smem + (chunk % S::kStages) * S::kFloats, *k = q + kMini * S::kDim, *v = k + kMini * S::kDim;
+            float *cf = v + kMini * S::kCols;
+            const uint32_t t0 = chunk * kMini;
+            if (vec) {
+                const uint32_t per = a.dim / 4;
+                for (uint32_t i = threadIdx.x; i < kMini * per; i += kChunkWarps * 32) {
+                    const uint32_t t = i / per, d = (i % per) * 4;
+                    const uint32_t bytes = t0 + t < n_tokens ? 16 : 0;
+                    const float *src = a.qkv + (size_t)min(t0 + t, n_tokens - 1) * a.channels + kvh * a.dim + d;
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(
+                                     (uint32_t)__cvta_generic_to_shared(q + t * S::kDim + d)), "l"(src), "r"(bytes) : "memory");
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(
+                                     (uint32_t)__cvta_generic_to_shared(k + t * S::kDim + d)), "l"(src + key0), "r"(bytes) : "memory");
+                }
+            } else {
+                for (uint32_t i = threadIdx.x; i < kMini * a.dim; i += kChunkWarps * 32) {
+                    const uint32_t t = i / a.dim, d = i % a.dim;
+                    const uint32_t bytes = t0 + t < n_tokens ? 4 : 0;
+                    const float *src = a.qkv + (size_t)min(t0 + t, n_tokens - 1) * a.channels + kvh * a.dim + d;
+                    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(
+                                     (uint32_t)__cvta_generic_to_shared(q + t * S::kDim + d)), "l"(src), "r"(bytes) : "memory");
+                    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(
+                                     (uint32_t)__cvta_generic_to_shared(k + t * S::kDim + d)), "l"(src + key0), "r"(bytes) : "memory");
+                }
+            }
+            for (uint32_t i = threadIdx.x; i < kMini * S::kCols; i += kChunkWarps * 32) {
+                const uint32_t t = i / S::kCols, j = i % S::kCols;
+                const uint32_t bytes = t0 + t < n_tokens && col0 + j < a.vdim ? 4 : 0;
+                const float *src = a.qkv + (size_t)min(t0 + t, n_tokens - 1) * a.channels + 2 * key0 + h * a.vdim +
+                                   min(col0 + j, a.vdim - 1);
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(
+                                 (uint32_t)__cvta_generic_to_shared(v + t * S::kCols + j)), "l"(src), "r"(bytes) : "memory");
+            }
+            if (threadIdx.x < kMini * kCoef / 4)
+                copy_async16(cf + threadIdx.x * 4, a.gates + ((size_t)chunk * a.heads + h) * kMini * kCoef + threadIdx.x * 4);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+#pragma unroll
+    for (int i = 0; i < S::kStages - 1; ++i) stage(i);
+
+    f32x2 s[kChunkCols][kPairs];
+    auto entry = [&](int pair) -> uint32_t {  // first entry of a pair
+        return kE < 4 ? 2 * lane : 128 * (pair / 2) + 4 * lane + 2 * (pair % 2);
+    };
+#pragma unroll
+    for (int c = 0; c < kChunkCols; ++c) {
+        const uint32_t col = col0 + warp * kChunkCols + c;
+        const float *st = a.state + (((size_t)slot * a.heads + h) * a.vdim + min(col, a.vdim - 1)) * a.dim;
+#pragma unroll
+        for (int p = 0; p < kPairs; ++p) {
+            const uint32_t d = entry(p);
+            const float x = pos0 != 0 && d < a.dim ? st[d] : 0.f, y = pos0 != 0 && d + 1 < a.dim ? st[d + 1] : 0.f;
+            s[c][p] = pack2(x, y);
+        }
+    }
+    const uint32_t my_t = lane / kChunkCols, my_c = lane % kChunkCols;
+    const uint32_t my_col = col0 + warp * kChunkCols + my_c;
+    for (uint32_t chunk = 0; chunk < n_chunks; ++chunk) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(S::kStages - 2) : "memory");
+        __syncthreads();  // chunk has landed; the stage before it may be filled again
+        stage(chunk + S::kStages - 1);
+        const float *q = cs_smem + (chunk % S::kStages) * S::kFloats, *k = q + kMini * S::kDim, *v = k + kMini * S::kDim;
+        const float *cf = v + kMini * S::kCols + my_t * kCoef;
+        auto piece = [&](const float *row, f32x2 (&x)[kPairs]) {
+#pragma unroll
+            for (int p = 0; p < kE / kPiece; ++p) {
+                if constexpr (kE < 4) {
+                    x[0] = *reinterpret_cast<const f32x2 *>(row + 2 * lane);
+                } else {
+                    const ulonglong2 w = *reinterpret_cast<const ulonglong2 *>(row + 128 * p + 4 * lane);
+                    x[2 * p] = w.x;
+                    x[2 * p + 1] = w.y;
+                }
+            }
+        };
+        auto products = [&](const float *rows) -> float {
+            float part[32];
+#pragma unroll
+            for (int t = 0; t < kMini; ++t) {
+                f32x2 x[kPairs];
+                piece(rows + t * S::kDim, x);
+#pragma unroll
+                for (int c = 0; c < kChunkCols; ++c) {
+                    f32x2 acc = mul2(s[c][0], x[0]);
+#pragma unroll
+                    for (int p = 1; p < kPairs; ++p) acc = fma2(s[c][p], x[p], acc);
+                    float lo, hi;
+                    unpack2(acc, lo, hi);
+                    part[t * kChunkCols + c] = lo + hi;
+                }
+            }
+            return scatter_sum(part, lane);
+        };
+        const float sk = products(k), sq = products(q);
+        // lane (t, c): the triangular solve over the tokens of column c
+        float kk[kMini], kq[kMini];
+#pragma unroll
+        for (int i = 0; i < kMini; i += 4) {
+            const float4 x = *reinterpret_cast<const float4 *>(cf + i), y = *reinterpret_cast<const float4 *>(cf + kMini + i);
+            kk[i] = x.x; kk[i + 1] = x.y; kk[i + 2] = x.z; kk[i + 3] = x.w;
+            kq[i] = y.x; kq[i + 1] = y.y; kq[i + 2] = y.z; kq[i + 3] = y.w;
+        }
+        const float4 g = *reinterpret_cast<const float4 *>(cf + 16);  // beta, beta P, P, R_8
+        float u = g.x * v[my_t * S::kCols + warp * kChunkCols + my_c] - g.y * sk, o = g.z * sq;
+#pragma unroll
+        for (int i = 0; i < kMini; ++i) {
+            const float ui = __shfl_sync(0xffffffffu, u, i * kChunkCols + my_c);
+            u = fmaf(-kk[i], ui, u);
+            o = fmaf(kq[i], ui, o);
+        }
+        const uint32_t t = chunk * kMini + my_t;
+        if (t < n_tokens && my_col < a.vdim) a.out[(size_t)t * a.out_stride + h * a.vdim + my_col] = o;
+        const float p8 = __shfl_sync(0xffffffffu, g.z, 31);  // P of the last token
+        us[lane] = u * g.w;
+        __syncwarp();
+        const f32x2 p2 = pack2(p8, p8);
+#pragma unroll
+        for (int c = 0; c < kChunkCols; ++c)
+#pragma unroll
+            for (int p = 0; p < kPairs; ++p) s[c][p] = mul2(p2, s[c][p]);
+#pragma unroll
+        for (int i = 0; i < kMini; ++i) {
+            const float4 w = *reinterpret_cast<const float4 *>(us + i * kChunkCols);
+            const float uw[4] = {w.x, w.y, w.z, w.w};
+            f32x2 x[kPairs];
+            piece(k + i * S::kDim, x);
+#pragma unroll
+            for (int c = 0; c < kChunkCols; ++c) {
+                const f32x2 u2 = pack2(uw[c], uw[c]);
+#pragma unroll
+                for (int p = 0; p < kPairs; ++p) s[c][p] = fma2(x[p], u2, s[c][p]);
+            }
+        }
+        __syncwarp();
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int c = 0; c < kChunkCols; ++c) {
+        const uint32_t col = col0 + warp * kChunkCols + c;
+        if (col >= a.vdim) break;
+        float *st = a.state + (((size_t)slot * a.heads + h) * a.vdim + col) * a.dim;
+#pragma unroll
+        for (int p = 0; p < kPairs; ++p) {
+            const uint32_t d = entry(p);
+            float x, y;
+            unpack2(s[c][p], x, y);
+            if (d < a.dim) st[d] = x;
+            if (d + 1 < a.dim) st[d + 1] = y;
+        }
+    }
+    keep_conv_inputs(a, slot, pos0, 0, n_tokens, kChunkWarps * 32);
+}
+
+template <int kE>
+qk_status launch_chunk_scan(qk_ctx *c, const DeltaArgs &a, size_t tokens, int vec) {
+    using S = ChunkShape<kE>;
+    QK_CUDA(cudaFuncSetAttribute(delta_chunk_scan_kernel<kE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
+    (void)qk::launch_pdl(c->pdl, delta_chunk_scan_kernel<kE>, dim3((a.vdim + S::kCols - 1) / S::kCols, a.heads),
+                         dim3(kChunkWarps * 32), S::kSmem, c->stream, a, (uint32_t)tokens, vec);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    return QK_OK;
 }
 
 qk_status enter(qk_ctx *ctx, qk_ctx **c) {
@@ -356,6 +634,7 @@ qk_status qk_delta(qk_ctx *ctx, const qk_delta_call *d) {
     if (d->kv_heads == 0 || d->heads % d->kv_heads || d->dim == 0 || d->vdim == 0 || d->taps == 0)
         return qk::fail(QK_ERR_VALUE, "qk_delta: %zu heads over %zu key heads, dim %zu, vdim %zu, %zu taps", d->heads,
                         d->kv_heads, d->dim, d->vdim, d->taps);
+    if (d->taps > 16) return qk::fail(QK_ERR_VALUE, "qk_delta: more than 16 taps are not supported, got %zu", d->taps);
     if (d->dim > 512) return qk::fail(QK_ERR_VALUE, "qk_delta: dim above 512 is not supported, got %zu", d->dim);
     if (d->tokens == 0) return QK_OK;
     DeltaArgs a{};
@@ -386,15 +665,36 @@ qk_status qk_delta(qk_ctx *ctx, const qk_delta_call *d) {
     a.decay_offset = (uint32_t)d->decay_offset;
     a.out_stride = (uint32_t)d->out_stride;
     a.unit_eps = d->unit_eps;
-    // few rows: a block per key head and row; many rows: a block for a few key heads
-    const size_t parts = d->tokens <= 64 ? d->kv_heads : qk::ceil_div(d->kv_heads, 8);
-    (void)qk::launch_pdl(c->pdl, delta_inputs_kernel, dim3((unsigned)d->tokens, (unsigned)parts), dim3(kPrepThreads),
-                         d->kv_heads * sizeof(float), c->stream, a);
-    QK_CUDA(cudaGetLastError());
-    c->launches++;
-    const dim3 grid((unsigned)qk::ceil_div(d->vdim, kScanCols), (unsigned)d->heads, (unsigned)d->segments);
     const int vec = d->dim % 4 == 0 && a.channels % 4 == 0 && ((uintptr_t)d->qkv & 15) == 0 &&
                     ((uintptr_t)d->state & 15) == 0;
+    const bool portion = d->segments == 1 && d->tokens >= (size_t)kMini;  // eight tokens at a time
+    const size_t tok = portion ? kMini : 1;
+    const dim3 ig((unsigned)qk::ceil_div(d->tokens, tok), a.kv_heads);
+    const size_t smem = (2 * tok * (d->dim + 1) + 2 * tok * tok + d->heads / d->kv_heads * tok * 2) * 4;
+    if (smem > 200 * 1024) return qk::fail(QK_ERR_VALUE, "qk_delta: %zu heads over %zu key heads", d->heads, d->kv_heads);
+#define QK_INPUTS(taps, tok)                                                                                    \
+    do {                                                                                                        \
+        QK_CUDA(cudaFuncSetAttribute(delta_inputs_kernel<taps, tok>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+                                     (int)std::max(smem, (size_t)48 * 1024)));                                  \
+        (void)qk::launch_pdl(c->pdl, delta_inputs_kernel<taps, tok>, ig, dim3(256), smem, c->stream, a,         \
+                             (uint32_t)d->tokens);                                                              \
+    } while (0)
+    if (portion) {
+        if (d->taps <= 4) QK_INPUTS(4, kMini);
+        else QK_INPUTS(16, kMini);
+    } else {
+        if (d->taps <= 4) QK_INPUTS(4, 1);
+        else QK_INPUTS(16, 1);
+    }
+#undef QK_INPUTS
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    if (portion)
+        return d->dim <= 64 ? launch_chunk_scan<2>(c, a, d->tokens, vec)
+               : d->dim <= 128 ? launch_chunk_scan<4>(c, a, d->tokens, vec)
+               : d->dim <= 256 ? launch_chunk_scan<8>(c, a, d->tokens, vec)
+                               : launch_chunk_scan<16>(c, a, d->tokens, vec);
+    const dim3 grid((unsigned)qk::ceil_div(d->vdim, kScanCols), (unsigned)d->heads, (unsigned)d->segments);
 #define QK_SCAN(per) \
     (void)qk::launch_pdl(c->pdl, delta_scan_kernel<per>, grid, dim3(kScanThreads), 0, c->stream, a, vec)
     if (d->dim <= 32) QK_SCAN(4);

@@ -1,9 +1,10 @@
 // Dense linears y = W x with bfloat16 or float32 weights, in four forms:
 //   * vector (up to kVectorTokens rows): one launch; every block forms the input vectors itself
 //     (norm, pending residual, gate - see qk_dense_dev.cuh) and its warps stream weight rows;
-//   * skinny (bfloat16, up to kSkinnyTokens rows): mma.sync, the weights on the M side and read
-//     once, straight from global memory into fragments, the rows on the N side;
-//   * tcgen05 (bfloat16, more rows): TMA-fed tcgen05.mma with the accumulators in tensor memory;
+//   * narrow (bfloat16, up to kNarrowTokens rows): tcgen05.mma with the weights on the M side, each
+//     byte of them read once, the k range shared out over a cluster;
+//   * tcgen05 (bfloat16, more rows): persistent TMA-fed tcgen05.mma with two accumulators in
+//     tensor memory;
 //   * float32 (more rows, float32 weights): plain float32 multiply-adds, no reduced-precision
 //     matrix mode.
 // The matrix forms take their input rows from a kernel that runs the same device function as
@@ -19,7 +20,7 @@ namespace {
 
 constexpr int kVecThreads = 256, kVecWarps = kVecThreads / 32;
 constexpr int kVectorTokens = 4;
-constexpr int kSkinnyTokens = 64;
+constexpr int kNarrowTokens = 128;
 constexpr size_t kVecSmemMax = 200 * 1024;
 
 // ------------------------------------------------------------------ vector form
@@ -214,148 +215,6 @@ dense_input_kernel(InputArgs in, A *__restrict__ dst) {
     if (in.append.src) append_latent(in, t, red);
 }
 
-// ------------------------------------------------------------------ skinny form
-__device__ __forceinline__ void sk_mma(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3,
-                                       uint32_t b0, uint32_t b1) {
-    asm volatile(
-        "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, "
-        "{%0,%1,%2,%3};"
-        : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-        : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void sk_copy16(void *smem, const void *gmem, uint32_t bytes) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)),
-                 "l"(gmem), "r"(bytes)
-                 : "memory");
-}
-constexpr int kSkWarps = 8, kSkPitch = 96;  // bf16 entries per staged row: 64 k + 32 pad
-
-// A warp owns two tiles of 16 weight rows (32 consecutive rows, or 16 gate rows and their up
-// rows) and every ksplit-th chunk of 64 k; the staged x chunks of all ksplit parts are shared by
-// the block.  k order inside a 32-wide group as in the LM head's kernel: one 16-byte load feeds
-// two MMAs on either operand.
-template <int NT>
-__global__ void __launch_bounds__(kSkWarps * 32)
-dense_skinny_kernel(const uint16_t *__restrict__ x, uint32_t x_stride, uint32_t k,
-                    const uint16_t *__restrict__ w, uint32_t rows, uint32_t w_stride, uint32_t n_tokens,
-                    uint32_t ksplit, OutputArgs out) {
-    qk::pdl_launch();
-    extern __shared__ __align__(16) uint8_t sk_smem[];
-    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane >> 2, t = lane & 3;
-    const uint32_t part = warp % ksplit, tile = (blockIdx.x * kSkWarps + warp) / ksplit;
-    const bool pair = out.kind == QK_OUTPUT_GLU;
-    uint32_t first[2];
-    if (pair) {
-        first[0] = pair_row(tile * 16);
-        first[1] = first[0] + 32;
-    } else {
-        first[0] = tile * 32;
-        first[1] = first[0] + 16;
-    }
-    const uint16_t *row[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i)
-        row[i] = w + (size_t)min(first[i / 2] + g + (i % 2) * 8, rows - 1) * w_stride + 8 * t;
-    const uint32_t chunks = (k + 63) / 64, rounds = (chunks + ksplit - 1) / ksplit;
-    auto fetch = [&](uint32_t round, uint4 (&dst)[4][2]) {
-        const uint32_t c = round * ksplit + part;
-#pragma unroll
-        for (int gi = 0; gi < 2; ++gi) {
-            const uint32_t col = c * 64 + gi * 32;
-            const bool live = c < chunks && col + 8 * t < k;
-#pragma unroll
-            for (int i = 0; i < 4; ++i) dst[i][gi] = live ? load_weights16(row[i] + col) : make_uint4(0, 0, 0, 0);
-        }
-    };
-    const uint32_t buf_elems = ksplit * 8 * NT * kSkPitch;
-    uint16_t *stage_base = reinterpret_cast<uint16_t *>(sk_smem);
-    auto stage = [&](uint32_t round, uint32_t buf) {
-        for (uint32_t idx = threadIdx.x; idx < ksplit * 8 * NT * 8; idx += kSkWarps * 32) {
-            const uint32_t piece = idx % 8, tok = (idx / 8) % (8 * NT), p = idx / (8 * 8 * NT);
-            const uint32_t col = (round * ksplit + p) * 64 + piece * 8;
-            const bool live = tok < n_tokens && col < k;
-            sk_copy16(stage_base + buf * buf_elems + (p * 8 * NT + tok) * kSkPitch + piece * 8,
-                      x + (live ? (size_t)tok * x_stride + col : 0), live ? 16u : 0u);
-        }
-        asm volatile("cp.async.commit_group;" ::: "memory");
-    };
-    float acc[2][NT][4];
-#pragma unroll
-    for (int m = 0; m < 2; ++m)
-#pragma unroll
-        for (int nt = 0; nt < NT; ++nt) acc[m][nt][0] = acc[m][nt][1] = acc[m][nt][2] = acc[m][nt][3] = 0.f;
-    uint4 nxt[4][2];
-    fetch(0, nxt);
-    qk::pdl_wait();
-    stage(0, 0);
-    for (uint32_t c = 0; c < rounds; ++c) {
-        uint4 cur[4][2];
-#pragma unroll
-        for (int i = 0; i < 4; ++i) cur[i][0] = nxt[i][0], cur[i][1] = nxt[i][1];
-        fetch(c + 1, nxt);
-        if (c + 1 < rounds) {
-            stage(c + 1, (c + 1) & 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();
-        const uint16_t *xb = stage_base + (c & 1) * buf_elems + part * 8 * NT * kSkPitch;
-#pragma unroll
-        for (int gi = 0; gi < 2; ++gi)
-#pragma unroll
-            for (int nt = 0; nt < NT; ++nt) {
-                const uint4 b = *reinterpret_cast<const uint4 *>(xb + (8 * nt + g) * kSkPitch + gi * 32 + 8 * t);
-#pragma unroll
-                for (int m = 0; m < 2; ++m) {
-                    const uint4 lo = cur[2 * m][gi], hi = cur[2 * m + 1][gi];
-                    sk_mma(acc[m][nt], lo.x, hi.x, lo.y, hi.y, b.x, b.y);
-                    sk_mma(acc[m][nt], lo.z, hi.z, lo.w, hi.w, b.z, b.w);
-                }
-            }
-        __syncthreads();
-    }
-    if (ksplit > 1) {
-        // the parts' sums, part 0 first: [warp][value][lane]
-        float *sums = reinterpret_cast<float *>(sk_smem);
-        constexpr int kVals = 2 * NT * 4;
-        if (part != 0) {
-#pragma unroll
-            for (int m = 0; m < 2; ++m)
-#pragma unroll
-                for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-                    for (int e = 0; e < 4; ++e)
-                        sums[((size_t)warp * kVals + (m * NT + nt) * 4 + e) * 32 + lane] = acc[m][nt][e];
-        }
-        __syncthreads();
-        if (part == 0) {
-            for (uint32_t p = 1; p < ksplit; ++p)
-#pragma unroll
-                for (int m = 0; m < 2; ++m)
-#pragma unroll
-                    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-                        for (int e = 0; e < 4; ++e)
-                            acc[m][nt][e] += sums[((size_t)(warp + p) * kVals + (m * NT + nt) * 4 + e) * 32 + lane];
-        }
-    }
-    if (part != 0) return;
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const uint32_t tok = 8 * nt + 2 * t + (e & 1), r = g + (e >> 1) * 8;
-            if (tok >= n_tokens) continue;
-            if (pair) {
-                if (tile * 16 + r < rows / 2) finish_pair(out, tok, tile * 16 + r, acc[0][nt][e], acc[1][nt][e]);
-            } else {
-                if (first[0] + r < rows) finish(out, tok, first[0] + r, acc[0][nt][e]);
-                if (first[1] + r < rows) finish(out, tok, first[1] + r, acc[1][nt][e]);
-            }
-        }
-}
-
 // ------------------------------------------------------------------ float32 form
 constexpr int kFTile = 64, kFK = 16;
 __global__ void __launch_bounds__(256)
@@ -444,6 +303,17 @@ __device__ __forceinline__ bool tc_epilogue_vote(bool ok) {
         : "r"((uint32_t)ok), "r"(kTcEpiWarps * 32)
         : "memory");
     return all != 0;
+}
+
+// 16 consecutive 32-bit columns of this thread's tensor-memory lane.
+__device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
+    asm volatile(
+        "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+        "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+        : "=r"(v[0]), "=r"(v[1]), "=r"(v[2]), "=r"(v[3]), "=r"(v[4]), "=r"(v[5]), "=r"(v[6]), "=r"(v[7]),
+          "=r"(v[8]), "=r"(v[9]), "=r"(v[10]), "=r"(v[11]), "=r"(v[12]), "=r"(v[13]), "=r"(v[14]), "=r"(v[15])
+        : "r"(taddr)
+        : "memory");
 }
 
 // Thirty-two consecutive outputs n0 .. of token t.  `vec`: rows are 16-byte aligned.
@@ -664,6 +534,247 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     if (threadIdx.x == 0 && *abort_flag) atomicOr(g.error, 1);
 }
 
+// ------------------------------------------------------------------ narrow form
+// Few rows of x (a decode batch): the weights take the M side (128 weight rows per CTA), the rows of
+// x the N side, so that a weight byte is read once and the product is bound by reading it.  The k
+// range of a tile is shared out over the CTAs of a cluster (up to eight), which then add their
+// float32 accumulators through distributed shared memory, each CTA finishing its share of the
+// columns.  Weights depend on no other kernel: the first stages' copies start before the
+// dependency wait.  Warp 0 issues the copies, warp 1 the MMAs, warps 2..5 finish.
+template <int BN> struct NarrowShape {
+    static constexpr uint32_t kABytes = 128 * kTcK * 2, kBBytes = BN * kTcK * 2, kStage = kABytes + kBBytes;
+    static constexpr int kStages = BN >= 128 ? 6 : 8;
+    static constexpr uint32_t kTmemCols = BN < 32 ? 32 : BN;
+    static constexpr size_t kSmem = 1024 + kStages * kStage + (2 * kStages + 2) * 8 + 32;
+    static_assert(128 * BN * 4 + 2 * 32 * BN * 4 <= kStages * kStage, "the accumulators must fit the drained stages");
+};
+struct NarrowArgs {
+    uint32_t n_tokens, rows, k_chunks, splits, wait_limit;
+    int *error;
+};
+__device__ __forceinline__ void cluster_sync_all() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+
+template <int BN>
+__global__ void __launch_bounds__(kTcThreads, 1)
+dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map,
+                    NarrowArgs g, OutputArgs out) {
+    using S = NarrowShape<BN>;
+    qk::pdl_launch();
+    extern __shared__ __align__(1024) uint8_t nr_smem[];
+    uint8_t *tiles = reinterpret_cast<uint8_t *>(((uintptr_t)nr_smem + 1023) & ~(uintptr_t)1023);
+    uint64_t *full = reinterpret_cast<uint64_t *>(tiles + S::kStages * S::kStage);
+    uint64_t *empty = full + S::kStages;
+    uint64_t *acc_full = empty + S::kStages;
+    uint64_t *drain = acc_full + 1;
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(drain + 1);
+    volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+    volatile int *never = reinterpret_cast<volatile int *>(tmem_slot + 2);
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const uint32_t tile = blockIdx.x / g.splits, split = blockIdx.x % g.splits;  // (a cluster is one tile)
+    const uint32_t per = (g.k_chunks + g.splits - 1) / g.splits;
+    const uint32_t kc0 = min(split * per, g.k_chunks), kc1 = min(kc0 + per, g.k_chunks);
+    if (threadIdx.x == 0) {
+        for (int s = 0; s < S::kStages; ++s) {
+            mbar_init(&full[s], 1);
+            mbar_init(&empty[s], 1);
+        }
+        mbar_init(acc_full, 1);
+        mbar_init(drain, 1);
+        *abort_flag = 0;
+        *never = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)),
+                     "r"(S::kTmemCols)
+                     : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t ahead = min((uint32_t)S::kStages, kc1 - kc0);
+    if (warp == 0 && lane == 0)
+        for (uint32_t i = 0; i < ahead; ++i) {
+            asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(&full[i])),
+                         "r"(S::kStage)
+                         : "memory");
+            tma_load_2d(smem_u32(tiles + i * S::kStage), &w_map, (kc0 + i) * kTcK, tile * 128, &full[i]);
+        }
+    qk::pdl_wait();
+    const uint32_t tmem_base = *tmem_slot;
+    bool finished = true;  // (epilogue warps: the accumulator is complete)
+
+    if (warp == 0) {
+        uint32_t gc = 0;
+        bool dead = false;
+        for (uint32_t kc = kc0; kc < kc1; ++kc, ++gc) {
+            const uint32_t s = gc % S::kStages;
+            if (gc >= ahead && !mbar_wait(&empty[s], ((gc / S::kStages) & 1) ^ 1, abort_flag, g.wait_limit)) {
+                dead = true;
+                break;
+            }
+            if (lane == 0) {
+                const uint32_t a = smem_u32(tiles + s * S::kStage);
+                if (gc >= ahead) {
+                    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(&full[s])),
+                                 "r"(S::kStage)
+                                 : "memory");
+                    tma_load_2d(a, &w_map, kc * kTcK, tile * 128, &full[s]);
+                }
+                tma_load_2d(a + S::kABytes, &x_map, kc * kTcK, 0, &full[s]);
+            }
+            __syncwarp();
+        }
+        if (dead) *abort_flag = 1;
+        if (*abort_flag)  // the copies still in flight
+            for (uint32_t i = gc > (uint32_t)S::kStages ? gc - S::kStages : 0; i < gc; ++i)
+                (void)mbar_wait(&full[i % S::kStages], (i / S::kStages) & 1, never, g.wait_limit);
+    } else if (warp == 1) {
+        const uint32_t idesc = tc_idesc(BN);
+        uint32_t gc = 0;
+        bool dead = false;
+        for (uint32_t kc = kc0; kc < kc1; ++kc, ++gc) {
+            const uint32_t s = gc % S::kStages;
+            if (!mbar_wait(&full[s], (gc / S::kStages) & 1, abort_flag, g.wait_limit)) {
+                dead = true;
+                break;
+            }
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (lane == 0) {
+                const uint32_t a_addr = smem_u32(tiles + s * S::kStage), b_addr = a_addr + S::kABytes;
+#pragma unroll
+                for (int k = 0; k < kTcK / 16; ++k) {
+                    const uint64_t ad = umma_desc(a_addr + k * 32), bd = umma_desc(b_addr + k * 32);
+                    const uint32_t accumulate = (gc != 0 || k != 0) ? 1u : 0u;
+                    asm volatile(
+                        "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
+                        " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}" ::"r"(tmem_base),
+                        "l"(ad), "l"(bd), "r"(idesc), "r"(accumulate)
+                        : "memory");
+                }
+                umma_commit(&empty[s]);
+            }
+            __syncwarp();
+        }
+        if (!dead && lane == 0) umma_commit(acc_full);
+        __syncwarp();
+        if (dead) {
+            *abort_flag = 1;
+            if (lane == 0) umma_commit(drain);  // the products still in flight
+            __syncwarp();
+            (void)mbar_wait(drain, 0, never, g.wait_limit);
+        }
+    } else {
+        finished = tc_epilogue_vote(mbar_wait(acc_full, 0, abort_flag, g.wait_limit));
+        if (!finished) *abort_flag = 1;
+    }
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t quarter = warp % 4, row = quarter * 32 + lane;
+    float *own = reinterpret_cast<float *>(tiles);  // [BN][128]: the drained stages
+    if (g.splits > 1) {
+        if (warp >= 2 && finished) {
+            const uint32_t lane_addr = tmem_base + ((quarter * 32) << 16);
+#pragma unroll
+            for (int c0 = 0; c0 < BN; c0 += 16) {
+                uint32_t v[16];
+                tmem_ld16(lane_addr + c0, v);
+                tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 16; ++j)
+                    own[(c0 + j) * 128 + row] = kc1 > kc0 ? __uint_as_float(v[j]) : 0.f;
+            }
+        }
+        __syncwarp();
+        cluster_sync_all();  // every CTA of the tile has its accumulator in shared memory
+    }
+    if (warp >= 2 && finished) {
+        const bool pair = out.kind == QK_OUTPUT_GLU;
+        const uint32_t share = (BN + g.splits - 1) / g.splits;  // columns this CTA finishes
+        const uint32_t c_begin = split * share, c_end = min(min(c_begin + share, (uint32_t)BN), g.n_tokens);
+        float *ups = own + 128 * BN;  // [2][BN][32]: up rows for their gate rows
+        const uint32_t n = tile * 128 + row, lane_addr = tmem_base + ((quarter * 32) << 16);
+        auto value = [&](uint32_t c) -> float {  // (splits > 1) the sum over the cluster, in split order
+            float v = 0.f;
+            for (uint32_t p = 0; p < g.splits; ++p) {
+                uint32_t remote;
+                float x;
+                asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(smem_u32(own + c * 128 + row)), "r"(p));
+                asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(x) : "r"(remote) : "memory");
+                v += x;
+            }
+            return v;
+        };
+        auto done = [&](uint32_t c, float v) {
+            if (pair) {
+                if (quarter & 1) ups[((quarter >> 1) * BN + c) * 32 + lane] = v;
+            } else if (n < g.rows) {
+                finish(out, c, n, v);
+            }
+        };
+        float kept[BN <= 64 ? BN : 1];  // a gate row's values until its up row's arrive
+        if (g.splits == 1) {
+#pragma unroll
+            for (int c0 = 0; c0 < BN; c0 += 16) {
+                if ((uint32_t)c0 >= c_end) break;
+                uint32_t v[16];
+                tmem_ld16(lane_addr + c0, v);
+                tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 16; ++j) {
+                    if constexpr (BN <= 64) kept[c0 + j] = __uint_as_float(v[j]);
+                    if ((uint32_t)(c0 + j) < c_end) done(c0 + j, __uint_as_float(v[j]));
+                }
+            }
+        } else if (!pair) {
+#pragma unroll 4
+            for (uint32_t c = c_begin; c < c_end; ++c) done(c, value(c));
+        } else if (quarter & 1) {
+#pragma unroll 4
+            for (uint32_t c = c_begin; c < c_end; ++c) done(c, value(c));
+        }
+        if (pair) {
+            asm volatile("bar.sync 1, %0;" ::"r"(kTcEpiWarps * 32) : "memory");
+            const uint32_t j = tile * 64 + (quarter >> 1) * 32 + lane;
+            if (!(quarter & 1) && j < g.rows / 2) {
+                if (g.splits == 1) {
+#pragma unroll
+                    for (int c0 = 0; c0 < BN; c0 += 16) {
+                        if ((uint32_t)c0 >= c_end) break;
+                        uint32_t v[16];
+                        if constexpr (BN > 64) {
+                            tmem_ld16(lane_addr + c0, v);
+                            tmem_ld_wait();
+                        }
+#pragma unroll
+                        for (int e = 0; e < 16; ++e) {
+                            const uint32_t c = c0 + e;
+                            float gate;
+                            if constexpr (BN > 64) gate = __uint_as_float(v[e]);
+                            else gate = kept[c0 + e];
+                            if (c < c_end) finish_pair(out, c, j, gate, ups[((quarter >> 1) * BN + c) * 32 + lane]);
+                        }
+                    }
+                } else {
+#pragma unroll 4
+                    for (uint32_t c = c_begin; c < c_end; ++c)
+                        finish_pair(out, c, j, value(c), ups[((quarter >> 1) * BN + c) * 32 + lane]);
+                }
+            }
+        }
+    }
+    __syncwarp();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    if (g.splits > 1) cluster_sync_all();  // no CTA leaves while another still reads its shared memory
+    else __syncthreads();
+    if (warp == 1)
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(S::kTmemCols)
+                     : "memory");
+    if (threadIdx.x == 0 && *abort_flag) atomicOr(g.error, 1);
+}
+
 typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
                                   const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
                                   CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
@@ -727,22 +838,53 @@ qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_ca
     return QK_OK;
 }
 
-template <int NT>
-qk_status launch_skinny(qk_ctx *c, const uint16_t *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out) {
-    const bool pair = d.output == QK_OUTPUT_GLU;
-    const size_t tiles = pair ? qk::ceil_div(d.rows / 2, 16) : qk::ceil_div(d.rows, 32);
-    const size_t chunks = qk::ceil_div(d.k, 64);
-    uint32_t ks = 1;  // warps that share out a row tile's k range: enough blocks to fill the SMs
-    while (ks < kSkWarps && qk::ceil_div(tiles * ks, kSkWarps) < (size_t)c->sm_count && ks * 2 <= chunks) ks *= 2;
-    const size_t stage = 2 * (size_t)ks * 8 * NT * kSkPitch * 2;
-    const size_t sums = (size_t)kSkWarps * 2 * NT * 4 * 32 * 4;
-    const size_t smem = std::max(stage, ks > 1 ? sums : (size_t)0);
-    QK_CUDA(cudaFuncSetAttribute(dense_skinny_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    (void)qk::launch_pdl(c->pdl, dense_skinny_kernel<NT>, dim3((unsigned)qk::ceil_div(tiles * ks, kSkWarps)),
-                         dim3(kSkWarps * 32), smem, c->stream, x, (uint32_t)x_stride, (uint32_t)d.k,
-                         (const uint16_t *)d.w, (uint32_t)d.rows, (uint32_t)d.w_stride, (uint32_t)d.tokens, ks, out);
-    QK_CUDA(cudaGetLastError());
+// CTAs per tile: enough to occupy the SMs without splitting the k range finer than four chunks.
+uint32_t narrow_splits(size_t tiles, size_t k_chunks, size_t sms) {
+    uint32_t best = 1;
+    size_t best_cost = ~(size_t)0;
+    for (uint32_t s : {1u, 2u, 4u, 8u}) {
+        if (s > 1 && k_chunks / s < 4) break;
+        // (a cluster of CTAs does not find room on every SM)
+        const size_t room = s == 1 ? sms : s == 2 ? sms - 4 : sms - 20;
+        const size_t waves = qk::ceil_div(tiles * s, room);
+        const size_t cost = waves * (qk::ceil_div(k_chunks, s) + 10) + (s > 1 ? 6 : 0);
+        if (cost < best_cost) best = s, best_cost = cost;
+    }
+    return best;
+}
+
+template <int BN>
+qk_status launch_narrow(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out) {
+    using S = NarrowShape<BN>;
+    CUtensorMap xm, wm;
+    qk_status st;
+    if ((st = encode_map(x, d.tokens, d.k, x_stride, BN, &xm)) != QK_OK) return st;
+    if ((st = encode_map(d.w, d.rows, d.k, d.w_stride, 128, &wm)) != QK_OK) return st;
+    NarrowArgs g{};
+    g.n_tokens = (uint32_t)d.tokens;
+    g.rows = (uint32_t)d.rows;
+    g.k_chunks = (uint32_t)qk::ceil_div(d.k, kTcK);
+    const uint32_t tiles = (uint32_t)qk::ceil_div(d.rows, 128);
+    g.splits = narrow_splits(tiles, g.k_chunks, (size_t)c->sm_count);
+    g.wait_limit = c->wait_limit ? c->wait_limit : kTcWaitDefault;
+    g.error = (int *)c->d_err.ptr;
+    QK_CUDA(cudaFuncSetAttribute(dense_narrow_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(tiles * g.splits);
+    cfg.blockDim = dim3(kTcThreads);
+    cfg.dynamicSmemBytes = S::kSmem;
+    cfg.stream = c->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = c->pdl ? 1 : 0;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = g.splits;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    QK_CUDA(cudaLaunchKernelEx(&cfg, dense_narrow_kernel<BN>, wm, xm, g, out));
     c->launches++;
+    c->err_armed = true;
     return QK_OK;
 }
 
@@ -898,7 +1040,7 @@ extern "C" {
 int32_t qk_dense_form(size_t tokens, size_t k, int32_t w_dtype) {
     if (tokens <= (size_t)kVectorTokens && k * 4 <= kVecSmemMax) return QK_FORM_VECTOR;
     if (w_dtype == QK_F32) return QK_FORM_F32;
-    return tokens <= (size_t)kSkinnyTokens ? QK_FORM_SKINNY : QK_FORM_TCGEN05;
+    return tokens <= (size_t)kNarrowTokens ? QK_FORM_NARROW : QK_FORM_TCGEN05;
 }
 
 qk_status qk_dense_input(qk_ctx *ctx, const qk_dense_call *d) {
@@ -974,14 +1116,13 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
         c->launches++;
         return QK_OK;
     }
-    if (d->tokens <= (size_t)kSkinnyTokens) {
-        const uint16_t *x = (const uint16_t *)rows;
-        if (d->tokens <= 8) return launch_skinny<1>(c, x, stride, *d, out);
-        if (d->tokens <= 16) return launch_skinny<2>(c, x, stride, *d, out);
-        if (d->tokens <= 32) return launch_skinny<4>(c, x, stride, *d, out);
-        return launch_skinny<8>(c, x, stride, *d, out);
-    }
     if ((st = qk::error_word(c)) != QK_OK) return st;
+    if (d->tokens <= (size_t)kNarrowTokens) {
+        if (d->tokens <= 16) return launch_narrow<16>(c, rows, stride, *d, out);
+        if (d->tokens <= 32) return launch_narrow<32>(c, rows, stride, *d, out);
+        if (d->tokens <= 64) return launch_narrow<64>(c, rows, stride, *d, out);
+        return launch_narrow<128>(c, rows, stride, *d, out);
+    }
     const int per16 = d->out_dtype == QK_BF16 ? 8 : 4;
     const int vec = (!d->out || (((uintptr_t)d->out & 15) == 0 && d->out_stride % per16 == 0)) &&
                     (!d->residual || (((uintptr_t)d->residual & 15) == 0 && d->residual_stride % 4 == 0)) &&

@@ -186,6 +186,28 @@ latent_plain_kernel(LatentArgs a, const C *__restrict__ cache) {
 // 32 keys at a time.  Scores: each warp multiplies eight keys over all latent channels; sums: each
 // warp owns a quarter of the channels.  KV: staged channels per key (kv_stride <= KV).
 constexpr int kLatKeys = 32;
+__device__ __forceinline__ void lat_cluster_sync() {
+    __syncwarp();
+    asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+__device__ __forceinline__ uint32_t lat_map(const float *p, uint32_t cta) {
+    uint32_t r;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"((uint32_t)__cvta_generic_to_shared(p)), "r"(cta));
+    return r;
+}
+__device__ __forceinline__ float lat_peer(const float *p, uint32_t cta) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(lat_map(p, cta)) : "memory");
+    return v;
+}
+__device__ __forceinline__ float4 lat_peer4(const float *p, uint32_t cta) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0, %1, %2, %3}, [%4];"
+                 : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w)
+                 : "r"(lat_map(p, cta))
+                 : "memory");
+    return v;
+}
 template <int KV> struct LatShape {
     static constexpr int kPitch = KV + 8;
     static constexpr size_t kQBytes = 2 * 16 * kPitch * 2, kTileBytes = kLatKeys * kPitch * 2;
@@ -193,7 +215,7 @@ template <int KV> struct LatShape {
 };
 template <int KV>
 __global__ void __launch_bounds__(128)
-latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache) {
+latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t cluster) {
     using S = LatShape<KV>;
     constexpr int kTilesPerWarp = KV / 4 / 8;  // 8-channel tiles of the sums per warp
     qk::pdl_launch();
@@ -223,6 +245,7 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (keys.count) fetch(0, 0);
+#pragma unroll 8
     for (uint32_t i = threadIdx.x; i < 16 * (KV / 2); i += 128) {
         const uint32_t r = i / (KV / 2), c = (i % (KV / 2)) * 2;
         float x = 0.f, y = 0.f;
@@ -326,26 +349,59 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache) {
         }
         __syncthreads();  // the buffers may be filled again
     }
+    // The splits of a cluster are merged here: every CTA leaves its sums, maxima and weights in its
+    // shared memory (the tiles are idle) and each finishes a share of the channels.
+    float *sums = reinterpret_cast<float *>(lat_smem);  // [16][KV + 4]
+    constexpr int kSumPitch = KV + 4;
+    float *stat = sums + 16 * kSumPitch;                // [2][16]: maximum, weight
+    static_assert((16 * kSumPitch + 32) * 4 <= S::kQBytes + 2 * S::kTileBytes, "the sums must fit the tiles");
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
-        const uint32_t h = h0 + g + 8 * r;
-        if (h >= a.heads) continue;
-        float *dst = a.partial + (((size_t)t * a.heads + h) * a.n_splits + split) * (a.kv_stride + 8);
-        if (keys.count) {
 #pragma unroll
-            for (int n = 0; n < kTilesPerWarp; ++n) {
-                const uint32_t c = warp * (KV / 4) + n * 8 + 2 * c4;
-                if (c < a.kv_stride)
-                    *reinterpret_cast<float2 *>(dst + c) = make_float2(o[n][2 * r], o[n][2 * r + 1]);
-            }
-        }
+        for (int n = 0; n < kTilesPerWarp; ++n)
+            *reinterpret_cast<float2 *>(sums + (g + 8 * r) * kSumPitch + warp * (KV / 4) + n * 8 + 2 * c4) =
+                make_float2(o[n][2 * r], o[n][2 * r + 1]);
         if (warp == 0 && c4 == 0) {
-            dst[a.kv_stride] = m[r];
-            dst[a.kv_stride + 1] = l[r];
+            stat[g + 8 * r] = m[r];
+            stat[16 + g + 8 * r] = l[r];
         }
     }
+    const uint32_t n_cta = cluster, rank = split % n_cta;
+    if (n_cta > 1) lat_cluster_sync();
+    else __syncthreads();
+    const uint32_t share = (KV / 4 + n_cta - 1) / n_cta, p0 = rank * share, p1 = min(p0 + share, (uint32_t)KV / 4);
+    for (uint32_t i = threadIdx.x; i < 16 * share; i += 128) {
+        const uint32_t r = i / share, piece = p0 + i % share, h = h0 + r;
+        if (h >= a.heads || piece >= p1) continue;
+        float mc[8], mx = -INFINITY;
+#pragma unroll
+        for (int p = 0; p < 8; ++p) {
+            mc[p] = (uint32_t)p < n_cta ? lat_peer(stat + r, p) : -INFINITY;
+            mx = fmaxf(mx, mc[p]);
+        }
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+        float w = 0.f;
+#pragma unroll
+        for (int p = 0; p < 8; ++p) {
+            if ((uint32_t)p >= n_cta || mc[p] == -INFINITY) continue;
+            const float e = expf(mc[p] - mx);
+            const float4 x = lat_peer4(sums + r * kSumPitch + piece * 4, p);
+            v.x = fmaf(e, x.x, v.x);
+            v.y = fmaf(e, x.y, v.y);
+            v.z = fmaf(e, x.z, v.z);
+            v.w = fmaf(e, x.w, v.w);
+            w = fmaf(e, lat_peer(stat + 16 + r, p), w);
+        }
+        float *dst = a.partial + (((size_t)t * a.heads + h) * (a.n_splits / n_cta) + split / n_cta) * (a.kv_stride + 8);
+        if (piece * 4 < a.kv_stride) *reinterpret_cast<float4 *>(dst + piece * 4) = v;
+        if (piece == 0) {
+            dst[a.kv_stride] = mx;
+            dst[a.kv_stride + 1] = w;
+        }
+    }
+    if (n_cta > 1) lat_cluster_sync();  // no CTA leaves while another still reads its shared memory
 }
 
 // ------------------------------------------------------------------ absorbed: combine, W_uv
@@ -605,11 +661,24 @@ qk_status enter(qk_ctx *ctx, qk_ctx **c) {
     } while (0)
 
 template <int KV>
-qk_status launch_mma(qk_ctx *c, const LatentArgs &a, const uint16_t *cache) {
+qk_status launch_mma(qk_ctx *c, const LatentArgs &a, const uint16_t *cache, uint32_t cluster) {
     QK_CUDA(cudaFuncSetAttribute(latent_mma_kernel<KV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)LatShape<KV>::kSmem));
-    QK_LAUNCH(c, latent_mma_kernel<KV>, dim3(a.n_splits, (a.heads + 15) / 16, a.tokens), dim3(128), LatShape<KV>::kSmem,
-              a, cache);
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.n_splits, (a.heads + 15) / 16, a.tokens);
+    cfg.blockDim = dim3(128);
+    cfg.dynamicSmemBytes = LatShape<KV>::kSmem;
+    cfg.stream = c->stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = c->pdl ? 1 : 0;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = cluster;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 2;
+    QK_CUDA(cudaLaunchKernelEx(&cfg, latent_mma_kernel<KV>, a, cache, cluster));
+    c->launches++;
     return QK_OK;
 }
 
@@ -674,11 +743,13 @@ qk_status qk_latent_attention(qk_ctx *ctx, const qk_latent_call *d) {
     else QK_LAUNCH(c, absorb_query_kernel<float>, ag, dim3(kAbsWarps * 32), 0, a, (const float *)d->uk);
     if (bf16 && d->kv_stride <= 512 && c->decode_attention_kernel != 0) {
         const uint16_t *cache = (const uint16_t *)d->cache;
-        if (d->kv_stride <= 64) st = launch_mma<64>(c, a, cache);
-        else if (d->kv_stride <= 128) st = launch_mma<128>(c, a, cache);
-        else if (d->kv_stride <= 256) st = launch_mma<256>(c, a, cache);
-        else st = launch_mma<512>(c, a, cache);
+        const uint32_t cluster = a.n_splits % 8 == 0 ? 8 : a.n_splits % 4 == 0 ? 4 : a.n_splits % 2 == 0 ? 2 : 1;
+        if (d->kv_stride <= 64) st = launch_mma<64>(c, a, cache, cluster);
+        else if (d->kv_stride <= 128) st = launch_mma<128>(c, a, cache, cluster);
+        else if (d->kv_stride <= 256) st = launch_mma<256>(c, a, cache, cluster);
+        else st = launch_mma<512>(c, a, cache, cluster);
         if (st != QK_OK) return st;
+        a.n_splits /= cluster;  // (what is left for the last launch to combine)
     } else {
         const dim3 pg(a.n_splits, a.heads, a.tokens);
         const size_t smem = d->kv_stride * 8;

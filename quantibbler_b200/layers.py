@@ -255,7 +255,8 @@ class LatentAttention:
     def n_splits(self, rows: int, window: int) -> int:
         """Key splits of the absorbed form: about two blocks per SM, 32 keys or more each."""
         groups = -(-self.heads // 16) if self.weights.tag == QK_BF16 else self.heads
-        return max(1, min(64, 296 // max(1, rows * groups), -(-window // 32)))
+        want = max(1, min(64, 296 // max(1, rows * groups), -(-window // 32)))
+        return want // 8 * 8 if want >= 8 else want   # (clusters of eight merge their splits)
 
     def _split_floats(self, rows: Rows, window: int) -> int:
         """Scratch of the absorbed form for any number of rows it may get in this workspace."""
@@ -349,7 +350,7 @@ class GatedDelta:
         rows.settle()
         o_stride = padded(self.heads * self.vdim)
         out = rows.f32("readout", o_stride)
-        qkv, gates = rows.f32("qkv", self.channels), rows.f32("gates", self.heads * 4)
+        qkv, gates = rows.f32("qkv", self.channels), rows.buffer("gates", self.heads * 20, rows.torch.float32, rows=up_to(rows.cap, 8))
         c = DeltaCall(tokens=rows.n, segments=rows.segments, positions=rows.positions.data_ptr(),
                       slots=rows.slots.data_ptr(), seg_first=rows.seg_first.data_ptr(),
                       seg_len=rows.seg_len.data_ptr(), seg_row=rows.seg_row.data_ptr(), heads=self.heads,
