@@ -382,18 +382,28 @@ delta_inputs_kernel(DeltaArgs a, uint32_t n_tokens) {
     }
 }
 
-// Values j = 0 .. 31 of every lane -> the sum over the lanes of value `lane`, in each lane.
-__device__ __forceinline__ float scatter_sum(float (&v)[32], uint32_t lane) {
+// Sums over the lanes of 32 values each of two kinds, value (token, column): lane 4 t + c ends
+// with token t, column c.  The lanes' register slot i holds token i ^ lane / 4, so that in the
+// first three rounds every lane sends the upper half of its slots and keeps the lower.
+__device__ __forceinline__ void scatter_sums(float (&x)[32], float (&y)[32], uint32_t lane) {
 #pragma unroll
-    for (int half = 16; half > 0; half >>= 1) {
+    for (int half = 16; half > 2; half >>= 1)
+#pragma unroll
+        for (int j = 0; j < half; ++j) {
+            x[j] += __shfl_xor_sync(0xffffffffu, x[j + half], half);
+            y[j] += __shfl_xor_sync(0xffffffffu, y[j + half], half);
+        }
+#pragma unroll
+    for (int half = 2; half > 0; half >>= 1) {
         const bool up = (lane & half) != 0;
 #pragma unroll
         for (int j = 0; j < half; ++j) {
-            const float send = up ? v[j] : v[j + half], keep = up ? v[j + half] : v[j];
-            v[j] = keep + __shfl_xor_sync(0xffffffffu, send, half);
+            const float sx = up ? x[j] : x[j + half], kx = up ? x[j + half] : x[j];
+            const float sy = up ? y[j] : y[j + half], ky = up ? y[j + half] : y[j];
+            x[j] = kx + __shfl_xor_sync(0xffffffffu, sx, half);
+            y[j] = ky + __shfl_xor_sync(0xffffffffu, sy, half);
         }
     }
-    return v[0];
 }
 
 constexpr int kChunkWarps = 4, kChunkCols = 4;  // columns per warp
@@ -500,25 +510,30 @@ delta_chunk_scan_kernel(DeltaArgs a, uint32_t n_tokens, int vec) {
                 }
             }
         };
-        auto products = [&](const float *rows) -> float {
-            float part[32];
+        float dk[32], dq[32];
 #pragma unroll
-            for (int t = 0; t < kMini; ++t) {
-                f32x2 x[kPairs];
-                piece(rows + t * S::kDim, x);
+        for (int i = 0; i < kMini; ++i) {
+            f32x2 x[kPairs], y[kPairs];
+            const uint32_t at = ((uint32_t)i ^ my_t) * S::kDim;
+            piece(k + at, x);
+            piece(q + at, y);
 #pragma unroll
-                for (int c = 0; c < kChunkCols; ++c) {
-                    f32x2 acc = mul2(s[c][0], x[0]);
+            for (int c = 0; c < kChunkCols; ++c) {
+                f32x2 ak = mul2(s[c][0], x[0]), aq = mul2(s[c][0], y[0]);
 #pragma unroll
-                    for (int p = 1; p < kPairs; ++p) acc = fma2(s[c][p], x[p], acc);
-                    float lo, hi;
-                    unpack2(acc, lo, hi);
-                    part[t * kChunkCols + c] = lo + hi;
+                for (int p = 1; p < kPairs; ++p) {
+                    ak = fma2(s[c][p], x[p], ak);
+                    aq = fma2(s[c][p], y[p], aq);
                 }
+                float lo, hi;
+                unpack2(ak, lo, hi);
+                dk[i * kChunkCols + c] = lo + hi;
+                unpack2(aq, lo, hi);
+                dq[i * kChunkCols + c] = lo + hi;
             }
-            return scatter_sum(part, lane);
-        };
-        const float sk = products(k), sq = products(q);
+        }
+        scatter_sums(dk, dq, lane);
+        const float sk = dk[0], sq = dq[0];
         // lane (t, c): the triangular solve over the tokens of column c
         float kk[kMini], kq[kMini];
 #pragma unroll
@@ -582,7 +597,9 @@ template <int kE>
 qk_status launch_chunk_scan(qk_ctx *c, const DeltaArgs &a, size_t tokens, int vec) {
     using S = ChunkShape<kE>;
     QK_CUDA(cudaFuncSetAttribute(delta_chunk_scan_kernel<kE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
-    (void)qk::launch_pdl(c->pdl, delta_chunk_scan_kernel<kE>, dim3((a.vdim + S::kCols - 1) / S::kCols, a.heads),
+    // (no early launch: blocks that came in while the inputs kernel drains would crowd on the few
+    // SMs that are free first, and stay there)
+    (void)qk::launch_pdl(false, delta_chunk_scan_kernel<kE>, dim3((a.vdim + S::kCols - 1) / S::kCols, a.heads),
                          dim3(kChunkWarps * 32), S::kSmem, c->stream, a, (uint32_t)tokens, vec);
     QK_CUDA(cudaGetLastError());
     c->launches++;

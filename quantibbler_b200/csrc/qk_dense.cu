@@ -278,7 +278,8 @@ template <int BN> struct TcShape {
     static constexpr uint32_t kABytes = kTcM * kTcK * 2, kBBytes = BN * kTcK * 2, kStage = kABytes + kBBytes;
     static constexpr int kStages = BN == 256 ? 4 : BN == 128 ? 6 : 8;
     static constexpr uint32_t kTmemCols = 2 * BN;
-    static constexpr size_t kSmem = 1024 + kStages * kStage + (2 * kStages + 5) * 8 + 32;
+    static constexpr size_t kSmem = 1024 + kStages * kStage + kTcEpiWarps * 32 * 36 * 4 + (2 * kStages + 5) * 8 + 32;
+    static_assert(kSmem <= 227 * 1024, "the stages must fit the shared memory of a CTA");
 };
 struct TcArgs {
     uint32_t n_tokens, rows, k_chunks, m_tiles, tiles, wait_limit;
@@ -316,53 +317,71 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
         : "memory");
 }
 
-// Thirty-two consecutive outputs n0 .. of token t.  `vec`: rows are 16-byte aligned.
-__device__ __forceinline__ void tc_store32(const OutputArgs &o, uint32_t t, uint32_t n0, uint32_t limit,
-                                           float (&v)[32], bool vec) {
-    if (n0 >= limit) return;
-    if (!vec || n0 + 32 > limit) {
+// A warp's 32 rows x 32 columns go through shared memory, so that eight lanes hold 32 consecutive
+// columns of a row, four each: whole lines for every load and store of the epilogue.
+constexpr int kEpiPitch = 36;  // floats per staged row
+__device__ __forceinline__ void tc_store_tile(const OutputArgs &o, uint32_t t0, uint32_t n_tokens, uint32_t n0,
+                                              uint32_t limit, const float (&v)[32], float *stage, uint32_t lane, bool vec) {
+    __syncwarp();
 #pragma unroll
-        for (int j = 0; j < 32; ++j)
-            if (n0 + j < limit) {
-                if (o.kind == QK_OUTPUT_GLU) put(o.out, o.out_bf16, (size_t)t * o.out_stride + n0 + j, v[j]);
-                else finish(o, t, n0 + j, v[j]);
+    for (int j = 0; j < 32; j += 4)
+        *reinterpret_cast<float4 *>(stage + lane * kEpiPitch + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+    __syncwarp();
+    const uint32_t c = (lane % 8) * 4, n = n0 + c;
+    if (n >= limit) return;
+    const bool wide = vec && n + 4 <= limit;
+    float4 scale = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (wide && o.kind == QK_OUTPUT_RESIDUAL && o.scale) scale = *reinterpret_cast<const float4 *>(o.scale + n);
+    float4 old[8];
+    if (wide && o.kind == QK_OUTPUT_RESIDUAL) {
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const uint32_t t = min(t0 + i * 4 + lane / 8, n_tokens - 1);
+            old[i] = *reinterpret_cast<const float4 *>(o.residual + (size_t)t * o.residual_stride + n);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const uint32_t r = i * 4 + lane / 8, t = t0 + r;
+        if (t >= n_tokens) continue;
+        float4 x = *reinterpret_cast<const float4 *>(stage + r * kEpiPitch + c);
+        if (!wide) {
+            const float e[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (n + j < limit) {
+                    if (o.kind == QK_OUTPUT_GLU) put(o.out, o.out_bf16, (size_t)t * o.out_stride + n + j, e[j]);
+                    else finish(o, t, n + j, e[j]);
+                }
+            continue;
+        }
+        if (o.kind == QK_OUTPUT_RESIDUAL) {
+            x = make_float4(fmaf(x.x, scale.x, old[i].x), fmaf(x.y, scale.y, old[i].y), fmaf(x.z, scale.z, old[i].z),
+                            fmaf(x.w, scale.w, old[i].w));
+            *reinterpret_cast<float4 *>(o.residual + (size_t)t * o.residual_stride + n) = x;
+            if (!o.out) continue;
+        } else if (o.kind == QK_OUTPUT_SIDE) {
+            const uint32_t id = (uint32_t)min(max(o.ids[t], 0), (int)o.vocab - 1);
+            const size_t at = (size_t)id * o.side_stride + o.side_offset + n;
+            float e[4];
+            if (o.side_bf16) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) e[j] = bf16_bits_to_float(static_cast<const uint16_t *>(o.side)[at + j]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) e[j] = static_cast<const float *>(o.side)[at + j];
             }
-        return;
-    }
-    if (o.kind == QK_OUTPUT_RESIDUAL) {
-        float *r = o.residual + (size_t)t * o.residual_stride + n0;
-#pragma unroll
-        for (int j = 0; j < 32; j += 4) {
-            const float4 old = *reinterpret_cast<const float4 *>(r + j);
-            float4 s = make_float4(1.f, 1.f, 1.f, 1.f);
-            if (o.scale) s = *reinterpret_cast<const float4 *>(o.scale + n0 + j);
-            v[j] = old.x + v[j] * s.x;
-            v[j + 1] = old.y + v[j + 1] * s.y;
-            v[j + 2] = old.z + v[j + 2] * s.z;
-            v[j + 3] = old.w + v[j + 3] * s.w;
-            *reinterpret_cast<float4 *>(r + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+            x = make_float4(activate(o.act, x.x) * e[0], activate(o.act, x.y) * e[1], activate(o.act, x.z) * e[2],
+                            activate(o.act, x.w) * e[3]);
         }
-        if (!o.out) return;
-    } else if (o.kind == QK_OUTPUT_SIDE) {
-#pragma unroll
-        for (int j = 0; j < 32; ++j) v[j] = activate(o.act, v[j]) * side_value(o, t, n0 + j);
-    }
-    if (o.out_bf16) {
-        uint16_t *p = static_cast<uint16_t *>(o.out) + (size_t)t * o.out_stride + n0;
-#pragma unroll
-        for (int j = 0; j < 32; j += 8) {
-            uint32_t u[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-                u[e] = (uint32_t)float_to_bf16_bits(v[j + 2 * e]) |
-                       ((uint32_t)float_to_bf16_bits(v[j + 2 * e + 1]) << 16);
-            *reinterpret_cast<uint4 *>(p + j) = make_uint4(u[0], u[1], u[2], u[3]);
+        const size_t at = (size_t)t * o.out_stride + n;
+        if (o.out_bf16) {
+            const uint32_t lo = (uint32_t)float_to_bf16_bits(x.x) | ((uint32_t)float_to_bf16_bits(x.y) << 16);
+            const uint32_t hi = (uint32_t)float_to_bf16_bits(x.z) | ((uint32_t)float_to_bf16_bits(x.w) << 16);
+            *reinterpret_cast<uint2 *>(static_cast<uint16_t *>(o.out) + at) = make_uint2(lo, hi);
+        } else {
+            *reinterpret_cast<float4 *>(static_cast<float *>(o.out) + at) = x;
         }
-    } else {
-        float *p = static_cast<float *>(o.out) + (size_t)t * o.out_stride + n0;
-#pragma unroll
-        for (int j = 0; j < 32; j += 4)
-            *reinterpret_cast<float4 *>(p + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
     }
 }
 
@@ -374,7 +393,8 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     qk::pdl_launch();
     extern __shared__ __align__(1024) uint8_t tc_smem[];
     uint8_t *tiles = reinterpret_cast<uint8_t *>(((uintptr_t)tc_smem + 1023) & ~(uintptr_t)1023);
-    uint64_t *full = reinterpret_cast<uint64_t *>(tiles + S::kStages * S::kStage);
+    float *epi = reinterpret_cast<float *>(tiles + S::kStages * S::kStage);  // [epilogue warp][32][kEpiPitch]
+    uint64_t *full = reinterpret_cast<uint64_t *>(epi + kTcEpiWarps * 32 * kEpiPitch);
     uint64_t *empty = full + S::kStages;
     uint64_t *acc_full = empty + S::kStages;
     uint64_t *acc_empty = acc_full + 2;
@@ -491,7 +511,8 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
         uint32_t seg = 0;
         for (uint32_t tile = blockIdx.x; tile < g.tiles; tile += gridDim.x, ++seg) {
             const uint32_t acc = seg & 1;
-            const uint32_t t = (tile % g.m_tiles) * kTcM + quarter * 32 + lane, n0 = (tile / g.m_tiles) * BN;
+            const uint32_t t0 = (tile % g.m_tiles) * kTcM + quarter * 32, n0 = (tile / g.m_tiles) * BN;
+            float *stage = epi + (warp - 2) * 32 * kEpiPitch;
             if (!tc_epilogue_vote(mbar_wait(&acc_full[acc], (seg >> 1) & 1, abort_flag, g.wait_limit))) {
                 *abort_flag = 1;
                 break;
@@ -508,7 +529,7 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
 #pragma unroll
                     for (int j = 0; j < 32; ++j)
                         v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
-                    if (t < g.n_tokens) tc_store32(out, t, (n0 + c) / 2, g.rows / 2, v, vec != 0);
+                    tc_store_tile(out, t0, g.n_tokens, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
                 }
             } else {
                 for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += 32) {
@@ -518,7 +539,7 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(a[j]);
-                    if (t < g.n_tokens) tc_store32(out, t, n0 + c, g.rows, v, vec != 0);
+                    tc_store_tile(out, t0, g.n_tokens, n0 + c, g.rows, v, stage, lane, vec != 0);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -532,6 +553,88 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
         asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem_base), "r"(S::kTmemCols)
                      : "memory");
     if (threadIdx.x == 0 && *abort_flag) atomicOr(g.error, 1);
+}
+
+// The same rows for a normed or concatenated input whose rows are 16-byte aligned, bfloat16 out: a
+// thread keeps its kV pieces of four entries in registers, all loads of the row go out together.
+template <int kV>
+__global__ void __launch_bounds__(256)
+dense_norm_rows_kernel(InputArgs in, uint16_t *__restrict__ dst) {
+    qk::pdl_launch();
+    qk::pdl_wait();
+    __shared__ float red[8];
+    const uint32_t t = blockIdx.x, n = in.width, pieces = n / 4;
+    const float4 *xr = reinterpret_cast<const float4 *>(in.x + (size_t)t * in.x_stride);
+    float4 h[kV];
+#pragma unroll
+    for (int j = 0; j < kV; ++j) {
+        const uint32_t p = threadIdx.x + 256 * j;
+        h[j] = p < pieces ? xr[p] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    if (in.pending) {
+        const float4 *pr = reinterpret_cast<const float4 *>(in.pending + (size_t)t * in.pending_stride);
+        float4 y[kV];
+        float ps = 0.f;
+#pragma unroll
+        for (int j = 0; j < kV; ++j) {
+            const uint32_t p = threadIdx.x + 256 * j;
+            y[j] = p < pieces ? pr[p] : make_float4(0.f, 0.f, 0.f, 0.f);
+            ps += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+        }
+        const float inv = 1.0f / sqrtf(in_block_sum(ps, red) / (float)n + in.pending_eps);
+        const float4 *pw = reinterpret_cast<const float4 *>(in.pending_weight);
+        float4 *xo = in.x_out ? reinterpret_cast<float4 *>(in.x_out + (size_t)t * in.x_stride) : nullptr;
+#pragma unroll
+        for (int j = 0; j < kV; ++j) {
+            const uint32_t p = threadIdx.x + 256 * j;
+            if (p >= pieces) continue;
+            const float4 w = pw[p];
+            h[j].x += y[j].x * inv * w.x;
+            h[j].y += y[j].y * inv * w.y;
+            h[j].z += y[j].z * inv * w.z;
+            h[j].w += y[j].w * inv * w.w;
+            if (xo) xo[p] = h[j];
+        }
+    }
+    float mean = 0.f, inv = 1.f;
+    if (in.norm == QK_NORM_LAYER) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < kV; ++j) s += h[j].x + h[j].y + h[j].z + h[j].w;
+        mean = in_block_sum(s, red) / (float)n;
+    }
+    if (in.norm != QK_NORM_NONE) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < kV; ++j) {
+            if (threadIdx.x + 256 * j >= pieces) continue;
+            const float a = h[j].x - mean, b = h[j].y - mean, c = h[j].z - mean, d = h[j].w - mean;
+            s += a * a + b * b + c * c + d * d;
+        }
+        inv = 1.0f / sqrtf(in_block_sum(s, red) / (float)n + in.norm_eps);
+    }
+    uint2 *o = reinterpret_cast<uint2 *>(dst + (size_t)t * in.k);
+    const float4 *nw = reinterpret_cast<const float4 *>(in.norm_weight);
+    const uint32_t half = (in.kind == QK_INPUT_CONCAT ? in.k / 2 : in.k) / 4;
+    const float4 *second = reinterpret_cast<const float4 *>(in.second ? in.second + (size_t)t * in.x_stride : nullptr);
+    auto pack = [](float4 v) {
+        return make_uint2((uint32_t)float_to_bf16_bits(v.x) | ((uint32_t)float_to_bf16_bits(v.y) << 16),
+                          (uint32_t)float_to_bf16_bits(v.z) | ((uint32_t)float_to_bf16_bits(v.w) << 16));
+    };
+#pragma unroll
+    for (int j = 0; j < kV; ++j) {
+        const uint32_t p = threadIdx.x + 256 * j;
+        if (p >= half) continue;  // (pieces past the width are zeros)
+        float4 v = h[j];
+        if (in.norm != QK_NORM_NONE && p < pieces) {
+            const float4 w = nw[p];
+            v = make_float4((v.x - mean) * inv * w.x, (v.y - mean) * inv * w.y, (v.z - mean) * inv * w.z,
+                            (v.w - mean) * inv * w.w);
+        }
+        o[p] = pack(v);
+        if (in.kind == QK_INPUT_CONCAT) o[half + p] = pack(p < pieces ? second[p] : make_float4(0.f, 0.f, 0.f, 0.f));
+    }
+    if (in.append.src) append_latent(in, t, red);
 }
 
 // ------------------------------------------------------------------ narrow form
@@ -1023,6 +1126,22 @@ qk_status validate(const qk_dense_call *d, bool with_weights) {
 
 template <typename A>
 qk_status launch_input(qk_ctx *c, const InputArgs &in, size_t tokens, A *dst) {
+    auto aligned = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
+    const size_t half = in.kind == QK_INPUT_CONCAT ? in.k / 2 : in.k;
+    if (sizeof(A) == 2 && dst && (in.kind == QK_INPUT_NORM || in.kind == QK_INPUT_CONCAT) && in.width % 4 == 0 &&
+        half % 4 == 0 && half <= 8192 && in.x_stride % 4 == 0 && aligned(in.x) && aligned(in.x_out) && aligned(dst) &&
+        (!in.pending || (in.pending_stride % 4 == 0 && aligned(in.pending) && aligned(in.pending_weight))) &&
+        aligned(in.second) && aligned(in.norm_weight)) {
+        uint16_t *o = reinterpret_cast<uint16_t *>(dst);
+        const dim3 grid((unsigned)tokens), block(256);
+        if (half <= 1024) (void)qk::launch_pdl(c->pdl, dense_norm_rows_kernel<1>, grid, block, 0, c->stream, in, o);
+        else if (half <= 2048) (void)qk::launch_pdl(c->pdl, dense_norm_rows_kernel<2>, grid, block, 0, c->stream, in, o);
+        else if (half <= 4096) (void)qk::launch_pdl(c->pdl, dense_norm_rows_kernel<4>, grid, block, 0, c->stream, in, o);
+        else (void)qk::launch_pdl(c->pdl, dense_norm_rows_kernel<8>, grid, block, 0, c->stream, in, o);
+        QK_CUDA(cudaGetLastError());
+        c->launches++;
+        return QK_OK;
+    }
     const size_t smem = dst ? (size_t)in.k * 4 : 0;
     if (smem > kVecSmemMax) return qk::fail(QK_ERR_VALUE, "qk_dense: an input vector of %u entries does not fit shared memory", in.k);
     QK_CUDA(cudaFuncSetAttribute(dense_input_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1123,8 +1242,7 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
         if (d->tokens <= 64) return launch_narrow<64>(c, rows, stride, *d, out);
         return launch_narrow<128>(c, rows, stride, *d, out);
     }
-    const int per16 = d->out_dtype == QK_BF16 ? 8 : 4;
-    const int vec = (!d->out || (((uintptr_t)d->out & 15) == 0 && d->out_stride % per16 == 0)) &&
+    const int vec = (!d->out || (((uintptr_t)d->out & 15) == 0 && d->out_stride % 4 == 0)) &&
                     (!d->residual || (((uintptr_t)d->residual & 15) == 0 && d->residual_stride % 4 == 0)) &&
                     ((uintptr_t)d->out_scale & 15) == 0;
     switch (pick_tile(qk::ceil_div(d->tokens, kTcM), d->rows, (size_t)c->sm_count)) {
