@@ -254,7 +254,7 @@ constexpr int kMini = 8, kCoef = 20;
 // the unit norms, then the scalars.  kTok = 8: rows of one portion, kCoef scalars per row and
 // head; kTok = 1: any row, {beta, g, k . q} per row and head.
 template <int kTaps, int kTok>
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, kTaps <= 4 ? 4 : 2)
 delta_inputs_kernel(DeltaArgs a, uint32_t n_tokens) {
     qk::pdl_launch();
     extern __shared__ float ci_smem[];  // q, k [kTok][dim + 1], then products, then [ratio][kTok][2] gates
@@ -266,6 +266,7 @@ delta_inputs_kernel(DeltaArgs a, uint32_t n_tokens) {
     if (pos < 0) return;
     const int in_seg = a.seg_row[t0];
     const uint32_t slot = (uint32_t)a.slots[t0], key0 = a.kv_heads * a.dim, per = ratio * a.vdim;
+#pragma unroll 1
     for (uint32_t c = threadIdx.x; c < 2 * a.dim + per; c += 256) {
         const uint32_t which = c < a.dim ? 0 : c < 2 * a.dim ? 1 : 2;
         const uint32_t in = which == 0 ? c : which == 1 ? c - a.dim : c - 2 * a.dim;   // place in this head's part
@@ -273,6 +274,12 @@ delta_inputs_kernel(DeltaArgs a, uint32_t n_tokens) {
         const uint32_t ch = which == 0 ? own : which == 1 ? key0 + own : 2 * key0 + own;
         const float *taps = (which == 0 ? a.conv_q : which == 1 ? a.conv_k : a.conv_v) + (size_t)own * a.taps;
         float w[kTaps], x[kTaps - 1 + kTok];
+        if (in_seg >= kTaps - 1) {  // (uniform over the block) every earlier input is a row
+            const float *src = a.proj + (size_t)(t0 - (kTaps - 1)) * a.proj_stride + ch;
+#pragma unroll
+            for (int j = 0; j < kTaps - 1 + kTok; ++j)
+                x[j] = j - (kTaps - 1) < (int)n ? src[(size_t)j * a.proj_stride] : 0.f;
+        } else
 #pragma unroll
         for (int j = 0; j < kTaps - 1 + kTok; ++j) {
             const int r = j - (kTaps - 1), p = pos + r;  // row t0 + r at position p

@@ -320,6 +320,18 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&v)[16]) {
 // A warp's 32 rows x 32 columns go through shared memory, so that eight lanes hold 32 consecutive
 // columns of a row, four each: whole lines for every load and store of the epilogue.
 constexpr int kEpiPitch = 36;  // floats per staged row
+// Element by element: unaligned buffers and ragged column ends.  Out of line, so that the usual
+// path stays short enough for the instruction cache.
+__device__ __noinline__ void tc_store_slow(const OutputArgs &o, uint32_t t0, uint32_t n_tokens, uint32_t n0, uint32_t limit,
+                                           const float *stage, uint32_t lane, bool raw) {
+    for (uint32_t r = 0; r < 32 && t0 + r < n_tokens; ++r)
+        if (n0 + lane < limit) {
+            const float v = stage[r * kEpiPitch + lane];
+            if (raw) put(o.out, o.out_bf16, (size_t)(t0 + r) * o.out_stride + n0 + lane, v);
+            else finish(o, t0 + r, n0 + lane, v);
+        }
+}
+template <int KIND>
 __device__ __forceinline__ void tc_store_tile(const OutputArgs &o, uint32_t t0, uint32_t n_tokens, uint32_t n0,
                                               uint32_t limit, const float (&v)[32], float *stage, uint32_t lane, bool vec) {
     __syncwarp();
@@ -327,13 +339,15 @@ __device__ __forceinline__ void tc_store_tile(const OutputArgs &o, uint32_t t0, 
     for (int j = 0; j < 32; j += 4)
         *reinterpret_cast<float4 *>(stage + lane * kEpiPitch + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
     __syncwarp();
+    if (!vec || n0 + 32 > limit) {
+        tc_store_slow(o, t0, n_tokens, n0, limit, stage, lane, KIND == QK_OUTPUT_GLU);
+        return;
+    }
     const uint32_t c = (lane % 8) * 4, n = n0 + c;
-    if (n >= limit) return;
-    const bool wide = vec && n + 4 <= limit;
     float4 scale = make_float4(1.f, 1.f, 1.f, 1.f);
-    if (wide && o.kind == QK_OUTPUT_RESIDUAL && o.scale) scale = *reinterpret_cast<const float4 *>(o.scale + n);
-    float4 old[8];
-    if (wide && o.kind == QK_OUTPUT_RESIDUAL) {
+    float4 old[KIND == QK_OUTPUT_RESIDUAL ? 8 : 1];
+    if constexpr (KIND == QK_OUTPUT_RESIDUAL) {
+        if (o.scale) scale = *reinterpret_cast<const float4 *>(o.scale + n);
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
             const uint32_t t = min(t0 + i * 4 + lane / 8, n_tokens - 1);
@@ -345,34 +359,14 @@ __device__ __forceinline__ void tc_store_tile(const OutputArgs &o, uint32_t t0, 
         const uint32_t r = i * 4 + lane / 8, t = t0 + r;
         if (t >= n_tokens) continue;
         float4 x = *reinterpret_cast<const float4 *>(stage + r * kEpiPitch + c);
-        if (!wide) {
-            const float e[4] = {x.x, x.y, x.z, x.w};
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                if (n + j < limit) {
-                    if (o.kind == QK_OUTPUT_GLU) put(o.out, o.out_bf16, (size_t)t * o.out_stride + n + j, e[j]);
-                    else finish(o, t, n + j, e[j]);
-                }
-            continue;
-        }
-        if (o.kind == QK_OUTPUT_RESIDUAL) {
+        if constexpr (KIND == QK_OUTPUT_RESIDUAL) {
             x = make_float4(fmaf(x.x, scale.x, old[i].x), fmaf(x.y, scale.y, old[i].y), fmaf(x.z, scale.z, old[i].z),
                             fmaf(x.w, scale.w, old[i].w));
             *reinterpret_cast<float4 *>(o.residual + (size_t)t * o.residual_stride + n) = x;
             if (!o.out) continue;
-        } else if (o.kind == QK_OUTPUT_SIDE) {
-            const uint32_t id = (uint32_t)min(max(o.ids[t], 0), (int)o.vocab - 1);
-            const size_t at = (size_t)id * o.side_stride + o.side_offset + n;
-            float e[4];
-            if (o.side_bf16) {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) e[j] = bf16_bits_to_float(static_cast<const uint16_t *>(o.side)[at + j]);
-            } else {
-#pragma unroll
-                for (int j = 0; j < 4; ++j) e[j] = static_cast<const float *>(o.side)[at + j];
-            }
-            x = make_float4(activate(o.act, x.x) * e[0], activate(o.act, x.y) * e[1], activate(o.act, x.z) * e[2],
-                            activate(o.act, x.w) * e[3]);
+        } else if constexpr (KIND == QK_OUTPUT_SIDE) {
+            x = make_float4(activate(o.act, x.x) * side_value(o, t, n), activate(o.act, x.y) * side_value(o, t, n + 1),
+                            activate(o.act, x.z) * side_value(o, t, n + 2), activate(o.act, x.w) * side_value(o, t, n + 3));
         }
         const size_t at = (size_t)t * o.out_stride + n;
         if (o.out_bf16) {
@@ -385,7 +379,7 @@ __device__ __forceinline__ void tc_store_tile(const OutputArgs &o, uint32_t t0, 
     }
 }
 
-template <int BN>
+template <int BN, int KIND>
 __global__ void __launch_bounds__(kTcThreads, 1)
 dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, TcArgs g,
                 OutputArgs out, int vec) {
@@ -519,27 +513,28 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
             }
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const uint32_t lane_addr = tmem_base + acc * BN + ((quarter * 32) << 16);
-            if (out.kind == QK_OUTPUT_GLU) {
-                for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += 64) {  // warp-uniform
-                    uint32_t a[32], b[32];
-                    tmem_ld32(lane_addr + c, a);
+#pragma unroll 1
+            for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += KIND == QK_OUTPUT_GLU ? 64 : 32) {  // warp-uniform
+                uint32_t a[32];
+                float v[32];
+                tmem_ld32(lane_addr + c, a);
+                if constexpr (KIND == QK_OUTPUT_GLU) {
+                    uint32_t b[32];
                     tmem_ld32(lane_addr + c + 32, b);
                     tmem_ld_wait();
-                    float v[32];
+                    if (out.act == QK_ACT_RELU) {
 #pragma unroll
-                    for (int j = 0; j < 32; ++j)
-                        v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
-                    tc_store_tile(out, t0, g.n_tokens, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
-                }
-            } else {
-                for (uint32_t c = 0; c < BN && n0 + c < g.rows; c += 32) {
-                    uint32_t a[32];
-                    tmem_ld32(lane_addr + c, a);
+                        for (int j = 0; j < 32; ++j) v[j] = fmaxf(__uint_as_float(a[j]), 0.f) * __uint_as_float(b[j]);
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
+                    }
+                    tc_store_tile<KIND>(out, t0, g.n_tokens, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
+                } else {
                     tmem_ld_wait();
-                    float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(a[j]);
-                    tc_store_tile(out, t0, g.n_tokens, n0 + c, g.rows, v, stage, lane, vec != 0);
+                    tc_store_tile<KIND>(out, t0, g.n_tokens, n0 + c, g.rows, v, stage, lane, vec != 0);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -916,8 +911,8 @@ int pick_tile(size_t m_tiles, size_t rows, size_t sms) {
     return best;
 }
 
-template <int BN>
-qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out,
+template <int BN, int KIND>
+qk_status launch_tc_kind(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out,
                     int vec) {
     using S = TcShape<BN>;
     CUtensorMap xm, wm;
@@ -932,8 +927,8 @@ qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_ca
     g.tiles = g.m_tiles * (uint32_t)qk::ceil_div(d.rows, BN);
     g.wait_limit = c->wait_limit ? c->wait_limit : kTcWaitDefault;
     g.error = (int *)c->d_err.ptr;
-    QK_CUDA(cudaFuncSetAttribute(dense_tc_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
-    (void)qk::launch_pdl(c->pdl, dense_tc_kernel<BN>, dim3(std::min(g.tiles, (uint32_t)c->sm_count)),
+    QK_CUDA(cudaFuncSetAttribute((dense_tc_kernel<BN, KIND>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
+    (void)qk::launch_pdl(c->pdl, (dense_tc_kernel<BN, KIND>), dim3(std::min(g.tiles, (uint32_t)c->sm_count)),
                          dim3(kTcThreads), S::kSmem, c->stream, xm, wm, g, out, vec);
     QK_CUDA(cudaGetLastError());
     c->launches++;
@@ -989,6 +984,16 @@ qk_status launch_narrow(qk_ctx *c, const void *x, size_t x_stride, const qk_dens
     c->launches++;
     c->err_armed = true;
     return QK_OK;
+}
+
+template <int BN>
+qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out, int vec) {
+    switch (d.output) {
+        case QK_OUTPUT_RESIDUAL: return launch_tc_kind<BN, QK_OUTPUT_RESIDUAL>(c, x, x_stride, d, out, vec);
+        case QK_OUTPUT_GLU: return launch_tc_kind<BN, QK_OUTPUT_GLU>(c, x, x_stride, d, out, vec);
+        case QK_OUTPUT_SIDE: return launch_tc_kind<BN, QK_OUTPUT_SIDE>(c, x, x_stride, d, out, vec);
+        default: return launch_tc_kind<BN, QK_OUTPUT_STORE>(c, x, x_stride, d, out, vec);
+    }
 }
 
 template <typename W, int NT, int R>

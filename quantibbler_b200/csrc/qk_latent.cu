@@ -80,29 +80,66 @@ __device__ __forceinline__ SplitKeys split_keys(const LatentArgs &a, int pos, ui
 }
 
 // ------------------------------------------------------------------ absorbed: W_uk^T q
-constexpr int kAbsRows = 4, kAbsWarps = 8;
+constexpr int kAbsRows = 4, kAbsWarps = 8, kAbsAhead = 8;
+__device__ __forceinline__ void lt_fetch8(const uint16_t *p, uint4 (&w)[1]) { w[0] = *reinterpret_cast<const uint4 *>(p); }
+__device__ __forceinline__ void lt_fetch8(const float *p, uint4 (&w)[2]) {
+    w[0] = *reinterpret_cast<const uint4 *>(p);
+    w[1] = *reinterpret_cast<const uint4 *>(p + 4);
+}
+__device__ __forceinline__ void lt_open8(const uint4 (&v)[1], float (&w)[8]) {
+    const uint32_t u[4] = {v[0].x, v[0].y, v[0].z, v[0].w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        w[2 * i] = __uint_as_float(u[i] << 16);
+        w[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+    }
+}
+__device__ __forceinline__ void lt_open8(const uint4 (&v)[2], float (&w)[8]) {
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        w[4 * i] = __uint_as_float(v[i].x);
+        w[4 * i + 1] = __uint_as_float(v[i].y);
+        w[4 * i + 2] = __uint_as_float(v[i].z);
+        w[4 * i + 3] = __uint_as_float(v[i].w);
+    }
+}
 template <typename W>
 __global__ void __launch_bounds__(kAbsWarps * 32)
 absorb_query_kernel(LatentArgs a, const W *__restrict__ uk) {
     qk::pdl_launch();
-    qk::pdl_wait();
-    __shared__ float sums[kAbsWarps][256];
+    extern __shared__ float ab_smem[];  // [kAbsRows][dim] queries, [kAbsWarps][256] sums
+    float *qs = ab_smem, *sums = ab_smem + kAbsRows * a.dim;
     const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32, h = blockIdx.y;
     const uint32_t c0 = blockIdx.x * 256 + lane * 8, t0 = blockIdx.z * kAbsRows;
+    const bool live = c0 < a.kv_stride;
+    const W *base = uk + (size_t)h * a.dim_stride * a.kv_stride + (live ? c0 : 0);
+    uint4 ahead[kAbsAhead][sizeof(W) / 2];
+    auto fetch = [&](uint32_t d0) {
+#pragma unroll
+        for (int i = 0; i < kAbsAhead; ++i)
+            lt_fetch8(base + (size_t)min(d0 + i * kAbsWarps, a.dim - 1) * a.kv_stride, ahead[i]);
+    };
+    fetch(warp);  // (weights depend on no other kernel)
+    qk::pdl_wait();
+    for (uint32_t i = threadIdx.x; i < kAbsRows * a.dim; i += kAbsWarps * 32)
+        qs[i] = a.q[(size_t)min(t0 + i / a.dim, a.tokens - 1) * a.q_stride + h * a.dim_stride + i % a.dim];
+    __syncthreads();
     float acc[kAbsRows][8];
 #pragma unroll
     for (int r = 0; r < kAbsRows; ++r)
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[r][e] = 0.f;
-    if (c0 < a.kv_stride) {
-        const W *base = uk + (size_t)h * a.dim_stride * a.kv_stride + c0;
-#pragma unroll 4
-        for (uint32_t d = warp; d < a.dim; d += kAbsWarps) {
+    for (uint32_t d0 = warp; d0 < a.dim; d0 += kAbsAhead * kAbsWarps) {
+        if (d0 != warp) fetch(d0);
+#pragma unroll
+        for (int i = 0; i < kAbsAhead; ++i) {
+            const uint32_t d = d0 + i * kAbsWarps;
+            if (d >= a.dim) break;
             float w[8];
-            lt_load8(base + (size_t)d * a.kv_stride, w);
+            lt_open8(ahead[i], w);
 #pragma unroll
             for (int r = 0; r < kAbsRows; ++r) {
-                const float q = a.q[(size_t)min(t0 + r, a.tokens - 1) * a.q_stride + h * a.dim_stride + d];
+                const float q = qs[r * a.dim + d];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) acc[r][e] = fmaf(q, w[e], acc[r][e]);
             }
@@ -112,13 +149,13 @@ absorb_query_kernel(LatentArgs a, const W *__restrict__ uk) {
     for (int r = 0; r < kAbsRows; ++r) {
         if (t0 + r >= a.tokens) break;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) sums[warp][lane * 8 + e] = acc[r][e];
+        for (int e = 0; e < 8; ++e) sums[warp * 256 + lane * 8 + e] = acc[r][e];
         __syncthreads();
         const uint32_t c = blockIdx.x * 256 + threadIdx.x;
         if (c < a.kv_stride) {
             float v = 0.f;
 #pragma unroll
-            for (int w = 0; w < kAbsWarps; ++w) v += sums[w][threadIdx.x];
+            for (int w = 0; w < kAbsWarps; ++w) v += sums[w * 256 + threadIdx.x];
             a.absorbed[((size_t)(t0 + r) * a.heads + h) * a.kv_stride + c] = v * a.scale;
         }
         __syncthreads();
@@ -183,9 +220,19 @@ latent_plain_kernel(LatentArgs a, const C *__restrict__ cache) {
 
 // ------------------------------------------------------------------ absorbed: scores and sums, tensor cores
 // A block of four warps takes up to 16 heads (the M side) of one row and one split of its keys,
-// 32 keys at a time.  Scores: each warp multiplies eight keys over all latent channels; sums: each
-// warp owns a quarter of the channels.  KV: staged channels per key (kv_stride <= KV).
+// 32 keys at a time.  Each warp owns a quarter of the latent channels: it stages that quarter of
+// the keys for itself, keeps the query's fragments of it in registers, multiplies the scores'
+// share of its channels and later sums the same channels; only the scores meet in shared
+// memory.  KV: staged channels per key (kv_stride <= KV).
 constexpr int kLatKeys = 32;
+template <int KV> struct LatShape {
+    static constexpr int kQuarter = KV / 4, kPitch = kQuarter + 8, kBufs = 2;
+    static constexpr int kScorePitch = kLatKeys + 4;
+    static constexpr size_t kTileBytes = kLatKeys * kPitch * 2;             // one warp's quarter of 32 keys
+    static constexpr size_t kRing = 4 * kBufs * kTileBytes, kScores = 2 * 4 * 16 * kScorePitch * 4;
+    static constexpr size_t kSums = (16 * (KV + 4) + 32) * 4;               // after the last tile
+    static constexpr size_t kSmem = (kRing > kSums ? kRing : kSums) + kScores;
+};
 __device__ __forceinline__ void lat_cluster_sync() {
     __syncwarp();
     asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -208,93 +255,87 @@ __device__ __forceinline__ float4 lat_peer4(const float *p, uint32_t cta) {
                  : "memory");
     return v;
 }
-template <int KV> struct LatShape {
-    static constexpr int kPitch = KV + 8;
-    static constexpr size_t kQBytes = 2 * 16 * kPitch * 2, kTileBytes = kLatKeys * kPitch * 2;
-    static constexpr size_t kSmem = kQBytes + 2 * kTileBytes + 16 * (kLatKeys + 4) * 4;
-};
 template <int KV>
 __global__ void __launch_bounds__(128)
 latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t cluster) {
     using S = LatShape<KV>;
-    constexpr int kTilesPerWarp = KV / 4 / 8;  // 8-channel tiles of the sums per warp
+    constexpr int kQ = S::kQuarter, kSteps = kQ / 16, kTilesPerWarp = kQ / 8;
     qk::pdl_launch();
     qk::pdl_wait();
     extern __shared__ __align__(16) uint8_t lat_smem[];
-    uint16_t *qs = reinterpret_cast<uint16_t *>(lat_smem);  // [hi, lo][16][pitch]
-    uint8_t *tiles = lat_smem + S::kQBytes;
-    float *sc = reinterpret_cast<float *>(tiles + 2 * S::kTileBytes);  // [16][kLatKeys + 4]
-    constexpr int kScPitch = kLatKeys + 4;
     const uint32_t split = blockIdx.x, h0 = blockIdx.y * 16, t = blockIdx.z;
     const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane >> 2, c4 = lane & 3;
     const int pos = a.positions[t];
-    if (pos < 0) return;
+    if (pos < 0) return;  // (the whole cluster works on one row)
+    uint8_t *ring = lat_smem + warp * S::kBufs * S::kTileBytes;
+    float *scores = reinterpret_cast<float *>(lat_smem + S::kSmem - S::kScores);  // [2][warp][16][pitch]
     const SplitKeys keys = split_keys(a, pos, split);
-    const uint16_t *base = cache + (size_t)a.slots[t] * a.ring * a.kv_stride;
-    const uint32_t ring0 = keys.first % a.ring;
-    auto fetch = [&](uint32_t k0, uint32_t buf) {
-        uint8_t *dst = tiles + buf * S::kTileBytes;
-        for (uint32_t i = threadIdx.x; i < kLatKeys * (KV / 8); i += 128) {
-            const uint32_t key = i / (KV / 8), piece = i % (KV / 8);
-            uint32_t r = ring0 + k0 + key;
-            while (r >= a.ring) r -= a.ring;
-            const bool live = k0 + key < keys.count && piece * 8 < a.kv_stride;
-            lt_copy16(dst + (key * S::kPitch + piece * 8) * 2, base + (live ? (size_t)r * a.kv_stride + piece * 8 : 0),
-                      live ? 16u : 0u);
+    const uint16_t *base = cache + (size_t)a.slots[t] * a.ring * a.kv_stride + warp * kQ;
+    const uint32_t ring0 = keys.first % a.ring, n_tiles = (keys.count + kLatKeys - 1) / kLatKeys;
+    auto fetch = [&](uint32_t tile) {
+        if (tile < n_tiles) {
+            uint8_t *dst = ring + (tile % S::kBufs) * S::kTileBytes;
+#pragma unroll 8
+            for (uint32_t i = lane; i < kLatKeys * (kQ / 8); i += 32) {
+                const uint32_t key = i / (kQ / 8), piece = i % (kQ / 8), j = tile * kLatKeys + key;
+                uint32_t r = ring0 + j;
+                if (r >= a.ring) r -= a.ring;  // (a window is no longer than the ring)
+                const bool live = j < keys.count && warp * kQ + piece * 8 < a.kv_stride;
+                lt_copy16(dst + (key * S::kPitch + piece * 8) * 2, live ? base + (size_t)r * a.kv_stride + piece * 8 : cache,
+                          live ? 16u : 0u);
+            }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    if (keys.count) fetch(0, 0);
-#pragma unroll 8
-    for (uint32_t i = threadIdx.x; i < 16 * (KV / 2); i += 128) {
-        const uint32_t r = i / (KV / 2), c = (i % (KV / 2)) * 2;
-        float x = 0.f, y = 0.f;
-        if (h0 + r < a.heads && c < a.kv_stride) {  // (kv_stride is even)
-            const float2 v = *reinterpret_cast<const float2 *>(
-                a.absorbed + ((size_t)t * a.heads + h0 + r) * a.kv_stride + c);
-            x = v.x;
-            y = v.y;
+    fetch(0);
+    // this warp's quarter of the query, as A fragments in two bfloat16 terms
+    uint32_t qh[kSteps][4], ql[kSteps][4];
+#pragma unroll
+    for (int ks = 0; ks < kSteps; ++ks)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const uint32_t r = g + (e & 1) * 8, c = warp * kQ + ks * 16 + 2 * c4 + (e >> 1) * 8;
+            float2 v = make_float2(0.f, 0.f);
+            if (h0 + r < a.heads && c < a.kv_stride)  // (kv_stride is even)
+                v = *reinterpret_cast<const float2 *>(a.absorbed + ((size_t)t * a.heads + h0 + r) * a.kv_stride + c);
+            lt_split2(v.x, v.y, qh[ks][e], ql[ks][e]);
         }
-        uint32_t hi, lo;
-        lt_split2(x, y, hi, lo);
-        *reinterpret_cast<uint32_t *>(qs + r * S::kPitch + c) = hi;
-        *reinterpret_cast<uint32_t *>(qs + (16 + r) * S::kPitch + c) = lo;
-    }
     float o[kTilesPerWarp][4];
 #pragma unroll
     for (int n = 0; n < kTilesPerWarp; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-    const uint32_t q_addr = (uint32_t)__cvta_generic_to_shared(
-        qs + ((lane & 7) + ((lane >> 3) & 1) * 8) * S::kPitch + (lane >> 4) * 8);
-    for (uint32_t k0 = 0, buf = 0; k0 < keys.count; k0 += kLatKeys, buf ^= 1) {
-        if (k0 + kLatKeys < keys.count) {
-            fetch(k0 + kLatKeys, buf ^ 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
-        }
-        __syncthreads();  // the tile (and, the first time, the query) is in place
-        const uint32_t tile = (uint32_t)__cvta_generic_to_shared(tiles + buf * S::kTileBytes);
-        float s[2][4] = {};  // two chains
-#pragma unroll 4
-        for (int ks = 0; ks < KV / 32; ++ks) {
-            uint32_t b[4];  // eight keys x 32 channels
-            lt_ldsm4(b, tile + ((warp * 8 + (lane & 7)) * S::kPitch + ks * 32 + (lane >> 3) * 8) * 2);
+#pragma unroll 1
+    for (uint32_t tile_i = 0; tile_i < n_tiles; ++tile_i) {
+        const uint32_t k0 = tile_i * kLatKeys;
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncwarp();  // the warp's tile is in place, and it is done with the one before
+        fetch(tile_i + 1);
+        const uint32_t tile = (uint32_t)__cvta_generic_to_shared(ring + (tile_i % S::kBufs) * S::kTileBytes);
+        float s[4][4], s2[4][4];  // (a chain per term)
 #pragma unroll
-            for (int term = 0; term < 2; ++term)
+        for (int n = 0; n < 4; ++n)
 #pragma unroll
-                for (int half = 0; half < 2; ++half) {
-                    uint32_t q[4];
-                    lt_ldsm4(q, q_addr + (term * 16 * S::kPitch + ks * 32 + half * 16) * 2);
-                    lt_mma(s[half], q, b[half * 2], b[half * 2 + 1]);
-                }
-        }
+            for (int e = 0; e < 4; ++e) s[n][e] = s2[n][e] = 0.f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const uint32_t key = warp * 8 + 2 * c4 + (e & 1);
-            sc[(g + (e >> 1) * 8) * kScPitch + key] = k0 + key < keys.count ? s[0][e] + s[1][e] : -INFINITY;
-        }
-        __syncthreads();
+        for (int ks = 0; ks < kSteps; ++ks)
+#pragma unroll
+            for (int pr = 0; pr < 2; ++pr) {
+                uint32_t b[4];  // two tiles of eight keys x 16 channels
+                lt_ldsm4(b, tile + (((2 * pr + (lane >> 4)) * 8 + (lane & 7)) * S::kPitch + ks * 16 +
+                                    ((lane >> 3) & 1) * 8) * 2);
+                lt_mma(s[2 * pr], qh[ks], b[0], b[1]);
+                lt_mma(s[2 * pr + 1], qh[ks], b[2], b[3]);
+                lt_mma(s2[2 * pr], ql[ks], b[0], b[1]);
+                lt_mma(s2[2 * pr + 1], ql[ks], b[2], b[3]);
+            }
+        float *sc = scores + (tile_i & 1) * 4 * 16 * S::kScorePitch;
+#pragma unroll
+        for (int n = 0; n < 4; ++n)
+#pragma unroll
+            for (int r = 0; r < 2; ++r)
+                *reinterpret_cast<float2 *>(sc + (warp * 16 + g + 8 * r) * S::kScorePitch + n * 8 + 2 * c4) =
+                    make_float2(s[n][2 * r] + s2[n][2 * r], s[n][2 * r + 1] + s2[n][2 * r + 1]);
+        __syncthreads();  // (the other of the two score buffers is free: every warp is past its reads)
         // every warp forms the weights of all 32 keys for rows g and g + 8
         float v[2][2][4];  // [row][16-key step][2 c4, 2 c4 + 1, 2 c4 + 8, 2 c4 + 9]
         float alpha[2];
@@ -302,13 +343,21 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
         for (int r = 0; r < 2; ++r) {
             float mx = m[r];
 #pragma unroll
-            for (int kk = 0; kk < 2; ++kk) {
-                const float2 x = *reinterpret_cast<const float2 *>(sc + (g + 8 * r) * kScPitch + kk * 16 + 2 * c4);
-                const float2 y = *reinterpret_cast<const float2 *>(sc + (g + 8 * r) * kScPitch + kk * 16 + 2 * c4 + 8);
-                v[r][kk][0] = x.x; v[r][kk][1] = x.y; v[r][kk][2] = y.x; v[r][kk][3] = y.y;
+            for (int kk = 0; kk < 2; ++kk)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) mx = fmaxf(mx, v[r][kk][e]);
-            }
+                for (int half = 0; half < 2; ++half) {
+                    const uint32_t key = kk * 16 + half * 8 + 2 * c4;
+                    float2 x = make_float2(0.f, 0.f);
+#pragma unroll
+                    for (int w = 0; w < 4; ++w) {
+                        const float2 y = *reinterpret_cast<const float2 *>(sc + (w * 16 + g + 8 * r) * S::kScorePitch + key);
+                        x.x += y.x;
+                        x.y += y.y;
+                    }
+                    v[r][kk][2 * half] = k0 + key < keys.count ? x.x : -INFINITY;
+                    v[r][kk][2 * half + 1] = k0 + key + 1 < keys.count ? x.y : -INFINITY;
+                    mx = fmaxf(mx, fmaxf(v[r][kk][2 * half], v[r][kk][2 * half + 1]));
+                }
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
             mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
             alpha[r] = m[r] == -INFINITY ? 0.f : expf(m[r] - mx);  // (every tile has a live key: mx is finite)
@@ -340,21 +389,21 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
             for (int n = 0; n < kTilesPerWarp; n += 2) {
                 uint32_t b[4];
                 lt_ldsm4_trans(b, tile + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kPitch +
-                                          warp * (KV / 4) + (n + (lane >> 4)) * 8) * 2);
+                                          (n + (lane >> 4)) * 8) * 2);
                 lt_mma(o[n], ph, b[0], b[1]);
-                lt_mma(o[n], pl, b[0], b[1]);
                 lt_mma(o[n + 1], ph, b[2], b[3]);
+                lt_mma(o[n], pl, b[0], b[1]);
                 lt_mma(o[n + 1], pl, b[2], b[3]);
             }
         }
-        __syncthreads();  // the buffers may be filled again
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
     // The splits of a cluster are merged here: every CTA leaves its sums, maxima and weights in its
     // shared memory (the tiles are idle) and each finishes a share of the channels.
     float *sums = reinterpret_cast<float *>(lat_smem);  // [16][KV + 4]
     constexpr int kSumPitch = KV + 4;
     float *stat = sums + 16 * kSumPitch;                // [2][16]: maximum, weight
-    static_assert((16 * kSumPitch + 32) * 4 <= S::kQBytes + 2 * S::kTileBytes, "the sums must fit the tiles");
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
         l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
@@ -405,59 +454,90 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
 }
 
 // ------------------------------------------------------------------ absorbed: combine, W_uv
+// A block takes kRows rows of one head: the weights are read once for all of them.
 constexpr int kOutThreads = 256;
-template <typename W>
+template <typename W, int kRows>
 __global__ void __launch_bounds__(kOutThreads)
 latent_output_kernel(LatentArgs a, const W *__restrict__ uv, uint32_t per_block) {
     qk::pdl_launch();
-    qk::pdl_wait();
-    extern __shared__ __align__(16) float lo_smem[];  // [kv_stride] combined latent, [n_splits] weights
-    float *lat = lo_smem, *wt = lo_smem + a.kv_stride;
-    const uint32_t h = blockIdx.x, t = blockIdx.z, warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-    const uint32_t j0 = blockIdx.y * per_block, j1 = min(j0 + per_block, a.vdim);
-    if (a.positions[t] < 0) {
-        for (uint32_t j = j0 + threadIdx.x; j < j1; j += kOutThreads)
-            put(a.out, a.out_bf16, (size_t)t * a.out_stride + h * a.vdim + j, 0.f);
-        return;
+    {   // the weights depend on no other kernel: on their way to L2 before the dependency wait
+        const uint32_t first = blockIdx.y * per_block, n = min(per_block, a.vdim - min(first, a.vdim));
+        const uint8_t *w = reinterpret_cast<const uint8_t *>(uv + ((size_t)blockIdx.x * a.vdim_stride + first) * a.kv_stride);
+        for (uint32_t i = threadIdx.x * 128; i < n * a.kv_stride * (uint32_t)sizeof(W); i += kOutThreads * 128)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(w + i));
     }
-    const float *src = a.partial + ((size_t)t * a.heads + h) * a.n_splits * (a.kv_stride + 8);
-    const uint32_t pitch = a.kv_stride + 8;
-    if (warp == 0) {
-        float m = -INFINITY;
-        for (uint32_t s = lane; s < a.n_splits; s += 32) m = fmaxf(m, src[(size_t)s * pitch + a.kv_stride]);
+    qk::pdl_wait();
+    extern __shared__ __align__(16) float lo_smem[];  // [kRows][kv_stride] combined latents, [kRows][n_splits] weights
+    float *lat = lo_smem, *wt = lo_smem + kRows * a.kv_stride;
+    const uint32_t h = blockIdx.x, t0 = blockIdx.z * kRows, warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const uint32_t j0 = blockIdx.y * per_block, j1 = min(j0 + per_block, a.vdim), pitch = a.kv_stride + 8;
+    // a warp per row forms its splits' weights (and with several rows its combined latent as well)
+    for (uint32_t r = warp; r < (uint32_t)kRows; r += kOutThreads / 32) {
+        const uint32_t t = t0 + r;
+        const bool live = t < a.tokens && a.positions[t] >= 0;  // (an idle row's output is zero)
+        const float *src = a.partial + ((size_t)min(t, a.tokens - 1) * a.heads + h) * a.n_splits * pitch;
+        float m = -INFINITY, l = 0.f;
+        for (uint32_t s = lane; s < a.n_splits && live; s += 32) m = fmaxf(m, src[(size_t)s * pitch + a.kv_stride]);
         for (int off = 16; off > 0; off >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, off));
-        float l = 0.f;
         for (uint32_t s = lane; s < a.n_splits; s += 32) {
-            const float ms = src[(size_t)s * pitch + a.kv_stride];
+            const float ms = live ? src[(size_t)s * pitch + a.kv_stride] : -INFINITY;
             const float e = ms == -INFINITY ? 0.f : expf(ms - m);
-            wt[s] = e;
-            l += e * src[(size_t)s * pitch + a.kv_stride + 1];
+            wt[r * a.n_splits + s] = e;
+            if (e != 0.f) l += e * src[(size_t)s * pitch + a.kv_stride + 1];
         }
         for (int off = 16; off > 0; off >>= 1) l += __shfl_xor_sync(0xffffffffu, l, off);
-        for (uint32_t s = lane; s < a.n_splits; s += 32) wt[s] /= l;
+        for (uint32_t s = lane; s < a.n_splits && live; s += 32) wt[r * a.n_splits + s] /= l;
+        __syncwarp();
+        if constexpr (kRows > 1)
+#pragma unroll 4
+            for (uint32_t i = lane * 4; i < a.kv_stride; i += 128) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (uint32_t s = 0; s < a.n_splits; ++s) {
+                    const float e = wt[r * a.n_splits + s];
+                    if (e == 0.f) continue;  // (an empty split holds no sums)
+                    const float4 x = *reinterpret_cast<const float4 *>(src + (size_t)s * pitch + i);
+                    v = make_float4(fmaf(e, x.x, v.x), fmaf(e, x.y, v.y), fmaf(e, x.z, v.z), fmaf(e, x.w, v.w));
+                }
+                *reinterpret_cast<float4 *>(lat + r * a.kv_stride + i) = v;
+            }
     }
     __syncthreads();
-    for (uint32_t i = threadIdx.x; i < a.kv_stride; i += kOutThreads) {
-        float v = 0.f;
+    if constexpr (kRows == 1) {  // one row: the whole block combines it
+        const float *src = a.partial + ((size_t)t0 * a.heads + h) * a.n_splits * pitch;
+        for (uint32_t i = threadIdx.x; i < a.kv_stride; i += kOutThreads) {
+            float v = 0.f;
 #pragma unroll 8
-        for (uint32_t s = 0; s < a.n_splits; ++s) {
-            const float e = wt[s];
-            if (e != 0.f) v = fmaf(e, src[(size_t)s * pitch + i], v);  // (an empty split holds no sums)
+            for (uint32_t s = 0; s < a.n_splits; ++s) {
+                const float e = wt[s];
+                if (e != 0.f) v = fmaf(e, src[(size_t)s * pitch + i], v);
+            }
+            lat[i] = v;
         }
-        lat[i] = v;
+        __syncthreads();
     }
-    __syncthreads();
     for (uint32_t j = j0 + warp; j < j1; j += kOutThreads / 32) {
         const W *row = uv + ((size_t)h * a.vdim_stride + j) * a.kv_stride;
-        float v = 0.f;
+        float v[kRows];
+#pragma unroll
+        for (int r = 0; r < kRows; ++r) v[r] = 0.f;
+#pragma unroll 2
         for (uint32_t i = lane * 8; i < a.kv_stride; i += 256) {
             float w[8];
             lt_load8(row + i, w);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v = fmaf(w[e], lat[i + e], v);
+            for (int r = 0; r < kRows; ++r) {
+                const float4 x = *reinterpret_cast<const float4 *>(lat + r * a.kv_stride + i);
+                const float4 y = *reinterpret_cast<const float4 *>(lat + r * a.kv_stride + i + 4);
+                v[r] = fmaf(w[0], x.x, fmaf(w[1], x.y, fmaf(w[2], x.z, fmaf(w[3], x.w, v[r]))));
+                v[r] = fmaf(w[4], y.x, fmaf(w[5], y.y, fmaf(w[6], y.z, fmaf(w[7], y.w, v[r]))));
+            }
         }
-        for (int off = 16; off > 0; off >>= 1) v += __shfl_xor_sync(0xffffffffu, v, off);
-        if (lane == 0) put(a.out, a.out_bf16, (size_t)t * a.out_stride + h * a.vdim + j, v);
+#pragma unroll
+        for (int r = 0; r < kRows; ++r) {
+            for (int off = 16; off > 0; off >>= 1) v[r] += __shfl_xor_sync(0xffffffffu, v[r], off);
+            if (lane == 0 && t0 + r < a.tokens)
+                put(a.out, a.out_bf16, (size_t)(t0 + r) * a.out_stride + h * a.vdim + j, v[r]);
+        }
     }
 }
 
@@ -739,8 +819,10 @@ qk_status qk_latent_attention(qk_ctx *ctx, const qk_latent_call *d) {
     a.out_bf16 = d->out_dtype == QK_BF16;
     const bool bf16 = d->w_dtype == QK_BF16;
     const dim3 ag((unsigned)qk::ceil_div(d->kv_stride, 256), (unsigned)d->heads, (unsigned)qk::ceil_div(d->tokens, kAbsRows));
-    if (bf16) QK_LAUNCH(c, absorb_query_kernel<uint16_t>, ag, dim3(kAbsWarps * 32), 0, a, (const uint16_t *)d->uk);
-    else QK_LAUNCH(c, absorb_query_kernel<float>, ag, dim3(kAbsWarps * 32), 0, a, (const float *)d->uk);
+    const size_t ab_smem = (kAbsRows * d->dim + kAbsWarps * 256) * 4;
+    if (ab_smem > 48 * 1024) return qk::fail(QK_ERR_VALUE, "qk_latent_attention: dim %zu does not fit shared memory", d->dim);
+    if (bf16) QK_LAUNCH(c, absorb_query_kernel<uint16_t>, ag, dim3(kAbsWarps * 32), ab_smem, a, (const uint16_t *)d->uk);
+    else QK_LAUNCH(c, absorb_query_kernel<float>, ag, dim3(kAbsWarps * 32), ab_smem, a, (const float *)d->uk);
     if (bf16 && d->kv_stride <= 512 && c->decode_attention_kernel != 0) {
         const uint16_t *cache = (const uint16_t *)d->cache;
         const uint32_t cluster = a.n_splits % 8 == 0 ? 8 : a.n_splits % 4 == 0 ? 4 : a.n_splits % 2 == 0 ? 2 : 1;
@@ -761,18 +843,24 @@ qk_status qk_latent_attention(qk_ctx *ctx, const qk_latent_call *d) {
             QK_LAUNCH(c, latent_plain_kernel<float>, pg, dim3(kPlainThreads), smem, a, (const float *)d->cache);
         }
     }
-    // few rows: several blocks share the value channels of a head
+    // few rows: several blocks share the value channels of a head; many: a block takes eight rows
+    const bool tiled = d->tokens >= 16;
     const uint32_t parts = d->tokens * d->heads >= 256 ? 1u : (uint32_t)std::min<size_t>(4, qk::ceil_div(d->vdim, 16));
-    const uint32_t per = (uint32_t)qk::ceil_div(d->vdim, parts);
-    const dim3 og(a.heads, parts, a.tokens);
-    const size_t smem = (d->kv_stride + d->n_splits) * 4;
-    if (bf16) {
-        QK_CUDA(cudaFuncSetAttribute(latent_output_kernel<uint16_t>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        QK_LAUNCH(c, latent_output_kernel<uint16_t>, og, dim3(kOutThreads), smem, a, (const uint16_t *)d->uv, per);
-    } else {
-        QK_CUDA(cudaFuncSetAttribute(latent_output_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-        QK_LAUNCH(c, latent_output_kernel<float>, og, dim3(kOutThreads), smem, a, (const float *)d->uv, per);
-    }
+    const uint32_t per = (uint32_t)qk::ceil_div(d->vdim, parts), rows = tiled ? 8 : 1;
+    const dim3 og(a.heads, parts, (a.tokens + rows - 1) / rows);
+    const size_t smem = rows * (d->kv_stride + a.n_splits) * 4;
+    if (smem > 200 * 1024)
+        return qk::fail(QK_ERR_VALUE, "qk_latent_attention: a latent of %zu entries does not fit shared memory", d->kv_stride);
+#define QK_LATENT_OUT(W, R)                                                                                                 \
+    do {                                                                                                                    \
+        QK_CUDA(cudaFuncSetAttribute(latent_output_kernel<W, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
+        QK_LAUNCH(c, (latent_output_kernel<W, R>), og, dim3(kOutThreads), smem, a, (const W *)d->uv, per);                  \
+    } while (0)
+    if (bf16 && tiled) QK_LATENT_OUT(uint16_t, 8);
+    else if (bf16) QK_LATENT_OUT(uint16_t, 1);
+    else if (tiled) QK_LATENT_OUT(float, 8);
+    else QK_LATENT_OUT(float, 1);
+#undef QK_LATENT_OUT
     return QK_OK;
 }
 
