@@ -255,7 +255,8 @@ __device__ __forceinline__ float4 lat_peer4(const float *p, uint32_t cta) {
                  : "memory");
     return v;
 }
-template <int KV>
+// TERMS: bfloat16 terms of the query and of the weights (two keep float32 accuracy).
+template <int KV, int TERMS>
 __global__ void __launch_bounds__(128)
 latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t cluster) {
     using S = LatShape<KV>;
@@ -325,8 +326,10 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
                                     ((lane >> 3) & 1) * 8) * 2);
                 lt_mma(s[2 * pr], qh[ks], b[0], b[1]);
                 lt_mma(s[2 * pr + 1], qh[ks], b[2], b[3]);
-                lt_mma(s2[2 * pr], ql[ks], b[0], b[1]);
-                lt_mma(s2[2 * pr + 1], ql[ks], b[2], b[3]);
+                if constexpr (TERMS == 2) {
+                    lt_mma(s2[2 * pr], ql[ks], b[0], b[1]);
+                    lt_mma(s2[2 * pr + 1], ql[ks], b[2], b[3]);
+                }
             }
         float *sc = scores + (tile_i & 1) * 4 * 16 * S::kScorePitch;
 #pragma unroll
@@ -392,8 +395,10 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
                                           (n + (lane >> 4)) * 8) * 2);
                 lt_mma(o[n], ph, b[0], b[1]);
                 lt_mma(o[n + 1], ph, b[2], b[3]);
-                lt_mma(o[n], pl, b[0], b[1]);
-                lt_mma(o[n + 1], pl, b[2], b[3]);
+                if constexpr (TERMS == 2) {
+                    lt_mma(o[n], pl, b[0], b[1]);
+                    lt_mma(o[n + 1], pl, b[2], b[3]);
+                }
             }
         }
     }
@@ -538,6 +543,74 @@ latent_output_kernel(LatentArgs a, const W *__restrict__ uv, uint32_t per_block)
             if (lane == 0 && t0 + r < a.tokens)
                 put(a.out, a.out_bf16, (size_t)(t0 + r) * a.out_stride + h * a.vdim + j, v[r]);
         }
+    }
+}
+
+// The same for 16 rows of one head on the tensor cores (bfloat16 weights): the combined latents, in
+// two bfloat16 terms, are the M side, the value channels the N side, 16 per warp.
+template <int TERMS>
+__global__ void __launch_bounds__(kOutThreads)
+latent_output_mma_kernel(LatentArgs a, const uint16_t *__restrict__ uv) {
+    qk::pdl_launch();
+    qk::pdl_wait();
+    extern __shared__ __align__(16) uint8_t om_smem[];  // [TERMS][16][kv_stride + 8] bfloat16
+    uint16_t *lat = reinterpret_cast<uint16_t *>(om_smem);
+    const uint32_t h = blockIdx.x, t0 = blockIdx.y * 16, warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const uint32_t g = lane >> 2, c4 = lane & 3, lp = a.kv_stride + 8, pitch = a.kv_stride + 8;
+    for (uint32_t r = warp; r < 16; r += kOutThreads / 32) {
+        const uint32_t t = t0 + r;
+        const bool live = t < a.tokens && a.positions[t] >= 0;  // (an idle row's output is zero)
+        const float *src = a.partial + ((size_t)min(t, a.tokens - 1) * a.heads + h) * a.n_splits * pitch;
+        float m = -INFINITY, l = 0.f;
+        for (uint32_t s = 0; s < a.n_splits && live; ++s) m = fmaxf(m, src[(size_t)s * pitch + a.kv_stride]);
+        for (uint32_t s = 0; s < a.n_splits && live; ++s) {
+            const float ms = src[(size_t)s * pitch + a.kv_stride];
+            if (ms != -INFINITY) l += expf(ms - m) * src[(size_t)s * pitch + a.kv_stride + 1];
+        }
+        for (uint32_t i = lane * 2; i < a.kv_stride; i += 64) {
+            float x = 0.f, y = 0.f;
+            for (uint32_t s = 0; s < a.n_splits && live; ++s) {
+                const float ms = src[(size_t)s * pitch + a.kv_stride];
+                if (ms == -INFINITY) continue;  // (an empty split holds no sums)
+                const float e = expf(ms - m) / l;
+                const float2 v = *reinterpret_cast<const float2 *>(src + (size_t)s * pitch + i);
+                x = fmaf(e, v.x, x);
+                y = fmaf(e, v.y, y);
+            }
+            uint32_t hi, lo;
+            lt_split2(x, y, hi, lo);
+            *reinterpret_cast<uint32_t *>(lat + r * lp + i) = hi;
+            if constexpr (TERMS == 2) *reinterpret_cast<uint32_t *>(lat + (16 + r) * lp + i) = lo;
+        }
+    }
+    __syncthreads();
+    const uint32_t a_addr = (uint32_t)__cvta_generic_to_shared(lat + ((lane & 7) + ((lane >> 3) & 1) * 8) * lp + (lane >> 4) * 8);
+    for (uint32_t j0 = warp * 16; j0 < a.vdim; j0 += kOutThreads / 32 * 16) {
+        const uint32_t *row[2];
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+            row[n] = reinterpret_cast<const uint32_t *>(
+                uv + ((size_t)h * a.vdim_stride + min(j0 + n * 8 + g, a.vdim_stride - 1)) * a.kv_stride) + c4;
+        float acc[2][4] = {};
+#pragma unroll 8
+        for (uint32_t k = 0; k < a.kv_stride; k += 16) {  // (kv_stride is a multiple of 16 here)
+            uint32_t x[4], y[4];
+            lt_ldsm4(x, a_addr + k * 2);
+            if constexpr (TERMS == 2) lt_ldsm4(y, a_addr + (16 * lp + k) * 2);
+#pragma unroll
+            for (int n = 0; n < 2; ++n) {
+                const uint32_t b0 = row[n][k / 2], b1 = row[n][k / 2 + 4];
+                lt_mma(acc[n], x, b0, b1);
+                if constexpr (TERMS == 2) lt_mma(acc[n], y, b0, b1);
+            }
+        }
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const uint32_t t = t0 + g + (e >> 1) * 8, j = j0 + n * 8 + 2 * c4 + (e & 1);
+                if (t < a.tokens && j < a.vdim) put(a.out, a.out_bf16, (size_t)t * a.out_stride + h * a.vdim + j, acc[n][e]);
+            }
     }
 }
 
@@ -733,16 +806,19 @@ qk_status enter(qk_ctx *ctx, qk_ctx **c) {
     QK_CUDA(cudaSetDevice((*c)->device));
     return QK_OK;
 }
+// With many rows a kernel is launched only when the one before it has finished: blocks that come in
+// early crowd on the SMs that have room at that moment, and stay there.
+constexpr uint32_t kFewRows = 8, kManyRows = 16;
 #define QK_LAUNCH(c, kernel, grid, block, smem, ...)                                                   \
     do {                                                                                               \
-        (void)qk::launch_pdl((c)->pdl, kernel, grid, block, smem, (c)->stream, __VA_ARGS__);           \
+        (void)qk::launch_pdl((c)->pdl && a.tokens <= kFewRows, kernel, grid, block, smem, (c)->stream, __VA_ARGS__);           \
         QK_CUDA(cudaGetLastError());                                                                   \
         (c)->launches++;                                                                               \
     } while (0)
 
-template <int KV>
-qk_status launch_mma(qk_ctx *c, const LatentArgs &a, const uint16_t *cache, uint32_t cluster) {
-    QK_CUDA(cudaFuncSetAttribute(latent_mma_kernel<KV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+template <int KV, int TERMS>
+qk_status launch_mma_terms(qk_ctx *c, const LatentArgs &a, const uint16_t *cache, uint32_t cluster) {
+    QK_CUDA(cudaFuncSetAttribute((latent_mma_kernel<KV, TERMS>), cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)LatShape<KV>::kSmem));
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(a.n_splits, (a.heads + 15) / 16, a.tokens);
@@ -751,15 +827,20 @@ qk_status launch_mma(qk_ctx *c, const LatentArgs &a, const uint16_t *cache, uint
     cfg.stream = c->stream;
     cudaLaunchAttribute attr[2];
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = c->pdl ? 1 : 0;
+    attr[0].val.programmaticStreamSerializationAllowed = c->pdl && a.tokens <= kFewRows ? 1 : 0;
     attr[1].id = cudaLaunchAttributeClusterDimension;
     attr[1].val.clusterDim.x = cluster;
     attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = 2;
-    QK_CUDA(cudaLaunchKernelEx(&cfg, latent_mma_kernel<KV>, a, cache, cluster));
+    QK_CUDA(cudaLaunchKernelEx(&cfg, (latent_mma_kernel<KV, TERMS>), a, cache, cluster));
     c->launches++;
     return QK_OK;
+}
+
+template <int KV>
+qk_status launch_mma(qk_ctx *c, const LatentArgs &a, const uint16_t *cache, uint32_t cluster) {
+    return a.tokens < kManyRows ? launch_mma_terms<KV, 2>(c, a, cache, cluster) : launch_mma_terms<KV, 1>(c, a, cache, cluster);
 }
 
 template <int DK, int DV>
@@ -856,7 +937,12 @@ qk_status qk_latent_attention(qk_ctx *ctx, const qk_latent_call *d) {
         QK_CUDA(cudaFuncSetAttribute(latent_output_kernel<W, R>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)); \
         QK_LAUNCH(c, (latent_output_kernel<W, R>), og, dim3(kOutThreads), smem, a, (const W *)d->uv, per);                  \
     } while (0)
-    if (bf16 && tiled) QK_LATENT_OUT(uint16_t, 8);
+    const size_t mma_smem = 2 * 16 * (d->kv_stride + 8) * 2;
+    if (bf16 && tiled && d->kv_stride % 16 == 0 && mma_smem <= 200 * 1024 && c->decode_attention_kernel != 0) {
+        QK_CUDA(cudaFuncSetAttribute(latent_output_mma_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        QK_LAUNCH(c, latent_output_mma_kernel<2>, dim3(a.heads, (a.tokens + 15) / 16), dim3(kOutThreads), mma_smem, a,
+                  (const uint16_t *)d->uv);
+    } else if (bf16 && tiled) QK_LATENT_OUT(uint16_t, 8);
     else if (bf16) QK_LATENT_OUT(uint16_t, 1);
     else if (tiled) QK_LATENT_OUT(float, 8);
     else QK_LATENT_OUT(float, 1);
@@ -873,6 +959,7 @@ qk_status qk_latent_gather(qk_ctx *ctx, const void *cache, int32_t dtype, size_t
     if (!cache || !out || bytes % 16 || count > ring)
         return qk::fail(QK_ERR_VALUE, "qk_latent_gather: %zu rows of %zu bytes from a ring of %zu", count, bytes, ring);
     if (count == 0) return QK_OK;
+    const struct { uint32_t tokens; } a{(uint32_t)count};
     QK_LAUNCH(c, latent_gather_kernel, dim3((unsigned)count), dim3(128), 0, (const uint4 *)cache, (uint32_t)ring,
               (uint32_t)(bytes / 16), (uint32_t)slot, (uint32_t)first, (uint4 *)out);
     return QK_OK;
