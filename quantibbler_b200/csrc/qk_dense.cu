@@ -78,8 +78,9 @@ __device__ __forceinline__ void vec_fma(float (&acc)[NT], const uint4 &w, const 
 
 // A warp (or `ksplit` warps that share out the k range) owns R weight rows; with a gated pair,
 // R / 2 gate rows and their up rows.
+// (The blocks per SM matter more than a spilled register: they hide each other's prologues.)
 template <typename W, int NT, int R>
-__global__ void __launch_bounds__(kVecThreads)
+__global__ void __launch_bounds__(kVecThreads, NT == 4 && R == 4 ? 2 : R == 1 && NT <= 2 ? 4 : 3)
 dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint32_t rows, uint32_t w_stride,
                     uint32_t n_tokens, uint32_t ksplit) {
     using T = VecTraits<W>;
@@ -1015,8 +1016,9 @@ qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out,
 template <typename W, int NT>
 qk_status launch_vector(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
                         size_t n_tokens) {
-    // rows per warp and warps per row group: about two blocks per SM or more
-    const size_t want = 2 * (size_t)c->sm_count * kVecWarps, steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
+    // rows per warp and warps per row group: about two blocks per SM or more (one, where a block
+    // has a long vector to stage first)
+    const size_t want = (d.k > 8192 ? 1 : 2) * (size_t)c->sm_count * kVecWarps, steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
     const bool pair = d.output == QK_OUTPUT_GLU;
     if (d.rows / 4 >= want) return launch_vector_r<W, NT, 4>(c, in, out, d, n_tokens, 1);
     if (d.rows / 2 >= want || pair) {

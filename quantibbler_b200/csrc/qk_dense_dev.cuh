@@ -50,10 +50,9 @@ struct OutputArgs {
 // The sum over a block of `kInThreads` threads; `red` holds one float per warp.
 __device__ __forceinline__ float in_block_sum(float v, float *red) { return block_sum(v, red); }
 
-// kBatch values per thread are requested together before any of them is used: these loops are
+// kInBatch values per thread are requested together before any of them is used: these loops are
 // pure latency when a step has one row.
-constexpr int kInBatch = 8;
-template <typename F>
+template <int kInBatch = 8, typename F>
 __device__ __forceinline__ void in_load(const float *__restrict__ p, uint32_t n, F &&use) {
     for (uint32_t base = threadIdx.x; base < n; base += kInBatch * blockDim.x) {
         float v[kInBatch];
@@ -75,7 +74,7 @@ __device__ __forceinline__ void build_input(const InputArgs &a, uint32_t t, bool
     const uint32_t n = a.width;
     const float *xr = a.x + (size_t)t * a.x_stride;
     if (a.kind == QK_INPUT_PLAIN) {
-        in_load(xr, n, [&](uint32_t i, float v) { at(i) = v; });
+        in_load<16>(xr, n, [&](uint32_t i, float v) { at(i) = v; });
         for (uint32_t i = n + threadIdx.x; i < a.k; i += blockDim.x) at(i) = 0.f;
         __syncthreads();
         return;
