@@ -349,3 +349,18 @@ def test_trace_runner(gpu_ctx, tmp_path, serving):
             want[name][i], expected = row, want[name].copy()
             assert_rows(want[name], expected, lims[name], f"step {n}")
             want[name] = expected
+
+
+def test_command_line_generates(gpu_ctx, tmp_path):
+    cfg = vm.mixed()
+    w = vm.weights(cfg, 22)
+    vm.write_model(tmp_path, cfg, w)
+    prompt = vm.prompt(cfg, 19)
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    p = subprocess.run([sys.executable, "-m", "quantibbler_b200", "generate", "--model", str(tmp_path), "--dtype", "float32",
+                        "--prompt", ",".join(map(str, prompt)), "--max-tokens", "6"], cwd=root, capture_output=True,
+                       text=True, timeout=300)
+    assert p.returncode == 0, p.stderr[-2000:]
+    out = json.loads(p.stdout)
+    assert out["prompt_tokens"] == 19 and out["finish"] == "length"
+    agree(out["completion_tokens"], greedy_oracle(cfg, w, prompt, 6), "float32")
