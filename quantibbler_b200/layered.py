@@ -10,7 +10,7 @@ leaves behind in a slot is never read by the next one (positions decide what is 
 from __future__ import annotations
 
 import ctypes
-from dataclasses import dataclass, field
+from dataclasses import dataclass
 
 import numpy as np
 
@@ -49,7 +49,6 @@ class LayeredConfig:
     prefill_min_tokens: int = 2
     prefill_chunk: int = 2048
     vector_rows: int = 4                    # portions this short keep float32 activations
-    extras: dict = field(default_factory=dict)
 
     def run_order(self) -> list:
         """[(layer, starts a pass)] in running order."""
