@@ -550,6 +550,10 @@ qk_status qk_embed(qk_ctx *ctx, const void *table, int32_t table_dtype, const in
 qk_status qk_lm_head(qk_ctx *ctx, const float *hidden, const void *weight, int32_t weight_dtype,
                      size_t n_tokens, size_t vocab, size_t d, size_t logits_stride,
                      float *logits);
+/* The same with logits <- softcap * tanh(logits / softcap) (0: none).  No reference counterpart. */
+qk_status qk_lm_head_capped(qk_ctx *ctx, const float *hidden, const void *weight, int32_t weight_dtype,
+                            size_t n_tokens, size_t vocab, size_t d, size_t logits_stride, float softcap,
+                            float *logits);
 /* crates/quantibbler-server/src/sampler.rs:5-16 (greedy): the first maximum of each row;
  * out_idx is offset by index_base (for a vocabulary shard). */
 qk_status qk_argmax_first(qk_ctx *ctx, const float *logits, size_t n_tokens, size_t vocab,
@@ -627,10 +631,37 @@ typedef struct {
     const void *side;
     int32_t side_dtype;
     size_t side_stride, side_offset;
-    /* scratch for the input rows of the matrix forms: tokens * k * (2 or 4) bytes */
+    /* scratch for the input rows of the matrix forms: rows * k * (2 or 4) bytes, a row per token or,
+     * with experts, per choice */
     void *scratch;
     size_t scratch_bytes;
+    /* With pending_top > 0 the pending value's y of row t is the sum of pending_top rows of
+     * `pending` times pending_scale: rows pending_rows[t][..] (null: t * pending_top + ..). */
+    const int32_t *pending_rows;
+    size_t pending_top;
+    float pending_scale;
+    /* experts > 0: `w` holds [experts][rows][w_stride].  Row t has `top` choices, the experts
+     * table[ids[t]][..] ([vocab][top], all different); each gives an output row, at place
+     * t * top + j in the vector form, at places[t][j] (sorted by expert, see qk_route) in the others.
+     * by_choice: the input rows are such rows too (and plain), else every choice reads row t.
+     * QK_OUTPUT_STORE and QK_OUTPUT_GLU only. */
+    size_t experts, top;
+    int32_t by_choice;
+    const int32_t *table, *places, *offsets, *tiles;
 } qk_dense_call;
+/* Sorts the choices of `tokens` rows by expert, for n_jobs tables at once (one launch).  tiles:
+ * the number of tiles, then per tile its expert, first and last + 1 place, every tile at most
+ * tile_rows (qk_route_tile_rows) places of one expert; room for ceil(tokens * top / tile_rows) +
+ * experts tiles.  The launch lets no dependent kernel start early: a kernel after it may read
+ * these before its own dependency wait. */
+typedef struct {
+    const int32_t *table;                    /* [vocab][top] */
+    int32_t *places, *offsets, *tiles;       /* [tokens][top], [experts + 1], [1 + 3 * tiles] */
+    uint64_t top, experts;
+} qk_route_job;
+qk_status qk_route(qk_ctx *ctx, const qk_route_job *device_jobs, size_t n_jobs, size_t max_experts, const int32_t *ids,
+                   size_t tokens, size_t vocab, size_t tile_rows);
+size_t qk_route_tile_rows(size_t tokens, size_t k, int32_t w_dtype);
 /* One dense linear.  Up to QK_DENSE_VECTOR_TOKENS rows (qk_dense_form says which form a shape
  * takes) run as one launch that forms the input in every block; more rows as a launch for the
  * input (none for a plain input of the weights' dtype) and a matrix product. */
@@ -705,6 +736,46 @@ qk_status qk_window_attention(qk_ctx *ctx, const void *q, size_t q_stride, const
                               size_t key0, size_t n_keys, size_t first_position, size_t tokens, size_t heads,
                               size_t dim_stride, size_t vdim, size_t vdim_stride, size_t window, float scale,
                               void *out, size_t out_stride);
+
+/* Grouped causal attention over a full cache, with a query temperature and a distance bias:
+ * score(i, j) = (q_i . k_j) * scale * (1 + temp_coef * ln(floor((p_i + 1) / temp_every) + 1))
+ * + bias[head][min(p_i - p_j, bias_len - 1)] (temp_every 0: no temperature; bias null: none).
+ * Query head h reads key/value head h / (heads / kv_heads).  Projection rows hold
+ * q [heads][dim_stride] k [kv_heads][dim_stride] v [kv_heads][vdim_stride], entries past dim and
+ * vdim zero; the caches are [slots][kv_heads][s_max][dim_stride or vdim_stride]; out
+ * [tokens][heads][vdim_stride].  Strides are multiples of 16.  A row at position p sees cache rows
+ * 0 .. p of its slot; a row outside the cache is skipped and reported by qk_gpu_synchronize. */
+typedef struct {
+    size_t tokens;
+    const int32_t *positions, *slots;
+    size_t heads, kv_heads, dim_stride, vdim_stride, s_max, n_slots;
+    float scale, temp_coef;
+    double temp_every;
+    const float *bias;
+    size_t bias_len;
+    const void *proj;
+    int32_t proj_dtype;
+    size_t proj_stride;
+    int32_t cache_dtype;
+    void *cache_k, *cache_v;
+    size_t n_splits;
+    float *scratch;                          /* qk_grouped_scratch() bytes, zeroed once by the caller */
+    void *out;
+    int32_t out_dtype;
+    size_t out_stride;
+    /* qk_grouped_attention: rows of different slots, one each: their keys and values are appended
+     * by the attention itself.  0: qk_grouped_append has done it. */
+    int32_t append;
+    /* qk_grouped_portion: rows are positions first_position .. of one slot */
+    size_t slot, first_position;
+} qk_grouped_call;
+/* The rows' keys and values into the caches. */
+qk_status qk_grouped_append(qk_ctx *ctx, const qk_grouped_call *call);
+/* Any mix of rows (float32 projections), the keys split over n_splits blocks. */
+qk_status qk_grouped_attention(qk_ctx *ctx, const qk_grouped_call *call);
+size_t qk_grouped_scratch(size_t tokens, size_t heads, size_t kv_heads, size_t vdim_stride, size_t n_splits);
+/* One portion of one sequence (bfloat16 projections, caches and output; strides up to 256). */
+qk_status qk_grouped_portion(qk_ctx *ctx, const qk_grouped_call *call);
 
 /* Which GEMV kernel qk_layer_apply and the group calls use: 0 = sign-select SIMT, 1 = bit-sliced
  * INT8 tensor-core (default; many instances per launch run in the persistent streaming form),

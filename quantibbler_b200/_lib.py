@@ -128,6 +128,8 @@ _SIGNATURES = {
                            c_void_p]),
     "qk_lm_head": (c_int32, [c_void_p, c_void_p, c_void_p, c_int32, c_size_t, c_size_t, c_size_t,
                              c_size_t, c_void_p]),
+    "qk_lm_head_capped": (c_int32, [c_void_p, c_void_p, c_void_p, c_int32, c_size_t, c_size_t, c_size_t,
+                                    c_size_t, c_float, c_void_p]),
     "qk_argmax_first": (c_int32, [c_void_p, c_void_p, c_size_t, c_size_t, c_size_t, c_int32,
                                   c_void_p, c_void_p]),
     "qk_set_gemv_kernel": (c_int32, [c_void_p, c_int32]),
@@ -154,6 +156,12 @@ _SIGNATURES = {
                                        c_void_p, c_size_t, c_size_t, c_void_p, c_void_p, c_void_p,
                                        c_void_p, c_void_p, c_void_p, c_void_p]),
     "qk_dense": (c_int32, [c_void_p, c_void_p]),
+    "qk_route": (c_int32, [c_void_p, c_void_p, c_size_t, c_size_t, c_void_p, c_size_t, c_size_t, c_size_t]),
+    "qk_route_tile_rows": (c_size_t, [c_size_t, c_size_t, c_int32]),
+    "qk_grouped_append": (c_int32, [c_void_p, c_void_p]),
+    "qk_grouped_attention": (c_int32, [c_void_p, c_void_p]),
+    "qk_grouped_portion": (c_int32, [c_void_p, c_void_p]),
+    "qk_grouped_scratch": (c_size_t, [c_size_t, c_size_t, c_size_t, c_size_t, c_size_t]),
     "qk_dense_form": (c_int32, [c_size_t, c_size_t, c_int32]),
     "qk_dense_input": (c_int32, [c_void_p, c_void_p]),
     "qk_embed_scaled": (c_int32, [c_void_p, c_void_p, c_int32, c_size_t, c_void_p, c_void_p, c_size_t, c_size_t,

@@ -1006,11 +1006,13 @@ template <> struct HeadVec<float> {
     }
 };
 
+__device__ __forceinline__ float soft_capped(float v, float cap) { return cap > 0.f ? cap * tanhf(v / cap) : v; }
+
 template <typename W, int TT>
 __global__ void __launch_bounds__(256)
 lm_head_kernel(const float *__restrict__ hidden, const W *__restrict__ weight,
                float *__restrict__ logits, uint32_t n_tokens, uint32_t vocab, uint32_t d,
-               uint32_t vocab_stride) {
+               uint32_t vocab_stride, float softcap) {
     qk::pdl_launch();  // the next kernel may begin its prologue
     qk::pdl_wait();    // everything before this kernel on the stream is complete and visible
     constexpr int N = HeadVec<W>::kN;
@@ -1042,7 +1044,7 @@ lm_head_kernel(const float *__restrict__ hidden, const W *__restrict__ weight,
         for (int t = 0; t < TT; ++t) {
             float a = acc[t];
             for (int off = 16; off > 0; off >>= 1) a += __shfl_xor_sync(0xffffffffu, a, off);
-            if (lane == 0 && t0 + t < n_tokens) logits[(size_t)(t0 + t) * vocab_stride + v] = a;
+            if (lane == 0 && t0 + t < n_tokens) logits[(size_t)(t0 + t) * vocab_stride + v] = soft_capped(a, softcap);
         }
     }
 }
@@ -1196,7 +1198,7 @@ __global__ void __launch_bounds__(128)
 lm_head_mma_kernel(const uint16_t *__restrict__ hid_hi, const uint16_t *__restrict__ hid_lo,
                    const uint32_t *__restrict__ any_lo, const uint16_t *__restrict__ weight,
                    float *__restrict__ logits, uint32_t n_tokens, uint32_t vocab, uint32_t d,
-                   uint32_t vocab_stride) {
+                   uint32_t vocab_stride, float softcap) {
     qk::pdl_launch();  // the next kernel may begin its prologue
     qk::pdl_wait();    // everything before this kernel on the stream is complete and visible
     extern __shared__ __align__(16) uint16_t sm_head[];  // [2 buffers][hi, lo][8 NT][kHeadPitch]
@@ -1266,21 +1268,21 @@ lm_head_mma_kernel(const uint16_t *__restrict__ hid_hi, const uint16_t *__restri
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const uint32_t tok = tok0 + 8 * nt + 2 * t + (e & 1), v = v0 + (e >> 1) * 8;
-            if (tok < n_tokens && v < vocab) logits[(size_t)tok * vocab_stride + v] = acc[nt][e];
+            if (tok < n_tokens && v < vocab) logits[(size_t)tok * vocab_stride + v] = soft_capped(acc[nt][e], softcap);
         }
 }
 
 template <int NT>
 void launch_lm_head_mma(qk_ctx *c, const uint16_t *hi, const uint16_t *lo, const uint32_t *any_lo,
                         const uint16_t *weight, float *logits, size_t n_tokens, size_t vocab, size_t d,
-                        size_t stride) {
+                        size_t stride, float softcap) {
     const size_t smem = 2 * 2 * 8 * NT * kHeadPitch * sizeof(uint16_t);
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(lm_head_mma_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     dim3 grid((unsigned)qk::ceil_div(vocab, 64), (unsigned)qk::ceil_div(n_tokens, 8 * NT));
     QK_PDL(c, (lm_head_mma_kernel<NT>), dim3(grid), dim3(128), smem, hi, lo, any_lo, weight, logits,
                                                           (uint32_t)n_tokens, (uint32_t)vocab,
-                                                          (uint32_t)d, (uint32_t)stride);
+                                                          (uint32_t)d, (uint32_t)stride, softcap);
 }
 
 extern "C" {
@@ -1591,6 +1593,12 @@ qk_status qk_embed(qk_ctx *ctx, const void *table, int32_t table_dtype, const in
 qk_status qk_lm_head(qk_ctx *ctx, const float *hidden, const void *weight, int32_t weight_dtype,
                      size_t n_tokens, size_t vocab, size_t d, size_t logits_stride,
                      float *logits) {
+    return qk_lm_head_capped(ctx, hidden, weight, weight_dtype, n_tokens, vocab, d, logits_stride, 0.f, logits);
+}
+
+qk_status qk_lm_head_capped(qk_ctx *ctx, const float *hidden, const void *weight, int32_t weight_dtype,
+                            size_t n_tokens, size_t vocab, size_t d, size_t logits_stride, float softcap,
+                            float *logits) {
     qk_ctx *c;
     qk_status st = enter(ctx, &c);
     if (st != QK_OK) return st;
@@ -1601,11 +1609,11 @@ qk_status qk_lm_head(qk_ctx *ctx, const float *hidden, const void *weight, int32
         if (n_tokens == 1)
             QK_PDL(c, (lm_head_kernel<float, 1>), dim3(blocks), dim3(256), 0, 
                 hidden, (const float *)weight, logits, 1, (uint32_t)vocab, (uint32_t)d,
-                (uint32_t)logits_stride);
+                (uint32_t)logits_stride, softcap);
         else
             QK_PDL(c, (lm_head_kernel<float, 8>), dim3(blocks), dim3(256), 0, 
                 hidden, (const float *)weight, logits, (uint32_t)n_tokens, (uint32_t)vocab,
-                (uint32_t)d, (uint32_t)logits_stride);
+                (uint32_t)d, (uint32_t)logits_stride, softcap);
     } else if (weight_dtype == QK_BF16 && n_tokens >= 8 && d % 64 == 0) {
         // a batch: one pass over the head on the bf16 tensor cores
         const uint16_t *w = (const uint16_t *)weight;
@@ -1617,19 +1625,19 @@ qk_status qk_lm_head(qk_ctx *ctx, const float *hidden, const void *weight, int32
         QK_PDL(c, split_hidden_kernel, dim3((unsigned)qk::ceil_div(n, 256)), dim3(256), 0, hidden, hi, lo, any_lo, n);
         QK_CUDA(cudaGetLastError());
         c->launches++;
-        if (n_tokens <= 8) launch_lm_head_mma<1>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride);
-        else if (n_tokens <= 16) launch_lm_head_mma<2>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride);
-        else if (n_tokens <= 32) launch_lm_head_mma<4>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride);
-        else launch_lm_head_mma<8>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride);
+        if (n_tokens <= 8) launch_lm_head_mma<1>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride, softcap);
+        else if (n_tokens <= 16) launch_lm_head_mma<2>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride, softcap);
+        else if (n_tokens <= 32) launch_lm_head_mma<4>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride, softcap);
+        else launch_lm_head_mma<8>(c, hi, lo, any_lo, w, logits, n_tokens, vocab, d, logits_stride, softcap);
     } else if (weight_dtype == QK_BF16) {
         if (n_tokens == 1)
             QK_PDL(c, (lm_head_kernel<uint16_t, 1>), dim3(blocks), dim3(256), 0, 
                 hidden, (const uint16_t *)weight, logits, 1, (uint32_t)vocab, (uint32_t)d,
-                (uint32_t)logits_stride);
+                (uint32_t)logits_stride, softcap);
         else
             QK_PDL(c, (lm_head_kernel<uint16_t, 8>), dim3(blocks), dim3(256), 0, 
                 hidden, (const uint16_t *)weight, logits, (uint32_t)n_tokens, (uint32_t)vocab,
-                (uint32_t)d, (uint32_t)logits_stride);
+                (uint32_t)d, (uint32_t)logits_stride, softcap);
     } else {
         return qk::fail(QK_ERR_VALUE, "head dtype must be float32 or bfloat16, got tag %d",
                         weight_dtype);

@@ -82,7 +82,7 @@ __device__ __forceinline__ void vec_fma(float (&acc)[NT], const uint4 &w, const 
 template <typename W, int NT, int R>
 __global__ void __launch_bounds__(kVecThreads, NT == 4 && R == 4 ? 2 : R == 1 && NT <= 2 ? 4 : 3)
 dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint32_t rows, uint32_t w_stride,
-                    uint32_t n_tokens, uint32_t ksplit) {
+                    uint32_t n_tokens, uint32_t ksplit, ChoiceArgs ch) {
     using T = VecTraits<W>;
     constexpr int U = R >= 4 ? 2 : 4;  // steps in flight
     constexpr int HR = R >= 2 ? R / 2 : 1;
@@ -95,7 +95,17 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
     const uint32_t group = (blockIdx.x * kVecWarps + warp) / ksplit, part = warp % ksplit;
     const bool pair = out.kind == QK_OUTPUT_GLU;
     const W *row[R];
-    uint32_t r0 = group * R;
+    uint32_t r0 = group * R, t_in = 0, t_out = 0;  // first input and output row
+    bool writer = blockIdx.x == 0;
+    if (ch.table) {
+        // one choice of one token per block row (NT is 1).  The token ids are written by copies and
+        // ordinary launches in front of the step, none of which lets a kernel start early.
+        const uint32_t t = blockIdx.y / ch.top, id = (uint32_t)min(max(ch.ids[t], 0), (int)ch.vocab - 1);
+        w += (size_t)ch.table[(size_t)id * ch.top + blockIdx.y % ch.top] * rows * w_stride;
+        t_out = blockIdx.y;
+        t_in = ch.by_choice ? t_out : t;
+        writer = writer && blockIdx.y % ch.top == 0;
+    }
 #pragma unroll
     for (int r = 0; r < R; ++r) {
         uint32_t n;
@@ -118,7 +128,7 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
     for (uint32_t t = 0; t < (uint32_t)NT; ++t) {
         float *dst = xs + t * pitch;
         if (t < n_tokens) {
-            build_input(in, t, blockIdx.x == 0, [&](uint32_t i) -> float & { return dst[T::place(i)]; }, red);
+            build_input(in, t_in + t, writer, [&](uint32_t i) -> float & { return dst[T::place(i)]; }, red);
         }
         // what lies between k and the pitch meets zero weights; it must only be finite
         for (uint32_t i = (t < n_tokens ? k : 0) + threadIdx.x; i < pitch; i += kVecThreads) dst[T::place(i)] = 0.f;
@@ -176,7 +186,7 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
                     for (int t = 0; t < NT; ++t) {
                         const uint32_t j = group * (R / 2) + r;
                         if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && j < rows / 2)
-                            finish_pair(out, t, j, acc[r][t], acc[r + R / 2][t]);
+                            finish_pair(out, t_out + t, j, acc[r][t], acc[r + R / 2][t]);
                     }
             }
         } else {
@@ -185,7 +195,7 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
 #pragma unroll
                 for (int t = 0; t < NT; ++t)
                     if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && r0 + r < rows)
-                        finish(out, t, r0 + r, acc[r][t]);
+                        finish(out, t_out + t, r0 + r, acc[r][t]);
         }
     }
     if (in.append.src && blockIdx.x == gridDim.x - 1)
@@ -203,14 +213,16 @@ dense_input_kernel(InputArgs in, A *__restrict__ dst) {
     const uint32_t t = blockIdx.x;
     if (dst) {
         build_input(in, t, true, [&](uint32_t i) -> float & { return row_smem[i]; }, red);
-        A *o = dst + (size_t)t * in.k;
-        if constexpr (sizeof(A) == 2) {
-            for (uint32_t i = threadIdx.x * 2; i < in.k; i += 512) {  // (k is a multiple of 8)
-                const uint32_t lo = float_to_bf16_bits(row_smem[i]), hi = float_to_bf16_bits(row_smem[i + 1]);
-                *reinterpret_cast<uint32_t *>(o + i) = lo | (hi << 16);
+        for (uint32_t j = 0; j < (in.places ? in.top : 1u); ++j) {
+            A *o = dst + (size_t)(in.places ? (uint32_t)in.places[t * in.top + j] : t) * in.k;
+            if constexpr (sizeof(A) == 2) {
+                for (uint32_t i = threadIdx.x * 2; i < in.k; i += 512) {  // (k is a multiple of 8)
+                    const uint32_t lo = float_to_bf16_bits(row_smem[i]), hi = float_to_bf16_bits(row_smem[i + 1]);
+                    *reinterpret_cast<uint32_t *>(o + i) = lo | (hi << 16);
+                }
+            } else {
+                for (uint32_t i = threadIdx.x; i < in.k; i += 256) o[i] = row_smem[i];
             }
-        } else {
-            for (uint32_t i = threadIdx.x; i < in.k; i += 256) o[i] = row_smem[i];
         }
     }
     if (in.append.src) append_latent(in, t, red);
@@ -220,12 +232,20 @@ dense_input_kernel(InputArgs in, A *__restrict__ dst) {
 constexpr int kFTile = 64, kFK = 16;
 __global__ void __launch_bounds__(256)
 dense_f32_kernel(const float *__restrict__ x, uint32_t x_stride, uint32_t k, const float *__restrict__ w,
-                 uint32_t rows, uint32_t w_stride, uint32_t n_tokens, OutputArgs out) {
+                 uint32_t rows, uint32_t w_stride, uint32_t n_tokens, OutputArgs out, const int32_t *__restrict__ tiles) {
     qk::pdl_launch();
     qk::pdl_wait();
     __shared__ float xt[kFK][kFTile + 1], wt[kFK][kFTile + 1];
     const uint32_t tx = threadIdx.x % 16, ty = threadIdx.x / 16;
-    const uint32_t t0 = blockIdx.y * kFTile, n0 = blockIdx.x * kFTile;
+    uint32_t t0 = blockIdx.y * kFTile;
+    const uint32_t n0 = blockIdx.x * kFTile;
+    if (tiles) {  // rows sorted by expert
+        if (blockIdx.y >= (uint32_t)tiles[0]) return;
+        const int32_t *tile = tiles + 1 + 3 * blockIdx.y;
+        w += (size_t)tile[0] * rows * w_stride;
+        t0 = (uint32_t)tile[1];
+        n_tokens = (uint32_t)tile[2];
+    }
     float acc[4][4] = {};
     for (uint32_t k0 = 0; k0 < k; k0 += kFK) {
         for (uint32_t i = threadIdx.x; i < kFTile * kFK; i += 256) {
@@ -285,7 +305,19 @@ template <int BN> struct TcShape {
 struct TcArgs {
     uint32_t n_tokens, rows, k_chunks, m_tiles, tiles, wait_limit;
     int *error;
+    const int32_t *expert_tiles;  // rows sorted by expert: the token tiles (qk_route); null: one matrix
 };
+// Tile `tile` of the walk over token tiles (fastest) and weight tiles.
+struct TcTile {
+    uint32_t t0, t_end, n0, w0;  // rows of x, first output column, first row of W
+};
+template <int BN>
+__device__ __forceinline__ TcTile tc_tile(const TcArgs &g, uint32_t m_tiles, uint32_t tile) {
+    const uint32_t m = tile % m_tiles, n0 = (tile / m_tiles) * BN;
+    if (!g.expert_tiles) return {m * kTcM, g.n_tokens, n0, n0};
+    const int32_t *e = g.expert_tiles + 1 + 3 * m;
+    return {(uint32_t)e[1], (uint32_t)e[2], n0, (uint32_t)e[0] * g.rows + n0};
+}
 __device__ __forceinline__ uint32_t tc_idesc(uint32_t bn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((bn >> 3) << 17) | ((uint32_t)(kTcM >> 4) << 24);
 }
@@ -425,12 +457,14 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     qk::pdl_wait();
     const uint32_t tmem_base = *tmem_slot;
+    const uint32_t m_tiles = g.expert_tiles ? (uint32_t)g.expert_tiles[0] : g.m_tiles;
+    const uint32_t n_tiles = g.expert_tiles ? m_tiles * ((g.rows + BN - 1) / BN) : g.tiles;
 
     if (warp == 0) {
         uint32_t gc = 0;
         bool dead = false;
-        for (uint32_t tile = blockIdx.x; tile < g.tiles && !dead; tile += gridDim.x) {
-            const uint32_t t0 = (tile % g.m_tiles) * kTcM, n0 = (tile / g.m_tiles) * BN;
+        for (uint32_t tile = blockIdx.x; tile < n_tiles && !dead; tile += gridDim.x) {
+            const TcTile at = tc_tile<BN>(g, m_tiles, tile);
             for (uint32_t kc = 0; kc < g.k_chunks; ++kc, ++gc) {
                 const uint32_t s = gc % S::kStages;
                 if (!mbar_wait(&empty[s], ((gc / S::kStages) & 1) ^ 1, abort_flag, g.wait_limit)) {
@@ -442,8 +476,8 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
                                  "r"(S::kStage)
                                  : "memory");
                     const uint32_t a = smem_u32(tiles + s * S::kStage);
-                    tma_load_2d(a, &x_map, kc * kTcK, t0, &full[s]);
-                    tma_load_2d(a + S::kABytes, &w_map, kc * kTcK, n0, &full[s]);
+                    tma_load_2d(a, &x_map, kc * kTcK, at.t0, &full[s]);
+                    tma_load_2d(a + S::kABytes, &w_map, kc * kTcK, at.w0, &full[s]);
                 }
                 __syncwarp();
             }
@@ -461,7 +495,7 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
         const uint32_t idesc = tc_idesc(BN);
         uint32_t gc = 0, seg = 0;
         bool dead = false;
-        for (uint32_t tile = blockIdx.x; tile < g.tiles && !dead; tile += gridDim.x, ++seg) {
+        for (uint32_t tile = blockIdx.x; tile < n_tiles && !dead; tile += gridDim.x, ++seg) {
             const uint32_t acc = seg & 1;
             if (!mbar_wait(&acc_empty[acc], ((seg >> 1) & 1) ^ 1, abort_flag, g.wait_limit)) {
                 dead = true;
@@ -504,9 +538,10 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     } else {
         const uint32_t quarter = warp % 4;
         uint32_t seg = 0;
-        for (uint32_t tile = blockIdx.x; tile < g.tiles; tile += gridDim.x, ++seg) {
+        for (uint32_t tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++seg) {
             const uint32_t acc = seg & 1;
-            const uint32_t t0 = (tile % g.m_tiles) * kTcM + quarter * 32, n0 = (tile / g.m_tiles) * BN;
+            const TcTile at = tc_tile<BN>(g, m_tiles, tile);
+            const uint32_t t0 = at.t0 + quarter * 32, n0 = at.n0;
             float *stage = epi + (warp - 2) * 32 * kEpiPitch;
             if (!tc_epilogue_vote(mbar_wait(&acc_full[acc], (seg >> 1) & 1, abort_flag, g.wait_limit))) {
                 *abort_flag = 1;
@@ -530,12 +565,12 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
 #pragma unroll
                         for (int j = 0; j < 32; ++j) v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
                     }
-                    tc_store_tile<KIND>(out, t0, g.n_tokens, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
+                    tc_store_tile<KIND>(out, t0, at.t_end, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
                 } else {
                     tmem_ld_wait();
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(a[j]);
-                    tc_store_tile<KIND>(out, t0, g.n_tokens, n0 + c, g.rows, v, stage, lane, vec != 0);
+                    tc_store_tile<KIND>(out, t0, at.t_end, n0 + c, g.rows, v, stage, lane, vec != 0);
                 }
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
@@ -568,13 +603,23 @@ dense_norm_rows_kernel(InputArgs in, uint16_t *__restrict__ dst) {
         h[j] = p < pieces ? xr[p] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     if (in.pending) {
-        const float4 *pr = reinterpret_cast<const float4 *>(in.pending + (size_t)t * in.pending_stride);
+        const uint32_t parts = in.pending_top ? in.pending_top : 1;
         float4 y[kV];
         float ps = 0.f;
+        for (uint32_t c = 0; c < parts; ++c) {
+            const float4 *pr = reinterpret_cast<const float4 *>(
+                in.pending_top ? pending_row(in, t, c) : in.pending + (size_t)t * in.pending_stride);
+#pragma unroll
+            for (int j = 0; j < kV; ++j) {
+                const uint32_t p = threadIdx.x + 256 * j;
+                const float4 v = p < pieces ? pr[p] : make_float4(0.f, 0.f, 0.f, 0.f);
+                y[j] = c ? make_float4(y[j].x + v.x, y[j].y + v.y, y[j].z + v.z, y[j].w + v.w) : v;
+            }
+        }
+        const float share = in.pending_top ? in.pending_scale : 1.f;
 #pragma unroll
         for (int j = 0; j < kV; ++j) {
-            const uint32_t p = threadIdx.x + 256 * j;
-            y[j] = p < pieces ? pr[p] : make_float4(0.f, 0.f, 0.f, 0.f);
+            y[j] = make_float4(y[j].x * share, y[j].y * share, y[j].z * share, y[j].w * share);
             ps += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
         }
         const float inv = 1.0f / sqrtf(in_block_sum(ps, red) / (float)n + in.pending_eps);
@@ -609,7 +654,7 @@ dense_norm_rows_kernel(InputArgs in, uint16_t *__restrict__ dst) {
         }
         inv = 1.0f / sqrtf(in_block_sum(s, red) / (float)n + in.norm_eps);
     }
-    uint2 *o = reinterpret_cast<uint2 *>(dst + (size_t)t * in.k);
+    const uint32_t copies = in.places ? in.top : 1;
     const float4 *nw = reinterpret_cast<const float4 *>(in.norm_weight);
     const uint32_t half = (in.kind == QK_INPUT_CONCAT ? in.k / 2 : in.k) / 4;
     const float4 *second = reinterpret_cast<const float4 *>(in.second ? in.second + (size_t)t * in.x_stride : nullptr);
@@ -627,8 +672,11 @@ dense_norm_rows_kernel(InputArgs in, uint16_t *__restrict__ dst) {
             v = make_float4((v.x - mean) * inv * w.x, (v.y - mean) * inv * w.y, (v.z - mean) * inv * w.z,
                             (v.w - mean) * inv * w.w);
         }
-        o[p] = pack(v);
-        if (in.kind == QK_INPUT_CONCAT) o[half + p] = pack(p < pieces ? second[p] : make_float4(0.f, 0.f, 0.f, 0.f));
+        for (uint32_t c = 0; c < copies; ++c) {
+            uint2 *o = reinterpret_cast<uint2 *>(dst + (size_t)(in.places ? (uint32_t)in.places[t * in.top + c] : t) * in.k);
+            o[p] = pack(v);
+            if (in.kind == QK_INPUT_CONCAT) o[half + p] = pack(p < pieces ? second[p] : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
     }
     if (in.append.src) append_latent(in, t, red);
 }
@@ -650,6 +698,8 @@ template <int BN> struct NarrowShape {
 struct NarrowArgs {
     uint32_t n_tokens, rows, k_chunks, splits, wait_limit;
     int *error;
+    const int32_t *offsets;  // rows sorted by expert: [experts + 1]; null: one matrix
+    uint32_t tiles;          // weight tiles of an expert
 };
 __device__ __forceinline__ void cluster_sync_all() {
     asm volatile("barrier.cluster.arrive.release.aligned;\n barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -671,7 +721,21 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
     volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
     volatile int *never = reinterpret_cast<volatile int *>(tmem_slot + 2);
     const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-    const uint32_t tile = blockIdx.x / g.splits, split = blockIdx.x % g.splits;  // (a cluster is one tile)
+    uint32_t tile = blockIdx.x / g.splits;  // (a cluster is one tile)
+    const uint32_t split = blockIdx.x % g.splits;
+    uint32_t t0 = 0, n_rows = g.n_tokens, w0 = tile * 128;  // rows of x, first row of W
+    if (g.offsets) {
+        // (qk_route lets nothing start early: the offsets may be read before the dependency wait)
+        const uint32_t e = tile / g.tiles;
+        tile %= g.tiles;
+        t0 = (uint32_t)g.offsets[e];
+        n_rows = (uint32_t)g.offsets[e + 1] - t0;
+        w0 = e * g.rows + tile * 128;
+        if (n_rows == 0) {  // (the same for the whole cluster)
+            qk::pdl_wait();
+            return;
+        }
+    }
     const uint32_t per = (g.k_chunks + g.splits - 1) / g.splits;
     const uint32_t kc0 = min(split * per, g.k_chunks), kc1 = min(kc0 + per, g.k_chunks);
     if (threadIdx.x == 0) {
@@ -700,7 +764,7 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
             asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(&full[i])),
                          "r"(S::kStage)
                          : "memory");
-            tma_load_2d(smem_u32(tiles + i * S::kStage), &w_map, (kc0 + i) * kTcK, tile * 128, &full[i]);
+            tma_load_2d(smem_u32(tiles + i * S::kStage), &w_map, (kc0 + i) * kTcK, w0, &full[i]);
         }
     qk::pdl_wait();
     const uint32_t tmem_base = *tmem_slot;
@@ -721,9 +785,9 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
                     asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(smem_u32(&full[s])),
                                  "r"(S::kStage)
                                  : "memory");
-                    tma_load_2d(a, &w_map, kc * kTcK, tile * 128, &full[s]);
+                    tma_load_2d(a, &w_map, kc * kTcK, w0, &full[s]);
                 }
-                tma_load_2d(a + S::kABytes, &x_map, kc * kTcK, 0, &full[s]);
+                tma_load_2d(a + S::kABytes, &x_map, kc * kTcK, t0, &full[s]);
             }
             __syncwarp();
         }
@@ -792,7 +856,7 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
     if (warp >= 2 && finished) {
         const bool pair = out.kind == QK_OUTPUT_GLU;
         const uint32_t share = (BN + g.splits - 1) / g.splits;  // columns this CTA finishes
-        const uint32_t c_begin = split * share, c_end = min(min(c_begin + share, (uint32_t)BN), g.n_tokens);
+        const uint32_t c_begin = split * share, c_end = min(min(c_begin + share, (uint32_t)BN), n_rows);
         float *ups = own + 128 * BN;  // [2][BN][32]: up rows for their gate rows
         const uint32_t n = tile * 128 + row, lane_addr = tmem_base + ((quarter * 32) << 16);
         auto value = [&](uint32_t c) -> float {  // (splits > 1) the sum over the cluster, in split order
@@ -810,7 +874,7 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
             if (pair) {
                 if (quarter & 1) ups[((quarter >> 1) * BN + c) * 32 + lane] = v;
             } else if (n < g.rows) {
-                finish(out, c, n, v);
+                finish(out, t0 + c, n, v);
             }
         };
         float kept[BN <= 64 ? BN : 1];  // a gate row's values until its up row's arrive
@@ -853,13 +917,13 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
                             float gate;
                             if constexpr (BN > 64) gate = __uint_as_float(v[e]);
                             else gate = kept[c0 + e];
-                            if (c < c_end) finish_pair(out, c, j, gate, ups[((quarter >> 1) * BN + c) * 32 + lane]);
+                            if (c < c_end) finish_pair(out, t0 + c, j, gate, ups[((quarter >> 1) * BN + c) * 32 + lane]);
                         }
                     }
                 } else {
 #pragma unroll 4
                     for (uint32_t c = c_begin; c < c_end; ++c)
-                        finish_pair(out, c, j, value(c), ups[((quarter >> 1) * BN + c) * 32 + lane]);
+                        finish_pair(out, t0 + c, j, value(c), ups[((quarter >> 1) * BN + c) * 32 + lane]);
                 }
             }
         }
@@ -912,20 +976,28 @@ int pick_tile(size_t m_tiles, size_t rows, size_t sms) {
     return best;
 }
 
+// Rows of x and of W as the matrix forms see them, and their row tiles.
+size_t input_rows(const qk_dense_call &d) { return d.experts ? d.tokens * d.top : d.tokens; }
+size_t weight_rows(const qk_dense_call &d) { return d.experts ? d.rows * d.experts : d.rows; }
+size_t row_tiles(const qk_dense_call &d, size_t tile) {
+    return qk::ceil_div(input_rows(d), tile) + (d.experts ? std::min(d.experts, input_rows(d)) : 0);
+}
+
 template <int BN, int KIND>
 qk_status launch_tc_kind(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_call &d, const OutputArgs &out,
                     int vec) {
     using S = TcShape<BN>;
     CUtensorMap xm, wm;
     qk_status st;
-    if ((st = encode_map(x, d.tokens, d.k, x_stride, kTcM, &xm)) != QK_OK) return st;
-    if ((st = encode_map(d.w, d.rows, d.k, d.w_stride, BN, &wm)) != QK_OK) return st;
+    if ((st = encode_map(x, input_rows(d), d.k, x_stride, kTcM, &xm)) != QK_OK) return st;
+    if ((st = encode_map(d.w, weight_rows(d), d.k, d.w_stride, BN, &wm)) != QK_OK) return st;
     TcArgs g{};
     g.n_tokens = (uint32_t)d.tokens;
     g.rows = (uint32_t)d.rows;
     g.k_chunks = (uint32_t)qk::ceil_div(d.k, kTcK);
-    g.m_tiles = (uint32_t)qk::ceil_div(d.tokens, kTcM);
+    g.m_tiles = (uint32_t)row_tiles(d, kTcM);  // (with experts: the most there can be)
     g.tiles = g.m_tiles * (uint32_t)qk::ceil_div(d.rows, BN);
+    g.expert_tiles = d.experts ? d.tiles : nullptr;
     g.wait_limit = c->wait_limit ? c->wait_limit : kTcWaitDefault;
     g.error = (int *)c->d_err.ptr;
     QK_CUDA(cudaFuncSetAttribute((dense_tc_kernel<BN, KIND>), cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
@@ -957,14 +1029,18 @@ qk_status launch_narrow(qk_ctx *c, const void *x, size_t x_stride, const qk_dens
     using S = NarrowShape<BN>;
     CUtensorMap xm, wm;
     qk_status st;
-    if ((st = encode_map(x, d.tokens, d.k, x_stride, BN, &xm)) != QK_OK) return st;
-    if ((st = encode_map(d.w, d.rows, d.k, d.w_stride, 128, &wm)) != QK_OK) return st;
+    if ((st = encode_map(x, input_rows(d), d.k, x_stride, BN, &xm)) != QK_OK) return st;
+    if ((st = encode_map(d.w, weight_rows(d), d.k, d.w_stride, 128, &wm)) != QK_OK) return st;
     NarrowArgs g{};
     g.n_tokens = (uint32_t)d.tokens;
     g.rows = (uint32_t)d.rows;
     g.k_chunks = (uint32_t)qk::ceil_div(d.k, kTcK);
-    const uint32_t tiles = (uint32_t)qk::ceil_div(d.rows, 128);
-    g.splits = narrow_splits(tiles, g.k_chunks, (size_t)c->sm_count);
+    const uint32_t per_matrix = (uint32_t)qk::ceil_div(d.rows, 128);
+    const uint32_t tiles = per_matrix * (uint32_t)(d.experts ? d.experts : 1);
+    g.offsets = d.experts ? d.offsets : nullptr;
+    g.tiles = per_matrix;
+    g.splits = narrow_splits(per_matrix * (d.experts ? std::min(d.experts, input_rows(d)) : 1), g.k_chunks,
+                             (size_t)c->sm_count);
     g.wait_limit = c->wait_limit ? c->wait_limit : kTcWaitDefault;
     g.error = (int *)c->d_err.ptr;
     QK_CUDA(cudaFuncSetAttribute(dense_narrow_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)S::kSmem));
@@ -1006,9 +1082,12 @@ qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out,
                                                     : qk::ceil_div(d.rows, R);
     QK_CUDA(cudaFuncSetAttribute(dense_vector_kernel<W, NT, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)std::max(smem, (size_t)48 * 1024)));
-    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>, dim3((unsigned)qk::ceil_div(groups * ks, kVecWarps)),
+    ChoiceArgs ch{};
+    if (d.experts) ch = ChoiceArgs{d.table, d.ids, (uint32_t)d.top, (uint32_t)d.vocab, d.by_choice ? 1u : 0u};
+    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>,
+                         dim3((unsigned)qk::ceil_div(groups * ks, kVecWarps), (unsigned)(d.experts ? input_rows(d) : 1)),
                          dim3(kVecThreads), smem, c->stream, in, out, (const W *)d.w, (uint32_t)d.rows,
-                         (uint32_t)d.w_stride, (uint32_t)n_tokens, ks);
+                         (uint32_t)d.w_stride, (uint32_t)n_tokens, ks, ch);
     QK_CUDA(cudaGetLastError());
     c->launches++;
     return QK_OK;
@@ -1018,7 +1097,9 @@ qk_status launch_vector(qk_ctx *c, const InputArgs &in, const OutputArgs &out, c
                         size_t n_tokens) {
     // rows per warp and warps per row group: about two blocks per SM or more (one, where a block
     // has a long vector to stage first)
-    const size_t want = (d.k > 8192 ? 1 : 2) * (size_t)c->sm_count * kVecWarps, steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
+    const size_t share = d.experts ? input_rows(d) : 1;  // (every choice has blocks of its own)
+    const size_t want = qk::ceil_div((d.k > 8192 ? 1 : 2) * (size_t)c->sm_count * kVecWarps, share);
+    const size_t steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
     const bool pair = d.output == QK_OUTPUT_GLU;
     if (d.rows / 4 >= want) return launch_vector_r<W, NT, 4>(c, in, out, d, n_tokens, 1);
     if (d.rows / 2 >= want || pair) {
@@ -1055,6 +1136,9 @@ InputArgs input_args(const qk_dense_call &d) {
     a.append = AppendArgs{d.append.src, d.append.weight, d.append.cache, (uint32_t)d.append.src_stride,
                           (uint32_t)d.append.width, (uint32_t)d.append.ring, (uint32_t)d.append.stride, d.append.eps,
                           d.append.cache_dtype == QK_BF16};
+    a.pending_rows = d.pending_rows;
+    a.pending_top = (uint32_t)d.pending_top;
+    a.pending_scale = d.pending_scale;
     return a;
 }
 OutputArgs output_args(const qk_dense_call &d) {
@@ -1077,7 +1161,8 @@ OutputArgs output_args(const qk_dense_call &d) {
 }
 void advance(InputArgs &a, OutputArgs &o, size_t t) {  // the same call from row t on
     a.x += t * a.x_stride;
-    if (a.pending) a.pending += t * a.pending_stride;
+    if (a.pending && a.pending_rows) a.pending_rows += t * a.pending_top;
+    else if (a.pending) a.pending += t * (a.pending_top ? a.pending_top : 1) * a.pending_stride;
     if (a.second) a.second += t * a.x_stride;
     if (a.gate) a.gate += t * a.gate_stride;
     if (a.x_out) a.x_out += t * a.x_stride;
@@ -1126,9 +1211,70 @@ qk_status validate(const qk_dense_call *d, bool with_weights) {
         return qk::fail(QK_ERR_VALUE, "qk_dense: no output buffer");
     if (d->output == QK_OUTPUT_GLU && d->rows % 64)
         return qk::fail(QK_ERR_VALUE, "qk_dense: gated pairs come in blocks of 64 rows, got %zu", d->rows);
+    if (d->experts) {
+        if (!d->ids || !d->table || d->vocab == 0 || d->top == 0 || d->top > d->experts)
+            return qk::fail(QK_ERR_VALUE, "qk_dense: %zu of %zu experts need token ids and a table", d->top, d->experts);
+        if (d->output != QK_OUTPUT_STORE && d->output != QK_OUTPUT_GLU)
+            return qk::fail(QK_ERR_VALUE, "qk_dense: the rows of experts are stored, not added to a stream");
+        if (d->by_choice && d->input != QK_INPUT_PLAIN)
+            return qk::fail(QK_ERR_VALUE, "qk_dense: input rows by choice must be plain");
+        if (d->append.src) return qk::fail(QK_ERR_VALUE, "qk_dense: no append beside experts");
+    }
     if (d->output == QK_OUTPUT_SIDE && (!d->side || !d->ids || d->vocab == 0))
         return qk::fail(QK_ERR_VALUE, "qk_dense: a side product needs its table and token ids");
     return QK_OK;
+}
+
+// ------------------------------------------------------------------ choices sorted by expert
+constexpr int kRouteThreads = 1024;
+__global__ void __launch_bounds__(kRouteThreads)
+route_kernel(const qk_route_job *__restrict__ jobs, const int32_t *__restrict__ ids, uint32_t tokens, uint32_t vocab,
+             uint32_t tile_rows) {
+    qk::pdl_wait();
+    const qk_route_job j = jobs[blockIdx.x];
+    const uint32_t top = (uint32_t)j.top, experts = (uint32_t)j.experts, n = tokens * top;
+    extern __shared__ uint32_t route_smem[];  // [experts]: counts, then each expert's next place
+    uint32_t *next = route_smem;
+    for (uint32_t e = threadIdx.x; e < experts; e += kRouteThreads) next[e] = 0;
+    __syncthreads();
+    auto expert = [&](uint32_t i) {
+        const uint32_t id = (uint32_t)min(max(ids[i / top], 0), (int)vocab - 1);
+        return (uint32_t)j.table[(size_t)id * top + i % top];
+    };
+    for (uint32_t i = threadIdx.x; i < n; i += kRouteThreads) atomicAdd(&next[expert(i)], 1u);
+    __syncthreads();
+    if (threadIdx.x < 32) {  // running sums of the counts and of the tiles, 32 experts at a time
+        uint32_t places = 0, tiles = 0;
+        for (uint32_t e0 = 0; e0 < experts; e0 += 32) {
+            const uint32_t e = e0 + threadIdx.x, count = e < experts ? next[e] : 0;
+            const uint32_t own = (count + tile_rows - 1) / tile_rows;
+            uint32_t p = count, q = own;
+            for (int off = 1; off < 32; off *= 2) {
+                const uint32_t a = __shfl_up_sync(0xffffffffu, p, off), b = __shfl_up_sync(0xffffffffu, q, off);
+                if (threadIdx.x >= (uint32_t)off) p += a, q += b;
+            }
+            const uint32_t first = places + p - count, tile0 = tiles + q - own;
+            if (e < experts) {
+                next[e] = first;
+                j.offsets[e] = (int32_t)first;
+                for (uint32_t k = 0; k < own; ++k) {
+                    int32_t *t = j.tiles + 1 + 3 * (tile0 + k);
+                    t[0] = (int32_t)e;
+                    t[1] = (int32_t)(first + k * tile_rows);
+                    t[2] = (int32_t)min(first + (k + 1) * tile_rows, first + count);
+                }
+            }
+            places += __shfl_sync(0xffffffffu, p, 31);
+            tiles += __shfl_sync(0xffffffffu, q, 31);
+        }
+        if (threadIdx.x == 0) {
+            j.offsets[experts] = (int32_t)places;
+            j.tiles[0] = (int32_t)tiles;
+        }
+    }
+    __syncthreads();
+    // (the order of an expert's places is free: no row's result depends on its place)
+    for (uint32_t i = threadIdx.x; i < n; i += kRouteThreads) j.places[i] = (int32_t)atomicAdd(&next[expert(i)], 1u);
 }
 
 template <typename A>
@@ -1169,6 +1315,26 @@ int32_t qk_dense_form(size_t tokens, size_t k, int32_t w_dtype) {
     return tokens <= (size_t)kNarrowTokens ? QK_FORM_NARROW : QK_FORM_TCGEN05;
 }
 
+size_t qk_route_tile_rows(size_t tokens, size_t k, int32_t w_dtype) {
+    return qk_dense_form(tokens, k, w_dtype) == QK_FORM_F32 ? kFTile : kTcM;
+}
+
+qk_status qk_route(qk_ctx *ctx, const qk_route_job *device_jobs, size_t n_jobs, size_t max_experts, const int32_t *ids,
+                   size_t tokens, size_t vocab, size_t tile_rows) {
+    qk_ctx *c;
+    qk_status st = qk::resolve_ctx(ctx, &c);
+    if (st != QK_OK) return st;
+    QK_CUDA(cudaSetDevice(c->device));
+    if (!device_jobs || !ids || vocab == 0 || tile_rows == 0) return qk::fail(QK_ERR_VALUE, "qk_route: bad arguments");
+    if (max_experts * 4 > 48 * 1024) return qk::fail(QK_ERR_VALUE, "qk_route: %zu experts do not fit shared memory", max_experts);
+    if (tokens == 0 || n_jobs == 0) return QK_OK;
+    (void)qk::launch_pdl(c->pdl, route_kernel, dim3((unsigned)n_jobs), dim3(kRouteThreads), max_experts * 4, c->stream,
+                         device_jobs, ids, (uint32_t)tokens, (uint32_t)vocab, (uint32_t)tile_rows);
+    QK_CUDA(cudaGetLastError());
+    c->launches++;
+    return QK_OK;
+}
+
 qk_status qk_dense_input(qk_ctx *ctx, const qk_dense_call *d) {
     qk_ctx *c;
     qk_status st = qk::resolve_ctx(ctx, &c);
@@ -1194,6 +1360,7 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
     InputArgs in = input_args(*d);
     OutputArgs out = output_args(*d);
     if (form == QK_FORM_VECTOR && d->x_dtype == QK_F32) {
+        if (d->experts) return bf16 ? launch_vector<uint16_t, 1>(c, in, out, *d, 1) : launch_vector<float, 1>(c, in, out, *d, 1);
         // as many rows per launch as fit shared memory
         for (size_t t = 0; t < d->tokens;) {
             const size_t left = d->tokens - t;
@@ -1216,12 +1383,16 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
     // the input rows in the weights' dtype
     const void *rows = d->x;
     size_t stride = d->x_stride;
-    const bool direct = d->input == QK_INPUT_PLAIN && d->x_dtype == d->w_dtype && d->x_stride >= d->k &&
+    const bool direct = d->input == QK_INPUT_PLAIN && (!d->experts || d->by_choice) && d->x_dtype == d->w_dtype && d->x_stride >= d->k &&
                         d->x_stride % 8 == 0 && ((uintptr_t)d->x & 15) == 0;
     if (d->x_dtype == QK_BF16 && !direct)
         return qk::fail(QK_ERR_VALUE, "qk_dense: bfloat16 rows of stride %zu cannot feed %zu columns", d->x_stride, d->k);
+    if (d->experts && (!d->offsets || !d->tiles || (!d->places && !d->by_choice)))
+        return qk::fail(QK_ERR_VALUE, "qk_dense: the matrix forms need the choices sorted by expert");
     if (!direct) {
-        const size_t need = d->tokens * d->k * (bf16 ? 2 : 4);
+        if (d->by_choice) return qk::fail(QK_ERR_VALUE, "qk_dense: rows by choice must be of the weights' dtype");
+        if (d->experts) in.places = d->places, in.top = (uint32_t)d->top;
+        const size_t need = input_rows(*d) * d->k * (bf16 ? 2 : 4);
         if (!d->scratch || d->scratch_bytes < need)
             return qk::fail(QK_ERR_VALUE, "qk_dense: %zu bytes of scratch are needed, %zu given", need,
                             d->scratch_bytes);
@@ -1234,10 +1405,10 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
         if ((st = launch_input<float>(c, in, d->tokens, nullptr)) != QK_OK) return st;
     }
     if (!bf16) {
-        dim3 grid((unsigned)qk::ceil_div(d->rows, kFTile), (unsigned)qk::ceil_div(d->tokens, kFTile));
+        dim3 grid((unsigned)qk::ceil_div(d->rows, kFTile), (unsigned)row_tiles(*d, kFTile));
         (void)qk::launch_pdl(c->pdl, dense_f32_kernel, grid, dim3(256), 0, c->stream, (const float *)rows,
                              (uint32_t)stride, (uint32_t)d->k, (const float *)d->w, (uint32_t)d->rows,
-                             (uint32_t)d->w_stride, (uint32_t)d->tokens, out);
+                             (uint32_t)d->w_stride, (uint32_t)d->tokens, out, d->experts ? d->tiles : nullptr);
         QK_CUDA(cudaGetLastError());
         c->launches++;
         return QK_OK;
@@ -1252,7 +1423,7 @@ qk_status qk_dense(qk_ctx *ctx, const qk_dense_call *d) {
     const int vec = (!d->out || (((uintptr_t)d->out & 15) == 0 && d->out_stride % 4 == 0)) &&
                     (!d->residual || (((uintptr_t)d->residual & 15) == 0 && d->residual_stride % 4 == 0)) &&
                     ((uintptr_t)d->out_scale & 15) == 0;
-    switch (pick_tile(qk::ceil_div(d->tokens, kTcM), d->rows, (size_t)c->sm_count)) {
+    switch (pick_tile(row_tiles(*d, kTcM), d->rows, (size_t)c->sm_count)) {
         case 256: return launch_tc<256>(c, rows, stride, *d, out, vec);
         case 128: return launch_tc<128>(c, rows, stride, *d, out, vec);
         default: return launch_tc<64>(c, rows, stride, *d, out, vec);

@@ -36,7 +36,23 @@ struct InputArgs {
     float pending_eps, norm_eps;
     int kind, norm;
     AppendArgs append;
+    // the pending value's y is a sum of pending_top rows times pending_scale (0: row t itself)
+    const int32_t *pending_rows;
+    uint32_t pending_top;
+    float pending_scale;
+    // the input rows of the matrix forms are stored once per choice, at places[t][..] (null: at t)
+    const int32_t *places;
+    uint32_t top;
 };
+// The choices of a linear with experts, for the vector form.
+struct ChoiceArgs {
+    const int32_t *table, *ids;
+    uint32_t top, vocab, by_choice;
+};
+__device__ __forceinline__ const float *pending_row(const InputArgs &a, uint32_t t, uint32_t j) {
+    const uint32_t at = t * a.pending_top + j;
+    return a.pending + (size_t)(a.pending_rows ? (uint32_t)a.pending_rows[at] : at) * a.pending_stride;
+}
 struct OutputArgs {
     void *out;
     float *residual;
@@ -102,12 +118,21 @@ __device__ __forceinline__ void build_input(const InputArgs &a, uint32_t t, bool
     // h = x + pending
     float sum = 0.f, sq = 0.f;
     if (a.pending) {
-        const float *pr = a.pending + (size_t)t * a.pending_stride;
         float ps = 0.f;
-        in_load(pr, n, [&](uint32_t i, float v) {
-            at(i) = v;
-            ps += v * v;
-        });
+        if (a.pending_top) {
+            for (uint32_t j = 0; j < a.pending_top; ++j)
+                in_load(pending_row(a, t, j), n, [&](uint32_t i, float v) { at(i) = j ? at(i) + v : v; });
+            for (uint32_t i = threadIdx.x; i < n; i += blockDim.x) {
+                const float v = at(i) * a.pending_scale;
+                at(i) = v;
+                ps += v * v;
+            }
+        } else {
+            in_load(a.pending + (size_t)t * a.pending_stride, n, [&](uint32_t i, float v) {
+                at(i) = v;
+                ps += v * v;
+            });
+        }
         const float inv = 1.0f / sqrtf(in_block_sum(ps, red) / (float)n + a.pending_eps);
         const float *pw = a.pending_weight;
         in_load(xr, n, [&](uint32_t i, float v) {

@@ -11,36 +11,10 @@
 #include <algorithm>
 
 #include "qk_dense_dev.cuh"
+#include "qk_mma.cuh"
 
 namespace {
 
-__device__ __forceinline__ void lt_ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
-__device__ __forceinline__ void lt_ldsm4_trans(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3])
-                 : "r"(addr));
-}
-__device__ __forceinline__ void lt_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    mma_bf16_full(c, a[0], a[1], a[2], a[3], b0, b1);
-}
-__device__ __forceinline__ void lt_copy16(void *smem, const void *gmem, uint32_t bytes) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)),
-                 "l"(gmem), "r"(bytes)
-                 : "memory");
-}
-__device__ __forceinline__ uint32_t lt_pack(float lo, float hi) {
-    return (uint32_t)float_to_bf16_bits(lo) | ((uint32_t)float_to_bf16_bits(hi) << 16);
-}
-// x as two bfloat16 terms, packed for two neighbouring values
-__device__ __forceinline__ void lt_split2(float a, float b, uint32_t &hi, uint32_t &lo) {
-    const uint16_t ah = float_to_bf16_bits(a), bh = float_to_bf16_bits(b);
-    hi = (uint32_t)ah | ((uint32_t)bh << 16);
-    lo = lt_pack(a - bf16_bits_to_float(ah), b - bf16_bits_to_float(bh));
-}
 // eight consecutive weights as floats
 __device__ __forceinline__ void lt_load8(const uint16_t *p, float (&w)[8]) {
     const uint4 v = *reinterpret_cast<const uint4 *>(p);
@@ -282,7 +256,7 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
                 uint32_t r = ring0 + j;
                 if (r >= a.ring) r -= a.ring;  // (a window is no longer than the ring)
                 const bool live = j < keys.count && warp * kQ + piece * 8 < a.kv_stride;
-                lt_copy16(dst + (key * S::kPitch + piece * 8) * 2, live ? base + (size_t)r * a.kv_stride + piece * 8 : cache,
+                copy16(dst + (key * S::kPitch + piece * 8) * 2, live ? base + (size_t)r * a.kv_stride + piece * 8 : cache,
                           live ? 16u : 0u);
             }
         }
@@ -299,7 +273,7 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
             float2 v = make_float2(0.f, 0.f);
             if (h0 + r < a.heads && c < a.kv_stride)  // (kv_stride is even)
                 v = *reinterpret_cast<const float2 *>(a.absorbed + ((size_t)t * a.heads + h0 + r) * a.kv_stride + c);
-            lt_split2(v.x, v.y, qh[ks][e], ql[ks][e]);
+            split_bf16(v.x, v.y, qh[ks][e], ql[ks][e]);
         }
     float o[kTilesPerWarp][4];
 #pragma unroll
@@ -322,13 +296,13 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
 #pragma unroll
             for (int pr = 0; pr < 2; ++pr) {
                 uint32_t b[4];  // two tiles of eight keys x 16 channels
-                lt_ldsm4(b, tile + (((2 * pr + (lane >> 4)) * 8 + (lane & 7)) * S::kPitch + ks * 16 +
+                ldsm4(b, tile + (((2 * pr + (lane >> 4)) * 8 + (lane & 7)) * S::kPitch + ks * 16 +
                                     ((lane >> 3) & 1) * 8) * 2);
-                lt_mma(s[2 * pr], qh[ks], b[0], b[1]);
-                lt_mma(s[2 * pr + 1], qh[ks], b[2], b[3]);
+                mma16(s[2 * pr], qh[ks], b[0], b[1]);
+                mma16(s[2 * pr + 1], qh[ks], b[2], b[3]);
                 if constexpr (TERMS == 2) {
-                    lt_mma(s2[2 * pr], ql[ks], b[0], b[1]);
-                    lt_mma(s2[2 * pr + 1], ql[ks], b[2], b[3]);
+                    mma16(s2[2 * pr], ql[ks], b[0], b[1]);
+                    mma16(s2[2 * pr + 1], ql[ks], b[2], b[3]);
                 }
             }
         float *sc = scores + (tile_i & 1) * 4 * 16 * S::kScorePitch;
@@ -384,20 +358,20 @@ latent_mma_kernel(LatentArgs a, const uint16_t *__restrict__ cache, uint32_t clu
 #pragma unroll
         for (int kk = 0; kk < 2; ++kk) {
             uint32_t ph[4], pl[4];
-            lt_split2(v[0][kk][0], v[0][kk][1], ph[0], pl[0]);
-            lt_split2(v[1][kk][0], v[1][kk][1], ph[1], pl[1]);
-            lt_split2(v[0][kk][2], v[0][kk][3], ph[2], pl[2]);
-            lt_split2(v[1][kk][2], v[1][kk][3], ph[3], pl[3]);
+            split_bf16(v[0][kk][0], v[0][kk][1], ph[0], pl[0]);
+            split_bf16(v[1][kk][0], v[1][kk][1], ph[1], pl[1]);
+            split_bf16(v[0][kk][2], v[0][kk][3], ph[2], pl[2]);
+            split_bf16(v[1][kk][2], v[1][kk][3], ph[3], pl[3]);
 #pragma unroll
             for (int n = 0; n < kTilesPerWarp; n += 2) {
                 uint32_t b[4];
-                lt_ldsm4_trans(b, tile + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kPitch +
+                ldsm4_trans(b, tile + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kPitch +
                                           (n + (lane >> 4)) * 8) * 2);
-                lt_mma(o[n], ph, b[0], b[1]);
-                lt_mma(o[n + 1], ph, b[2], b[3]);
+                mma16(o[n], ph, b[0], b[1]);
+                mma16(o[n + 1], ph, b[2], b[3]);
                 if constexpr (TERMS == 2) {
-                    lt_mma(o[n], pl, b[0], b[1]);
-                    lt_mma(o[n + 1], pl, b[2], b[3]);
+                    mma16(o[n], pl, b[0], b[1]);
+                    mma16(o[n + 1], pl, b[2], b[3]);
                 }
             }
         }
@@ -578,7 +552,7 @@ latent_output_mma_kernel(LatentArgs a, const uint16_t *__restrict__ uv) {
                 y = fmaf(e, v.y, y);
             }
             uint32_t hi, lo;
-            lt_split2(x, y, hi, lo);
+            split_bf16(x, y, hi, lo);
             *reinterpret_cast<uint32_t *>(lat + r * lp + i) = hi;
             if constexpr (TERMS == 2) *reinterpret_cast<uint32_t *>(lat + (16 + r) * lp + i) = lo;
         }
@@ -595,13 +569,13 @@ latent_output_mma_kernel(LatentArgs a, const uint16_t *__restrict__ uv) {
 #pragma unroll 8
         for (uint32_t k = 0; k < a.kv_stride; k += 16) {  // (kv_stride is a multiple of 16 here)
             uint32_t x[4], y[4];
-            lt_ldsm4(x, a_addr + k * 2);
-            if constexpr (TERMS == 2) lt_ldsm4(y, a_addr + (16 * lp + k) * 2);
+            ldsm4(x, a_addr + k * 2);
+            if constexpr (TERMS == 2) ldsm4(y, a_addr + (16 * lp + k) * 2);
 #pragma unroll
             for (int n = 0; n < 2; ++n) {
                 const uint32_t b0 = row[n][k / 2], b1 = row[n][k / 2 + 4];
-                lt_mma(acc[n], x, b0, b1);
-                if constexpr (TERMS == 2) lt_mma(acc[n], y, b0, b1);
+                mma16(acc[n], x, b0, b1);
+                if constexpr (TERMS == 2) mma16(acc[n], y, b0, b1);
             }
         }
 #pragma unroll
@@ -658,13 +632,13 @@ window_attention_kernel(BandArgs a) {
         for (uint32_t i = threadIdx.x; i < kBandK * (DK / 8); i += 128) {
             const uint32_t key = i / (DK / 8), piece = i % (DK / 8);
             const bool live = r0 + key < a.n_keys && piece * 8 < a.dim_stride;
-            lt_copy16(kt + (key * S::kKPitch + piece * 8) * 2,
+            copy16(kt + (key * S::kKPitch + piece * 8) * 2,
                       a.kv + (live ? (size_t)(r0 + key) * a.kv_row + h * a.dim_stride + piece * 8 : 0), live ? 16u : 0u);
         }
         for (uint32_t i = threadIdx.x; i < kBandK * (DV / 8); i += 128) {
             const uint32_t key = i / (DV / 8), piece = i % (DV / 8);
             const bool live = r0 + key < a.n_keys && piece * 8 < a.vdim_stride;
-            lt_copy16(vt + (key * S::kVPitch + piece * 8) * 2,
+            copy16(vt + (key * S::kVPitch + piece * 8) * 2,
                       a.kv + (live ? (size_t)(r0 + key) * a.kv_row + a.heads * a.dim_stride + h * a.vdim_stride + piece * 8
                                    : 0),
                       live ? 16u : 0u);
@@ -674,7 +648,7 @@ window_attention_kernel(BandArgs a) {
     for (uint32_t i = threadIdx.x; i < kBandQ * (DK / 8); i += 128) {
         const uint32_t r = i / (DK / 8), piece = i % (DK / 8);
         const bool live = q0 + r < a.tokens && piece * 8 < a.dim_stride;
-        lt_copy16(qs + (r * S::kKPitch + piece * 8) * 2,
+        copy16(qs + (r * S::kKPitch + piece * 8) * 2,
                   a.q + (live ? (size_t)(q0 + r) * a.q_stride + h * a.dim_stride + piece * 8 : 0), live ? 16u : 0u);
     }
     fetch(0, 0);
@@ -700,7 +674,7 @@ window_attention_kernel(BandArgs a) {
         if constexpr (DK <= 128) {
             if (jt == 0) {
 #pragma unroll
-                for (int ks = 0; ks < DK / 16; ++ks) lt_ldsm4(qf[ks], q_addr + ks * 32);
+                for (int ks = 0; ks < DK / 16; ++ks) ldsm4(qf[ks], q_addr + ks * 32);
             }
         }
         const int j0 = (int)(lo + jt * kBandK);
@@ -713,18 +687,18 @@ window_attention_kernel(BandArgs a) {
 #pragma unroll
             for (int ks = 0; ks < DK / 16; ++ks) {
                 uint32_t qa[4];
-                if constexpr (DK > 128) lt_ldsm4(qa, q_addr + ks * 32);
+                if constexpr (DK > 128) ldsm4(qa, q_addr + ks * 32);
 #pragma unroll
                 for (int pr = 0; pr < 4; ++pr) {
                     uint32_t b[4];
-                    lt_ldsm4(b, kt + (((2 * pr + (lane >> 4)) * 8 + (lane & 7)) * S::kKPitch + ks * 16 +
+                    ldsm4(b, kt + (((2 * pr + (lane >> 4)) * 8 + (lane & 7)) * S::kKPitch + ks * 16 +
                                       ((lane >> 3) & 1) * 8) * 2);
                     if constexpr (DK > 128) {
-                        lt_mma(s[2 * pr], qa, b[0], b[1]);
-                        lt_mma(s[2 * pr + 1], qa, b[2], b[3]);
+                        mma16(s[2 * pr], qa, b[0], b[1]);
+                        mma16(s[2 * pr + 1], qa, b[2], b[3]);
                     } else {
-                        lt_mma(s[2 * pr], qf[ks], b[0], b[1]);
-                        lt_mma(s[2 * pr + 1], qf[ks], b[2], b[3]);
+                        mma16(s[2 * pr], qf[ks], b[0], b[1]);
+                        mma16(s[2 * pr + 1], qf[ks], b[2], b[3]);
                     }
                 }
             }
@@ -768,16 +742,16 @@ window_attention_kernel(BandArgs a) {
             }
 #pragma unroll
             for (int kk = 0; kk < 4; ++kk) {
-                const uint32_t p[4] = {lt_pack(s[2 * kk][0], s[2 * kk][1]), lt_pack(s[2 * kk][2], s[2 * kk][3]),
-                                       lt_pack(s[2 * kk + 1][0], s[2 * kk + 1][1]),
-                                       lt_pack(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+                const uint32_t p[4] = {pack_bf16(s[2 * kk][0], s[2 * kk][1]), pack_bf16(s[2 * kk][2], s[2 * kk][3]),
+                                       pack_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1]),
+                                       pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3])};
 #pragma unroll
                 for (int i = 0; i < DV / 8; i += 2) {
                     uint32_t b[4];
-                    lt_ldsm4_trans(b, vt + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kVPitch +
+                    ldsm4_trans(b, vt + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kVPitch +
                                             (i + (lane >> 4)) * 8) * 2);
-                    lt_mma(o[i], p, b[0], b[1]);
-                    lt_mma(o[i + 1], p, b[2], b[3]);
+                    mma16(o[i], p, b[0], b[1]);
+                    mma16(o[i + 1], p, b[2], b[3]);
                 }
             }
         }

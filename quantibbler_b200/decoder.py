@@ -178,6 +178,7 @@ class SlotDecoder:
     ``_portion_hidden`` (final-normed hidden rows of the last portion)."""
 
     tp_size, group = 1, None
+    logit_softcap = None  # logits <- cap tanh(logits / cap)
     keeps_state = False   # True: a step changes more than the cache row of its own position
 
     def _setup_driver(self) -> None:
@@ -189,8 +190,8 @@ class SlotDecoder:
     def _head(self, hidden, n: int, logits) -> None:
         """logits[:n] from ``n`` final-normed rows (a vocabulary shard under tensor parallelism)."""
         tag = QK_BF16 if self.cfg.serving == "bfloat16" else QK_F32
-        check(_lib.lib().qk_lm_head(self.ctx.handle, _p(hidden), _p(self.lm_head), tag, n, self.v_loc,
-                                    self.head_width, self.v_loc, _p(logits)))
+        check(_lib.lib().qk_lm_head_capped(self.ctx.handle, _p(hidden), _p(self.lm_head), tag, n, self.v_loc,
+                                           self.head_width, self.v_loc, self.logit_softcap or 0.0, _p(logits)))
 
     def _greedy(self, logits, n: int, best_val, best_idx) -> None:
         """The first maximum of each row."""

@@ -1,6 +1,6 @@
 """Decoder of layered designs: a list of layers, each a mixer (``layers.py``) with an optional
-gated feed-forward, optionally with a block of layers that runs several times, layer scales,
-and a per-layer token input.
+feed-forward (gated, or a mixture of experts), optionally with a block of layers that runs several
+times, layer scales or norms behind the sublayers, and a per-layer token input.
 
 Slots, prompts in portions, greedy steps, graph capture and generation are ``SlotDecoder``'s; this
 class adds the trunk.  Every pass of a looped layer has its own cache or state; what a sequence
@@ -18,8 +18,8 @@ from . import _lib
 from ._lib import QK_F32, check
 from .decoder import SlotDecoder, check_cache_capacity
 from .gpu import GpuContext
-from .layers import (IN_CONCAT, IN_NORM, NORM_LAYER, NORM_NONE, NORM_RMS, GatedDelta, GatedMlp, LatentAttention,
-                     Linear, Rows, TokenSide, Weights, padded)
+from .layers import (IN_CONCAT, IN_NORM, NORM_LAYER, NORM_NONE, NORM_RMS, GatedDelta, GatedMlp, GroupedAttention, Join,
+                     LatentAttention, Linear, Rows, TableExperts, TokenSide, Weights, padded)
 
 NORMS = {"layer": NORM_LAYER, "rms": NORM_RMS}
 IDLE = -(1 << 30)   # position of a row without a sequence: far enough below zero to stay negative
@@ -27,9 +27,10 @@ IDLE = -(1 << 30)   # position of a row without a sequence: far enough below zer
 
 @dataclass
 class LayerSpec:
-    mixer: str                      # "latent_attention" or "delta"
+    mixer: str                      # a key of MIXERS
     sizes: dict                     # the mixer's keyword arguments
     activation: str | None = None   # feed-forward activation; None: no feed-forward
+    experts: int | None = None      # a mixture of this many, chosen by a table of token ids; None: one
 
 
 @dataclass
@@ -39,6 +40,9 @@ class LayeredConfig:
     layers: list
     norm: str = "layer"
     norm_eps: float = 1e-5
+    norm_offset: float = 0.0                # added to the norms' weights
+    post_norms: bool = False                # results join the stream through norms (norm1b, norm2b)
+    logit_softcap: float | None = None      # logits <- cap tanh(logits / cap)
     embedding_scale: float = 1.0
     sinusoid_base: float | None = None      # None: no position vector
     loop: tuple | None = None               # (start, stop, times)
@@ -60,18 +64,28 @@ class LayeredConfig:
         return [(i, False) for i in range(start)] + body * times + [(i, False) for i in range(stop, n)]
 
 
+MIXERS = {"latent_attention": LatentAttention, "delta": GatedDelta, "grouped_attention": GroupedAttention}
+
+
 class _Layer:
     def __init__(self, w: Weights, cfg: LayeredConfig, spec: LayerSpec, t: dict, index: int, side_table):
         def part(prefix):
             return {n[len(prefix):]: a for n, a in t.items() if n.startswith(prefix)}
 
-        mixers = {"latent_attention": LatentAttention, "delta": GatedDelta}
-        self.mixer = mixers[spec.mixer](w, part("mix."), eps=cfg.norm_eps, **spec.sizes)
-        self.norm1, self.norm2, self.mlp, self.side = w.vector(t["norm1"]), None, None, None
-        self.scale1, self.scale2 = (w.vector(t[n]) if n in t else None for n in ("ls1", "ls2"))
+        def join(which):
+            if cfg.post_norms:
+                return Join(norm=w.vector(t[f"norm{which}b"], cfg.norm_offset), eps=cfg.norm_eps)
+            return Join(scale=w.vector(t[f"ls{which}"]) if f"ls{which}" in t else None)
+
+        self.mixer = MIXERS[spec.mixer](w, part("mix."), eps=cfg.norm_eps, **spec.sizes)
+        self.norm1, self.norm2, self.mlp, self.side = w.vector(t["norm1"], cfg.norm_offset), None, None, None
+        self.join1, self.join2 = join(1), None
         if spec.activation is not None:
-            self.norm2 = w.vector(t["norm2"])
-            self.mlp = GatedMlp(w, part("mlp."), activation=spec.activation)
+            self.norm2, self.join2 = w.vector(t["norm2"], cfg.norm_offset), join(2)
+            if spec.experts is None:
+                self.mlp = GatedMlp(w, part("mlp."), activation=spec.activation)
+            else:
+                self.mlp = TableExperts(w, part("mlp."), experts=spec.experts, activation=spec.activation)
         if cfg.side_dim is not None:
             self.side = TokenSide(w, part("side."), side_table, dim=cfg.side_dim, offset=index * cfg.side_dim,
                                   eps=cfg.norm_eps)
@@ -79,7 +93,9 @@ class _Layer:
 
 class LayeredDecoder(SlotDecoder):
     """Batched greedy decoding of a ``LayeredConfig`` model on one GPU; ``tensors`` maps tensor
-    names (``embed``, ``l<i>.*``, ``loop.in``, ``side.embed``, ``final.norm``) to torch tensors."""
+    names (``embed``, ``l<i>.*``, ``loop.in``, ``side.embed``, ``final.norm``, ``head``) to torch
+    tensors; without ``head`` the embedding table serves as the head, without ``loop.in`` nothing
+    happens between the passes of a loop."""
 
     keeps_state = True
 
@@ -93,19 +109,24 @@ class LayeredDecoder(SlotDecoder):
         w = self.weights = Weights(torch, dev, cfg.serving)
         self.width, self.stride = cfg.width, padded(cfg.width)
         self.norm_kind = NORMS[cfg.norm]
-        # one table serves the embedding and, without its scale, the head; its columns are padded
-        self.lm_head = w.matrix(tensors["embed"]).w
+        if cfg.post_norms and cfg.side_dim is not None:
+            raise ValueError("a token input reads the settled stream: not beside norms behind the sublayers")
+        # (columns padded)
+        self.embedding = w.matrix(tensors["embed"]).w
+        self.lm_head = w.matrix(tensors["head"]).w if "head" in tensors else self.embedding
+        self.logit_softcap = cfg.logit_softcap
         self.head_width, self.v_loc, self.vocab_offset = self.stride, cfg.vocab, 0
-        self.final_norm = w.vector(tensors["final.norm"])
+        self.final_norm = w.vector(tensors["final.norm"], cfg.norm_offset)
         self.inv_freq = None
         if cfg.sinusoid_base is not None:
             i = np.arange((cfg.width + 1) // 2, dtype=np.float64)
             self.inv_freq = torch.from_numpy(float(cfg.sinusoid_base) ** (-2.0 * i / cfg.width)).to(dev)
         side = w.to(tensors["side.embed"]) if cfg.side_dim is not None else None
-        self.loop_in = w.halves(tensors["loop.in"], cfg.width) if cfg.loop is not None else None
+        self.loop_in = w.halves(tensors["loop.in"], cfg.width) if "loop.in" in tensors else None
         self.layers = [
             _Layer(w, cfg, spec, {n[len(f"l{i}."):]: t for n, t in tensors.items() if n.startswith(f"l{i}.")}, i, side)
             for i, spec in enumerate(cfg.layers)]
+        self.tables = [layer.mlp.table for layer in self.layers if isinstance(layer.mlp, TableExperts)]
         B = cfg.max_batch
         self.portion_rows = min(cfg.prefill_chunk, cfg.max_seq)
         self.runs = [(self.layers[i], starts,
@@ -127,20 +148,21 @@ class LayeredDecoder(SlotDecoder):
     def _trunk(self, rows: Rows, after_layer=None) -> None:
         cfg, ctx = self.cfg, self.ctx
         rows.pending = None
+        rows.route(ctx, self.tables, self.width, cfg.vocab)
         first = rows.f32("embedding", self.stride) if self.loop_in is not None else None
         check(_lib.lib().qk_embed_scaled(
-            ctx.handle, self.lm_head.data_ptr(), self.weights.tag, self.stride, rows.ids.data_ptr(),
+            ctx.handle, self.embedding.data_ptr(), self.weights.tag, self.stride, rows.ids.data_ptr(),
             rows.positions.data_ptr(), rows.n, self.width, cfg.vocab, float(cfg.embedding_scale),
             None if self.inv_freq is None else self.inv_freq.data_ptr(), rows.x.data_ptr(),
             None if first is None else first.data_ptr(), self.stride))
         for layer, starts_pass, state in self.runs:
-            if starts_pass:
+            if starts_pass and self.loop_in is not None:
                 f = dict(rows.stream_fields(NORM_NONE, None, 0.0), input=IN_CONCAT, second=first, x_out=None)
                 rows.dense(ctx, self.loop_in, **f, out=rows.x2, out_stride=self.stride)
                 rows.x, rows.x2, rows.pending = rows.x2, rows.x, None
-            layer.mixer.forward(ctx, rows, self.norm_kind, layer.norm1, cfg.norm_eps, layer.scale1, state, cfg.max_seq)
+            layer.mixer.forward(ctx, rows, self.norm_kind, layer.norm1, cfg.norm_eps, layer.join1, state, cfg.max_seq)
             if layer.mlp is not None:
-                layer.mlp.forward(ctx, rows, self.norm_kind, layer.norm2, cfg.norm_eps, layer.scale2)
+                layer.mlp.forward(ctx, rows, self.norm_kind, layer.norm2, cfg.norm_eps, layer.join2)
             if layer.side is not None:
                 layer.side.forward(ctx, rows)
             if after_layer is not None:
@@ -148,20 +170,18 @@ class LayeredDecoder(SlotDecoder):
 
     def _final(self, rows: Rows, places, out) -> None:
         """Final-normed rows: all of them (``places`` None) or the given ones."""
-        x, pending = rows.x, rows.pending
-        n = rows.n
-        y = None if pending is None else pending[0]
+        x, pending, n = rows.x, rows.pending, rows.n
         if places is not None:
             n = len(places)
-            if n == 1:
-                x, y = x[places[0]:], None if y is None else y[places[0]:]
+            if n == 1 and pending is None:
+                x = x[places[0]:]
             else:
                 idx = self.torch.as_tensor(places, device=self.device)
-                x, y = x.index_select(0, idx), None if y is None else y.index_select(0, idx)
+                x, pending = x.index_select(0, idx), None if pending is None else pending.at(self.torch, idx)
         fields = dict(tokens=n, input=IN_NORM, x=x, x_stride=self.stride, norm=self.norm_kind,
                       norm_weight=self.final_norm, norm_eps=self.cfg.norm_eps, out=out, out_dtype=QK_F32)
-        if y is not None:
-            fields.update(pending=y, pending_stride=self.stride, pending_weight=pending[1], pending_eps=pending[2])
+        if pending is not None:
+            fields.update(pending.fields())
         d = rows.call(Linear(self.lm_head, 0, self.width, self.stride), **fields)
         check(_lib.lib().qk_dense_input(self.ctx.handle, ctypes.byref(d)))
 

@@ -6,7 +6,7 @@ from __future__ import annotations
 import json
 import os
 
-from . import blob, model_dir, safetensors, vogizen
+from . import blob, model_dir, safetensors, virudra, vogizen
 from .decoder import Decoder
 from .layered import LayeredDecoder
 
@@ -16,7 +16,12 @@ def _load_vogizen(ctx, config: dict, tensors: dict, **settings):
     return LayeredDecoder(ctx, vogizen.parse(config, **settings), tensors)
 
 
-ARCHITECTURES = {"Vogizen": _load_vogizen}
+def _load_virudra(ctx, config: dict, tensors: dict, **settings):
+    virudra.check_tensors(config, tensors)
+    return LayeredDecoder(ctx, virudra.parse(config, **settings), tensors)
+
+
+ARCHITECTURES = {"Virudra": _load_virudra, "Vogizen": _load_vogizen}
 
 
 class UnknownArchitecture(ValueError):

@@ -93,7 +93,8 @@ def weights(cfg, seed=0):
 def tensors(w):
     """The weights as the torch tensors a file would hold."""
     import torch
-    return {n: torch.from_numpy(np.ascontiguousarray(a)).to(torch.bfloat16) for n, a in w.items()}
+    return {n: torch.from_numpy(np.ascontiguousarray(a)).to(torch.bfloat16 if a.dtype.kind == "f" else torch.int32)
+            for n, a in w.items()}
 
 
 def write_model(folder, cfg, w):
@@ -102,8 +103,11 @@ def write_model(folder, cfg, w):
         json.dump(cfg, f)
     header, blobs, at = {}, [], 0
     for name, a in w.items():
-        raw = (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype("<u2").tobytes()
-        header[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
+        if a.dtype.kind == "f":
+            kind, raw = "BF16", (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype("<u2").tobytes()
+        else:
+            kind, raw = "I32", np.ascontiguousarray(a).astype("<i4").tobytes()
+        header[name] = {"dtype": kind, "shape": list(a.shape), "data_offsets": [at, at + len(raw)]}
         blobs.append(raw)
         at += len(raw)
     head = json.dumps(header).encode()
