@@ -11,26 +11,15 @@ import pytest
 
 from oracle import vogizen_np as ref
 
+import layered_checks as checks
 import vogizen_models as vm
+from layered_checks import agree, assert_rows, decode_logits, greedy_oracle, prompt_logits
 
 pytestmark = pytest.mark.gpu
 
-def row_errors(got, want):
-    """Root-mean-square difference of each row, relative to the spread of the expected rows."""
-    got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
-    return np.sqrt(((got - want) ** 2).mean(axis=-1)) / want.std()
 
-
-class Limit:
-    """What a model's rows may differ by: in float32 a constant, in bfloat16 twice
-    what rounding the linears' inputs alone does to the restatement's worst row."""
-
-    def __init__(self, cfg, w, toks, want, serving):
-        self.value = 2e-5
-        if serving == "bfloat16":
-            with ref.rounded_operands(vm.bf16):
-                self.value = 2 * row_errors(ref.forward(cfg, w, toks), want).max()
-            assert self.value < 0.12, "too sensitive a model to tell a fault from rounding"
+def Limit(cfg, w, toks, want, serving):
+    return checks.Limit(ref, cfg, w, toks, want, serving)
 
 
 def decoder(ctx, cfg, w, serving, **settings):
@@ -38,33 +27,6 @@ def decoder(ctx, cfg, w, serving, **settings):
     from quantibbler_b200.layered import LayeredDecoder
     settings = dict(dict(max_seq=512, prefill_chunk=64), **settings)
     return LayeredDecoder(ctx, vogizen.parse(cfg, serving=serving, **settings), vm.tensors(w))
-
-
-def assert_rows(got, want, limit, what=""):
-    err = row_errors(got, want)
-    assert np.isfinite(err).all() and err.max() <= limit.value, (what, int(err.argmax()), float(err.max()), limit.value)
-
-
-def prompt_logits(dec, toks, slot=0, portions=None):
-    """Logits of every position, the tokens fed in the given portions."""
-    out, at = [], 0
-    for n in portions or [len(toks)]:
-        out.append(dec.prefill(toks[at:at + n], slot, at, want=range(n)).cpu().numpy())
-        at += n
-    assert at == len(toks)
-    return np.concatenate(out)
-
-
-def decode_logits(dec, toks, at, slot=0):
-    """Logits of tokens at positions ``at`` .., one batched step each."""
-    out = []
-    B = dec.cfg.max_batch
-    for i, t in enumerate(toks):
-        dec.start([t if s == slot else 0 for s in range(B)], [at + i if s == slot else None for s in range(B)])
-        dec.step()
-        dec.ctx.synchronize()
-        out.append(dec.logits[slot].cpu().numpy())
-    return np.stack(out)
 
 
 @pytest.mark.parametrize("serving", ["float32", "bfloat16"])
@@ -229,32 +191,13 @@ def test_longer_sequences_at_wider_sizes(gpu_ctx, serving):
     assert_rows(got, want, lim, "decoded")
 
 
-def greedy_oracle(cfg, w, prompt, n):
-    """Continuation and, per token, how far the choice was ahead of the second best."""
-    toks, out = list(prompt), []
-    for _ in range(n):
-        row = ref.forward(cfg, w, toks)[-1]
-        best = int(row.argmax())
-        out.append((best, float(row[best] - np.partition(row, -2)[-2]) / row.std()))
-        toks.append(best)
-    return out
-
-
-def agree(got, want, serving):
-    for g, (best, lead) in zip(got, want):
-        if g != best:
-            assert lead < (1e-4 if serving == "float32" else 0.1), (got, want)
-            return
-    assert len(got) == len(want)
-
-
 @pytest.mark.parametrize("serving", ["float32", "bfloat16"])
 def test_greedy_generation(gpu_ctx, serving):
     cfg = vm.mixed()
     w = vm.weights(cfg, 13)
     for n in (1, 23):
         prompt = vm.prompt(cfg, n, seed=n)
-        want = greedy_oracle(cfg, w, prompt, 12)
+        want = greedy_oracle(ref, cfg, w, prompt, 12)
         dec = decoder(gpu_ctx, cfg, w, serving)
         out = dec.generate(prompt, 12)
         assert out["finish"] == "length" and out["prompt_tokens"] == n
@@ -286,7 +229,7 @@ def test_batched_greedy_decode_through_a_graph(gpu_ctx):
     dec.capture()
     rest = dec.decode(8)
     for s, p in enumerate(prompts):
-        agree([int(first[s])] + [int(t) for t in rest[:, s]], greedy_oracle(cfg, w, p, 9), "float32")
+        agree([int(first[s])] + [int(t) for t in rest[:, s]], greedy_oracle(ref, cfg, w, p, 9), "float32")
 
 
 def test_refusals(gpu_ctx):
@@ -363,4 +306,4 @@ def test_command_line_generates(gpu_ctx, tmp_path):
     assert p.returncode == 0, p.stderr[-2000:]
     out = json.loads(p.stdout)
     assert out["prompt_tokens"] == 19 and out["finish"] == "length"
-    agree(out["completion_tokens"], greedy_oracle(cfg, w, prompt, 6), "float32")
+    agree(out["completion_tokens"], greedy_oracle(ref, cfg, w, prompt, 6), "float32")

@@ -47,18 +47,18 @@ def weights(cfg, seed=0, bias_rows=13):
         m, p = layer["mixer"], f"l{i}."
         H, G, dim, vdim = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         vec(p + "norm1", d)
-        vec(p + "norm1b", d, -0.3)
-        mat(p + "mix.q", H * dim, d, 1.5)
-        mat(p + "mix.k", G * dim, d, 1.5)
+        vec(p + "norm1b", d, -0.5)
+        mat(p + "mix.q", H * dim, d, 1.2)
+        mat(p + "mix.k", G * dim, d, 1.2)
         mat(p + "mix.v", G * vdim, d)
         rows = bias_rows[i] if isinstance(bias_rows, (list, tuple)) else bias_rows
-        out[p + "mix.rel"] = bf16(rng.standard_normal((rows, H)) * 1.5)
+        out[p + "mix.rel"] = bf16(rng.standard_normal((rows, H)) * 1.2)
         mat(p + "mix.o", d, H * vdim)
         mlp = layer["mlp"]
         if mlp is None:
             continue
         vec(p + "norm2", d)
-        vec(p + "norm2b", d, -0.3)
+        vec(p + "norm2b", d, -0.5)
         parts = [(p + "mlp.", mlp)]
         if mlp["kind"] == "moe":
             experts, top = mlp["router"]["experts"], mlp["router"]["top"]
@@ -101,7 +101,8 @@ MODELS = {
     "moe-single-expert": (config([moe(attention(), 64, 1, 1)]), 13),
     "moe-all": (config([moe(attention(), 20, 3, 3)]), 13),
     "moe-many": (config([moe(attention(), 16, 70, 5)]), 13),
-    "loop-whole": (config([dense(attention(), 40), moe(attention(), 30, 4, 2)], loop=(0, 2, 3)), 13),
+    "loop-whole": (config([dense(attention(), 40), moe(attention(), 30, 4, 2)], loop=(0, 2, 2)), 13),
+    "loop-thrice": (config([moe(attention(heads=2), 30, 4, 2)], loop=(0, 1, 3)), 13),
     "loop-once": (config([dense(attention(), 40), bare(attention())], loop=(1, 2, 1)), 13),
     "low-cap": (config([bare(attention())], cap=1.5), 13),
     "large-eps": (config([moe(attention(), 40, 6, 4)], eps=0.5), 13),
