@@ -647,17 +647,35 @@ def layered_config(size: str) -> dict:
             "loop": {"start": 0, "stop": 2, "times": 2}, "layers": [att, rec] * 3}
 
 
-def layered_tensors(config: dict, seed: int = 0) -> dict:
+def virudra_config(size: str) -> dict:
+    """A Virudra config with the layer sizes of a real model: four query heads per key/value head,
+    dense layers and mixtures of 16 experts (two per token, together as wide as a dense layer) in
+    turn, the first two layers looped, eight layer runs."""
+    z = LAYERED_SIZES[size]
+    mixer = {"heads": z["heads"], "kv_heads": z["heads"] // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+             "bias_max": 1024, "q_temp": {"coef": 0.2, "every": 512}}
+    dense = {"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": z["ff"]}}
+    mixture = {"type": "attention", "mixer": mixer,
+               "mlp": {"kind": "moe", "expert": {"ff": z["ff"] // 2}, "router": {"experts": 16, "top": 2}}}
+    return {"architecture": "Virudra", "width": z["width"], "vocab": LAYERED_VOCAB, "norm": {"eps": 1e-5},
+            "loop": {"start": 0, "stop": 2, "times": 2}, "logit_softcap": 30.0, "layers": [dense, mixture] * 3}
+
+
+def layered_tensors(design, config: dict, seed: int = 0) -> dict:
     import torch
-    from quantibbler_b200 import vogizen
     gen = torch.Generator(device="cuda").manual_seed(seed)
     out = {}
-    for name, shape in vogizen.shapes(config).items():
-        t = torch.randn(shape, device="cuda", generator=gen)
+    for name, shape in design.shapes(config).items():
+        if name.endswith(".table"):   # (every token's experts: neighbours of a random one)
+            layer = config["layers"][int(name.split(".")[0][1:])]["mlp"]["router"]
+            first = torch.randint(0, layer["experts"], (shape[0], 1), device="cuda", generator=gen)
+            out[name] = ((first + torch.arange(shape[1], device="cuda")) % layer["experts"]).to(torch.int32)
+            continue
+        t = torch.randn([32 if n is None else n for n in shape], device="cuda", generator=gen)
         if name.endswith(("A_log", "dt_bias")):
             t = t * 0.1 - 1.0
         elif len(shape) == 1:
-            t = 1.0 + 0.1 * t
+            t = (0.0 if config["architecture"] == "Virudra" else 1.0) + 0.1 * t
         else:
             t = t / shape[-1] ** 0.5
         out[name] = t.to(torch.bfloat16)
@@ -725,14 +743,11 @@ def timed_decode(dec, context: int, steps: int, warmup: int) -> float:
     return a.elapsed_time(b) / steps
 
 
-def layered_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
-    """The design's kernels one at a time: captured sequences over the layers' own weights (more
-    than L2 holds), against the roofline that bounds each."""
-    import torch
-    from quantibbler_b200 import layers as L
+def kernel_notes(peaks: dict):
+    """({name: entry}, note): ``note`` enters a kernel's time and its fraction of the roofline that
+    bounds it."""
     hbm, tc = peaks["hbm_gbs"], peaks["bf16_tflops"]
     out = {}
-    lays = dec.layers
 
     def note(name, ms, bytes_=None, flops=None, peak_flops=None):
         e = {"us": ms * 1e3}
@@ -743,6 +758,82 @@ def layered_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
                      frac=flops / ms / 1e9 / (peak_flops or tc))
         out[name] = e
 
+    return out, note
+
+
+def virudra_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
+    """The Virudra design's kernels one at a time, as ``layered_kernels`` does."""
+    import torch
+    from quantibbler_b200 import layers as L
+    out, note = kernel_notes(peaks)
+    lays = dec.layers
+    dense = [x.mlp for x in lays if isinstance(x.mlp, L.GatedMlp)]
+    moe = [x.mlp for x in lays if isinstance(x.mlp, L.TableExperts)]
+    states = {id(layer): st for layer, _, st in dec.runs}
+    for T in (1, 64, tokens):
+        rows = L.Rows(torch, dec.device, T, dec.stride, dec.weights, vector=T <= dec.cfg.vector_rows)
+        rows.positions.copy_(torch.arange(T) if T == tokens else torch.full((T,), dec.bench_context))
+        rows.ids.copy_(torch.randint(0, dec.cfg.vocab, (T,)))
+        x = torch.randn(2 * T, 1 << 15, device="cuda").to(rows.act)
+        o = torch.zeros(2 * T, 1 << 15, device="cuda")
+        o_act = torch.zeros(2 * T, 1 << 15, device="cuda", dtype=rows.act)
+        rows.route(ctx, dec.tables, dec.width, dec.cfg.vocab)
+        ctx.synchronize()
+
+        def linear(name, lins, kind, extra=lambda m: {}, weights=1, choices=1):
+            y, tag = (o_act, rows.act_tag) if kind == L.OUT_GLU else (o, L.QK_F32)
+            calls = [lambda m=m, f=dict(input=L.IN_PLAIN, x=x, x_dtype=rows.act_tag, x_stride=1 << 15, output=kind,
+                                        activation=1, out=y, out_dtype=tag, out_stride=1 << 15, **extra(i)):
+                     rows.dense(ctx, m, **f) for i, m in enumerate(lins)]
+            ms = graph_ms(ctx, calls * 4)
+            m = lins[0]
+            if T == tokens:
+                note(f"{name}, {T} rows", ms, flops=2.0 * T * choices * m.rows * m.width)
+            else:
+                note(f"{name}, {T} rows", ms, bytes_=2.0 * m.rows * m.width * weights)
+
+        linear("q, k, v", [y.mixer.proj for y in lays], L.OUT_STORE)
+        linear("output of the attention", [y.mixer.out for y in lays], L.OUT_STORE)
+        linear("gate, up", [m.pair for m in dense], L.OUT_GLU)
+        linear("down", [m.down for m in dense], L.OUT_STORE)
+        top = moe[0].table.top
+
+        def chosen(i):
+            t = moe[i].table
+            f = dict(experts=t.experts, top=t.top, table=t.rows, vocab=t.rows.shape[0])
+            if id(t) in rows.routes:
+                r = rows.routes[id(t)]
+                f.update(places=r.places, offsets=r.offsets, tiles=r.tiles)
+            return f
+
+        hit = len(set(moe[0].table.rows[rows.ids.long()].flatten().tolist()))
+        linear("gate, up of the experts", [m.pair for m in moe], L.OUT_GLU, lambda i: dict(chosen(i), by_choice=1), hit, top)
+        linear("down of the experts", [m.down for m in moe], L.OUT_STORE, lambda i: dict(chosen(i), by_choice=1), hit, top)
+        if T == tokens:
+            rows.portion = (0, 0)
+            rows.slots.fill_(0)
+        elif T > dec.cfg.max_batch:
+            continue
+        real, rows.dense = rows.dense, lambda *a, **k: None
+        m = lays[0].mixer
+        ms = graph_ms(ctx, [lambda y=y: y.mixer.forward(ctx, rows, 0, y.norm1, 1e-5, None, states[id(y)], 1 << 20)
+                            for y in lays] * 4)
+        rows.dense = real
+        if T == tokens:
+            note(f"attention of a portion (with the append), {T} rows", ms,
+                 flops=2.0 * m.heads * (m.dim + m.vdim) * T * (T + 1) / 2)
+        else:
+            note(f"attention, {T} rows", ms, bytes_=2.0 * T * (dec.bench_context + 1) * m.kv_heads * (m.dim + m.vdim))
+    return out
+
+
+def layered_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
+    """The Vogizen design's kernels one at a time: captured sequences over the layers' own weights
+    (more than L2 holds), against the roofline that bounds each."""
+    import torch
+    from quantibbler_b200 import layers as L
+    out, note = kernel_notes(peaks)
+    lays = dec.layers
     att = [x for x in lays if isinstance(x.mixer, L.LatentAttention)]
     rec = [x for x in lays if isinstance(x.mixer, L.GatedDelta)]
     states = {id(layer): st for layer, _, st in dec.runs}
@@ -841,12 +932,22 @@ def closest_kernels(ctx, dec, tokens: int, peaks: dict) -> dict:
     fl = 4.0 * H * hd * tokens * (tokens + 1) / 2
     out[f"prefill attention, {tokens} rows"] = {"us": ms * 1e3, "bound": "tensor", "tflops": fl / ms / 1e9,
                                                 "frac": fl / ms / 1e9 / tc}
+    out.update(closest_decode_attention(ctx, dec, peaks))
+    return out
+
+
+def closest_decode_attention(ctx, dec, peaks: dict) -> dict:
+    import torch
+    hbm, cfg, lib = peaks["hbm_gbs"], dec.cfg, _qk_lib()
+    P = lambda t: ctypes.c_void_p(t.data_ptr())
+    H, KV, hd, B = dec.h_loc, dec.kv_loc, cfg.head_dim, cfg.max_batch
+    q, o, out = torch.randn(B, H * hd, device="cuda"), torch.zeros(B, H * hd, device="cuda"), {}
     dec.kv_len.fill_(dec.bench_context)
     ms = graph_ms(ctx, [lambda i=i: lib.qk_decode_attention(
-        ctx.handle, P(q), P(dec.cache_k[i]), P(dec.cache_v[i]), dec.kv_tag, P(dec.kv_len), 1, H, KV, hd, cfg.max_seq,
+        ctx.handle, P(q), P(dec.cache_k[i]), P(dec.cache_v[i]), dec.kv_tag, P(dec.kv_len), B, H, KV, hd, cfg.max_seq,
         dec.n_splits, P(dec.att_scratch), P(o)) for i in range(cfg.n_layers)] * 4)
-    by = 4.0 * KV * hd * dec.bench_context
-    out["decode attention, 1 row"] = {"us": ms * 1e3, "bound": "hbm", "gbs": by / ms / 1e6, "frac": by / ms / 1e6 / hbm}
+    by = 4.0 * KV * hd * dec.bench_context * B
+    out[f"decode attention, {B} rows"] = {"us": ms * 1e3, "bound": "hbm", "gbs": by / ms / 1e6, "frac": by / ms / 1e6 / hbm}
     return out
 
 
@@ -856,12 +957,12 @@ def _qk_lib():
 
 
 def run_layered(args, local_rank: int) -> None:
-    """Prefill and decode throughput of the Vogizen design at the layer sizes of real models (random
+    """Prefill and decode throughput of a layered design at the layer sizes of real models (random
     weights) beside the factorized Llama-shaped decoder with the same width, heads, feed-forward,
-    vocabulary and number of layer runs."""
+    vocabulary and number of layer runs (--layered-beside: another design instead)."""
     import torch
 
-    from quantibbler_b200 import vogizen
+    from quantibbler_b200 import virudra, vogizen
     from quantibbler_b200.decoder import Decoder, DecoderConfig, random_model
     from quantibbler_b200.gpu import GpuContext
     from quantibbler_b200.layered import LayeredDecoder
@@ -870,18 +971,21 @@ def run_layered(args, local_rank: int) -> None:
     peaks_path = os.path.join(ROOT, "MEASURED_PEAKS.json")
     peaks = json.load(open(peaks_path)) if os.path.exists(peaks_path) else {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
     tokens, context = args.tokens, args.context
+    designs = {"vogizen": (vogizen, layered_config, layered_kernels), "virudra": (virudra, virudra_config, virudra_kernels)}
     sizes, launches = {}, 0
     with ClockSampler(local_rank) as clocks:
         for size in args.layered_sizes.split(","):
             z = LAYERED_SIZES[size]
-            config = layered_config(size)
-            tensors = layered_tensors(config)
             res = {"layer_runs": LAYERED_RUNS, "vocab": LAYERED_VOCAB, **z}
-            for name in ("vogizen", "closest"):
-                r = {}
+            for name in (args.layered_design, args.layered_beside):
+                r, tensors = {}, None
+                if name in designs:
+                    design, make_config, kernels = designs[name]
+                    config = make_config(size)
+                    tensors = layered_tensors(design, config)
                 for batch in (1, 64):
-                    if name == "vogizen":
-                        dec = LayeredDecoder(ctx, vogizen.parse(config, max_seq=context + 4096, max_batch=batch), tensors)
+                    if name in designs:
+                        dec = LayeredDecoder(ctx, design.parse(config, max_seq=context + 4096, max_batch=batch), tensors)
                         for _, _, st in dec.runs:
                             for t in vars(st).values():
                                 if isinstance(t, torch.Tensor):
@@ -901,25 +1005,30 @@ def run_layered(args, local_rank: int) -> None:
                     launches += dec.kernels_per_step * args.steps
                     r[f"decode_batch{batch}"] = {"context": context, "ms_per_step": ms, "tok_s": batch / ms * 1e3,
                                                  "kernels_per_step": dec.kernels_per_step}
-                    if batch == 1 and args.layered_kernels:
-                        dec.graph = None
-                        r["kernels"] = (layered_kernels if name == "vogizen" else closest_kernels)(
-                            ctx, dec, tokens, peaks)
                     dec.graph = None
+                    if args.layered_kernels and name == "virudra":
+                        # (the batched decoder has the slots for 64 rows; the rest does not depend on the batch)
+                        r.setdefault("kernels", {}).update(kernels(ctx, dec, tokens, peaks))
+                    elif batch == 1 and args.layered_kernels:
+                        r["kernels"] = (kernels if name in designs else closest_kernels)(ctx, dec, tokens, peaks)
+                    elif args.layered_kernels and name not in designs:
+                        r["kernels"].update(closest_decode_attention(ctx, dec, peaks))
                     del dec
                     ctx.set_stream(None)
                     torch.cuda.empty_cache()
                 res[name] = r
+                del tensors
             sizes[size] = res
             print(f"width {size}: {json.dumps(res)}", file=sys.stderr, flush=True)
-            del tensors
-    head = sizes[args.layered_sizes.split(",")[-1]]["vogizen"]
+    head = sizes[args.layered_sizes.split(",")[-1]][args.layered_design]
     print(json.dumps({
         "metric": "layered_decode_tok_s", "value": head["decode_batch1"]["tok_s"], "unit": "tok/s", "n_gpus": 1,
         "steps": args.steps, "warmup": max(args.warmup, 3), "ms_per_step": head["decode_batch1"]["ms_per_step"],
         "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
-        "config": {"workload": "Vogizen layers at real sizes, random weights, beside the factorized Llama-shaped "
-                               "decoder of equal width, heads, feed-forward, vocabulary and layer runs",
+        "config": {"workload": f"{args.layered_design.capitalize()} layers at real sizes, random weights, beside "
+                               + ("the factorized Llama-shaped decoder" if args.layered_beside == "closest"
+                                  else args.layered_beside.capitalize())
+                               + " of equal width, heads, feed-forward, vocabulary and layer runs",
                    "global_batch": 1, "seq_len": context,
                    "l2_policy": "weights larger than L2, streamed every step", "sizes": sizes},
         "gpu_launches": launches, "clocks": clocks.summary()}), flush=True)
@@ -942,6 +1051,9 @@ def main() -> None:
     ap.add_argument("--workload", default="gemv", choices=["gemv", "decode", "prefill", "attention", "layered"])
     ap.add_argument("--tokens", type=int, default=2048)
     ap.add_argument("--layered-sizes", default="2048,4096", help="layered workload: widths, with commas between them")
+    ap.add_argument("--layered-design", default="vogizen", choices=["vogizen", "virudra"], help="layered workload: which design")
+    ap.add_argument("--layered-beside", default="closest", choices=["closest", "vogizen", "virudra"],
+                    help="layered workload: what it stands beside (closest: the factorized Llama-shaped decoder)")
     ap.add_argument("--layered-kernels", type=int, default=1, help="layered workload: also time the kernels one by one")
     ap.add_argument("--model", default="llama3-8b", choices=["llama3-8b", "llama2-7b-layer"])
     ap.add_argument("--batch", type=int, default=1)

@@ -14,6 +14,7 @@
 #include <algorithm>
 
 #include "qk_dense_dev.cuh"
+#include "qk_tma.cuh"
 #include "qk_umma.cuh"
 
 namespace {
@@ -320,13 +321,6 @@ __device__ __forceinline__ TcTile tc_tile(const TcArgs &g, uint32_t m_tiles, uin
 }
 __device__ __forceinline__ uint32_t tc_idesc(uint32_t bn) {
     return (1u << 4) | (1u << 7) | (1u << 10) | ((bn >> 3) << 17) | ((uint32_t)(kTcM >> 4) << 24);
-}
-__device__ __forceinline__ void tma_load_2d(uint32_t dst, const CUtensorMap *map, uint32_t x, uint32_t y,
-                                            uint64_t *bar) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::
-            "r"(dst), "l"(map), "r"(x), "r"(y), "r"(smem_u32(bar))
-        : "memory");
 }
 __device__ __forceinline__ bool tc_epilogue_vote(bool ok) {
     uint32_t all;
@@ -938,30 +932,11 @@ dense_narrow_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_cons
     if (threadIdx.x == 0 && *abort_flag) atomicOr(g.error, 1);
 }
 
-typedef CUresult (*EncodeTiledFn)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *,
-                                  const cuuint64_t *, const cuuint32_t *, const cuuint32_t *, CUtensorMapInterleave,
-                                  CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
 // rows x k bfloat16 entries, `stride` entries from row to row; boxes of 64 k x box_rows.
 qk_status encode_map(const void *base, size_t rows, size_t k, size_t stride, uint32_t box_rows, CUtensorMap *out) {
-    static EncodeTiledFn fn = nullptr;
-    if (!fn) {
-        void *sym = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &sym, cudaEnableDefault, &qres);
-        if (e != cudaSuccess || qres != cudaDriverEntryPointSuccess || !sym)
-            return qk::fail(QK_ERR_CUDA, "cuTensorMapEncodeTiled is not available: %s", cudaGetErrorString(e));
-        fn = (EncodeTiledFn)sym;
-    }
-    const cuuint64_t dims[2] = {k, rows};
-    const cuuint64_t strides[1] = {stride * 2};
+    const cuuint64_t dims[2] = {k, rows}, strides[1] = {stride * 2};
     const cuuint32_t box[2] = {(cuuint32_t)kTcK, box_rows};
-    const cuuint32_t estr[2] = {1, 1};
-    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void *>(base), dims, strides, box, estr,
-                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
-                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) return qk::fail(QK_ERR_CUDA, "cuTensorMapEncodeTiled failed with code %d", (int)r);
-    return QK_OK;
+    return encode_bf16_map(base, 2, dims, strides, box, out);
 }
 
 // Weight rows per tile: the width whose number of waves over the SMs costs least.

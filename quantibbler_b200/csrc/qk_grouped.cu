@@ -6,14 +6,19 @@
 //     one key/value head as rows 0-7 and their second bfloat16 terms as rows 8-15, so that the
 //     queries and the softmax weights keep 16 bits of mantissa at no extra product.  A decode step's
 //     rows append their own key and value here;
-//   * portion (bfloat16): 64 consecutive rows of one sequence per block;
+//   * portion (bfloat16): consecutive rows of one sequence.  Head sizes of 64 to 128 on tcgen05, two
+//     tiles of 128 rows per CTA that share their keys and values; others on mma.sync, 64 rows per block;
 //   * plain: float32, and head sizes the others do not take.
 // The bias of a distance is looked up in a table per head that ends where the bias stops changing;
 // key tiles that lie wholly beyond it need no lookup.
+#include <cuda.h>  // CUtensorMap types only; the encoder is fetched through the runtime
+
 #include <algorithm>
 
 #include "qk_dense_dev.cuh"
 #include "qk_mma.cuh"
+#include "qk_tma.cuh"
+#include "qk_umma.cuh"
 
 namespace {
 
@@ -522,6 +527,360 @@ grouped_portion_kernel(GroupedArgs a) {
     }
 }
 
+// ------------------------------------------------------------------ portion, bfloat16, tcgen05
+// A CTA works on two units, each 128 rows of one query head; both read the same key/value head (two
+// heads of a group at the same rows, or neighbouring row tiles).  Per block of 128 keys: S = Q K^T into
+// tensor memory; four warps per unit turn their rows' scores into weights, which go back to tensor
+// memory over S as the A operand of O += P V; O stays in tensor memory.  While one unit's warps
+// exponentiate, the other unit's products run.  V is read as it lies in the cache (rows are keys), as an
+// MN-major B operand.  A row's accumulator is rescaled only when its maximum has grown by more than
+// 2^kUmLazy since its reference was set.  The bias of a block is a band of 255 distances: staged in
+// shared memory with the mask (-inf) built in, in four copies shifted by one so that every row reads
+// it in aligned pieces of four; blocks beyond the end of the bias table need no band.
+// Warps 0-3 and 4-7: the units' rows; warp 8: TMA; warp 9: MMA issue.  All waits are bounded.
+constexpr int kUmRows = 128, kUmKeys = 128, kUmThreads = 320, kUmStages = 2;
+constexpr uint32_t kUmChunk = 128 * 128;                       // 128 rows of 64 bfloat16
+constexpr uint32_t kUmTile = 2 * kUmChunk;                     // up to 128 channels
+constexpr int kUmBandPitch = 264;                              // floats per copy of the band
+constexpr uint32_t kUmBand = 4 * kUmBandPitch * 4;
+constexpr size_t kUmSmem = 1024 + (2 + 2 * kUmStages) * kUmTile + 4 * kUmBand + 256;
+constexpr uint32_t kUmOCol = 256, kUmTmemCols = 512;           // S of unit u at 128 u, O at 256 + 128 u
+constexpr float kUmLazy = 8.0f;
+constexpr uint32_t kUmWaitDefault = 1u << 22;
+static_assert(kUmSmem <= 227 * 1024, "the tiles must fit the shared memory of a CTA");
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ void tmem_store32(uint32_t taddr, const uint32_t *v) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, %17, %18, %19, %20, %21, %22, "
+        "%23, %24, %25, %26, %27, %28, %29, %30, %31, %32};" ::"r"(taddr),
+        "r"(v[0]), "r"(v[1]), "r"(v[2]), "r"(v[3]), "r"(v[4]), "r"(v[5]), "r"(v[6]), "r"(v[7]), "r"(v[8]), "r"(v[9]),
+        "r"(v[10]), "r"(v[11]), "r"(v[12]), "r"(v[13]), "r"(v[14]), "r"(v[15]), "r"(v[16]), "r"(v[17]), "r"(v[18]),
+        "r"(v[19]), "r"(v[20]), "r"(v[21]), "r"(v[22]), "r"(v[23]), "r"(v[24]), "r"(v[25]), "r"(v[26]), "r"(v[27]),
+        "r"(v[28]), "r"(v[29]), "r"(v[30]), "r"(v[31])
+        : "memory");
+}
+// bf16 x bf16 -> f32, M = 128, N = n; b_mn: B is MN-major
+__device__ __forceinline__ uint32_t portion_idesc(uint32_t n, uint32_t b_mn) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn << 16) | ((n >> 3) << 17) | ((uint32_t)(kUmRows >> 4) << 24);
+}
+// MN-major tile in chunks of 64 columns (128-byte rows, swizzled): 8-row groups 1024 bytes apart,
+// chunks kUmChunk apart.
+__device__ __forceinline__ uint64_t umma_desc_mn(uint32_t smem_addr) {
+    return umma_desc(smem_addr) | ((uint64_t)(kUmChunk >> 4) << 16);
+}
+// Barrier of the 128 threads of a unit; true when all of them say so.
+__device__ __forceinline__ bool unit_vote(uint32_t u, bool ok) {
+    uint32_t all;
+#define QK_UNIT_VOTE(id)                                                 \
+    asm volatile(                                                        \
+        "{\n .reg .pred p, q;\n setp.ne.b32 p, %1, 0;\n"                 \
+        " barrier.cta.red.and.pred q, " id ", 128, p;\n selp.u32 %0, 1, 0, q;\n}" \
+        : "=r"(all)                                                      \
+        : "r"((uint32_t)ok)                                              \
+        : "memory")
+    if (u == 0) QK_UNIT_VOTE("1");
+    else QK_UNIT_VOTE("2");
+#undef QK_UNIT_VOTE
+    return all != 0;
+}
+// The unit `index` of a key/value head: heads of the group fastest, then row tiles.
+struct PortionUnit {
+    uint32_t h, row0, n_blocks;
+};
+__device__ __forceinline__ PortionUnit portion_unit(const GroupedArgs &a, uint32_t kvh, uint32_t index) {
+    const uint32_t group = a.heads / a.kv_heads, row0 = index / group * kUmRows;
+    if (row0 >= a.tokens) return {0, 0, 0};
+    return {kvh * group + index % group, row0, (a.p0 + min(row0 + kUmRows, a.tokens) + kUmKeys - 1) / kUmKeys};
+}
+
+__global__ void __launch_bounds__(kUmThreads, 1)
+grouped_portion_umma_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
+                            const __grid_constant__ CUtensorMap v_map, GroupedArgs a, uint32_t wait_limit) {
+    qk::pdl_launch();
+    extern __shared__ __align__(1024) uint8_t um_smem[];
+    uint8_t *qs = reinterpret_cast<uint8_t *>(((uintptr_t)um_smem + 1023) & ~(uintptr_t)1023);
+    uint8_t *ks = qs + 2 * kUmTile, *vs = ks + kUmStages * kUmTile;
+    float *bands = reinterpret_cast<float *>(vs + kUmStages * kUmTile);  // [unit][2][4][kUmBandPitch]
+    uint64_t *q_full = reinterpret_cast<uint64_t *>(bands + 4 * 4 * kUmBandPitch);
+    uint64_t *k_full = q_full + 1, *k_empty = k_full + kUmStages, *v_full = k_empty + kUmStages, *v_empty = v_full + kUmStages;
+    uint64_t *s_full = v_empty + kUmStages, *p_full = s_full + 2, *o_full = p_full + 2, *drain = o_full + 2;
+    uint32_t *tmem_slot = reinterpret_cast<uint32_t *>(drain + 1);
+    volatile int *abort_flag = reinterpret_cast<volatile int *>(tmem_slot + 1);
+    volatile int *never = reinterpret_cast<volatile int *>(tmem_slot + 2);
+    const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const uint32_t kvh = blockIdx.x, pair = gridDim.y - 1 - blockIdx.y;  // (late rows see most keys)
+    const PortionUnit unit[2] = {portion_unit(a, kvh, 2 * pair), portion_unit(a, kvh, 2 * pair + 1)};
+    const uint32_t n_blocks = max(unit[0].n_blocks, unit[1].n_blocks);
+    const uint32_t d_chunks = (a.dim + 63) / 64, v_chunks = (a.vdim + 63) / 64;
+    if (threadIdx.x == 0) {
+        mbar_init(q_full, 1);
+        for (int s = 0; s < kUmStages; ++s) {
+            mbar_init(k_full + s, 1);
+            mbar_init(k_empty + s, 1);
+            mbar_init(v_full + s, 1);
+            mbar_init(v_empty + s, 1);
+        }
+        for (int u = 0; u < 2; ++u) {
+            mbar_init(s_full + u, 1);
+            mbar_init(p_full + u, 4);
+            mbar_init(o_full + u, 1);
+        }
+        mbar_init(drain, 1);
+        *abort_flag = 0;
+        *never = 0;
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&q_map) : "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&k_map) : "memory");
+        asm volatile("prefetch.tensormap [%0];" ::"l"(&v_map) : "memory");
+    }
+    if (warp == 9) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(tmem_slot)),
+                     "r"(kUmTmemCols)
+                     : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    qk::pdl_wait();
+    const uint32_t tmem = *tmem_slot;
+    uint32_t fetched = 0;  // (warp 8) blocks whose copies have been issued
+
+    if (warp == 8) {
+        if (lane == 0) {
+            const uint32_t live = (unit[0].n_blocks ? 1 : 0) + (unit[1].n_blocks ? 1 : 0);
+            mbar_expect(q_full, live * d_chunks * kUmChunk);
+#pragma unroll
+            for (uint32_t u = 0; u < 2; ++u)
+                for (uint32_t c = 0; c < d_chunks && unit[u].n_blocks; ++c)
+                    tma_load_2d(smem_u32(qs + u * kUmTile + c * kUmChunk), &q_map, unit[u].h * a.dim + c * 64, unit[u].row0, q_full);
+        }
+        __syncwarp();
+        for (uint32_t j = 0; j < n_blocks; ++j) {
+            const uint32_t s = j % kUmStages, parity = ((j / kUmStages) & 1) ^ 1;
+            if (!mbar_wait(k_empty + s, parity, abort_flag, wait_limit) || !mbar_wait(v_empty + s, parity, abort_flag, wait_limit)) {
+                *abort_flag = 1;
+                break;
+            }
+            if (lane == 0) {
+                mbar_expect(k_full + s, d_chunks * kUmChunk);
+                for (uint32_t c = 0; c < d_chunks; ++c)
+                    tma_load_3d(smem_u32(ks + s * kUmTile + c * kUmChunk), &k_map, c * 64, j * kUmKeys, kvh, k_full + s);
+                mbar_expect(v_full + s, v_chunks * kUmChunk);
+                for (uint32_t c = 0; c < v_chunks; ++c)
+                    tma_load_3d(smem_u32(vs + s * kUmTile + c * kUmChunk), &v_map, c * 64, j * kUmKeys, kvh, v_full + s);
+            }
+            fetched = j + 1;
+            __syncwarp();
+        }
+    } else if (warp == 9) {
+        const uint32_t idesc_s = portion_idesc(kUmKeys, 0), idesc_o = portion_idesc(a.vdim, 1);
+        auto scores = [&](uint32_t u, uint32_t j) {  // (lane 0)
+            const uint32_t q0 = smem_u32(qs + u * kUmTile), k0 = smem_u32(ks + (j % kUmStages) * kUmTile);
+            for (uint32_t k = 0; k < a.dim / 16; ++k) {
+                const uint32_t at = k / 4 * kUmChunk + k % 4 * 32;
+                const uint64_t ad = umma_desc(q0 + at), bd = umma_desc(k0 + at);
+                asm volatile(
+                    "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
+                    " tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n}" ::"r"(tmem + 128 * u),
+                    "l"(ad), "l"(bd), "r"(idesc_s), "r"(k)
+                    : "memory");
+            }
+            umma_commit(s_full + u);
+        };
+        auto values = [&](uint32_t u, uint32_t j) {  // (lane 0)
+            const uint32_t v0 = smem_u32(vs + (j % kUmStages) * kUmTile);
+#pragma unroll
+            for (uint32_t k = 0; k < kUmKeys / 16; ++k) {
+                const uint64_t bd = umma_desc_mn(v0 + k * 2048);
+                asm volatile(
+                    "{\n .reg .pred p;\n setp.ne.b32 p, %4, 0;\n"
+                    " tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n}" ::"r"(tmem + kUmOCol + 128 * u),
+                    "r"(tmem + 128 * u + k * 8), "l"(bd), "r"(idesc_o), "r"(j + k)
+                    : "memory");
+            }
+        };
+        bool ok = mbar_wait(q_full, 0, abort_flag, wait_limit) && mbar_wait(k_full, 0, abort_flag, wait_limit);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (ok && lane == 0) {
+#pragma unroll
+            for (uint32_t u = 0; u < 2; ++u)
+                if (unit[u].n_blocks) scores(u, 0);
+            umma_commit(k_empty);
+        }
+        __syncwarp();
+        for (uint32_t j = 0; j < n_blocks && ok; ++j) {
+            const uint32_t s = j % kUmStages, s1 = (j + 1) % kUmStages;
+            ok = mbar_wait(v_full + s, (j / kUmStages) & 1, abort_flag, wait_limit);
+            if (ok && j + 1 < n_blocks) ok = mbar_wait(k_full + s1, ((j + 1) / kUmStages) & 1, abort_flag, wait_limit);
+#pragma unroll
+            for (uint32_t u = 0; u < 2; ++u) {
+                if (!ok || j >= unit[u].n_blocks) continue;
+                ok = mbar_wait(p_full + u, j & 1, abort_flag, wait_limit);
+                if (!ok) continue;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                if (lane == 0) {
+                    values(u, j);
+                    if (j + 1 < unit[u].n_blocks) scores(u, j + 1);
+                    else umma_commit(o_full + u);
+                }
+                __syncwarp();
+            }
+            if (ok && lane == 0) {
+                umma_commit(v_empty + s);
+                if (j + 1 < n_blocks) umma_commit(k_empty + s1);
+            }
+            __syncwarp();
+        }
+        if (!ok) {
+            *abort_flag = 1;
+            if (lane == 0) umma_commit(drain);  // the products still in flight
+            __syncwarp();
+            (void)mbar_wait(drain, 0, never, kUmWaitDefault);
+        }
+    } else {
+        const uint32_t u = warp / 4, r = threadIdx.x % 128;
+        const PortionUnit me = u ? unit[1] : unit[0];
+        const uint32_t s_tmem = tmem + 128 * u + (((warp % 4) * 32) << 16), o_tmem = s_tmem - 128 * u + kUmOCol + 128 * u;
+        const int pos = (int)(a.p0 + me.row0 + r);
+        const uint32_t last = a.bias_len - 1;
+        const float factor = query_scale(a, pos) * kLog2E;
+        const float *bias = a.bias ? a.bias + (size_t)me.h * a.bias_len : nullptr;
+        const float far = bias ? bias[last] * kLog2E : 0.f;
+        float m = -INFINITY, l = 0.f;   // the accumulator's reference, the sum of the weights
+        bool ok = true;
+        float2 s[kUmKeys / 2];
+        for (uint32_t j = 0; j < me.n_blocks; ++j) {
+            // distance of the tile's first row to the block's last key; what lies before is masked
+            const int nearest = (int)(a.p0 + me.row0) - (int)(j * kUmKeys + kUmKeys - 1);
+            const bool near = nearest < (int)last || nearest < 0;
+            float *band = bands + (u * 2 + (j & 1)) * 4 * kUmBandPitch;
+            if (near) {
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int at = (int)r + 128 * half, distance = nearest + 2 * kUmKeys - 2 - at;
+                    float b = -INFINITY;
+                    if (distance >= 0) b = bias ? __ldg(bias + min((uint32_t)distance, last)) * kLog2E : 0.f;
+#pragma unroll
+                    for (int c = 0; c < 4; ++c)
+                        if (at >= c) band[c * kUmBandPitch + at - c] = b;
+                }
+            }
+            // (the unit's four warps go on together, or leave together; the band is complete then)
+            ok = unit_vote(u, mbar_wait(s_full + u, j & 1, abort_flag, wait_limit));
+            if (!ok) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            uint32_t raw[4][32];
+#pragma unroll
+            for (int c = 0; c < 4; ++c) tmem_ld32(s_tmem + 32 * c, raw[c]);
+            tmem_ld_wait();
+            const float2 f2 = make_float2(factor, factor);
+            float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+            if (near) {
+                const uint32_t shift = 127 - r;
+                const float4 *bp = reinterpret_cast<const float4 *>(band + (shift & 3) * kUmBandPitch + (shift & ~3u));
+#pragma unroll
+                for (int e = 0; e < kUmKeys / 4; ++e) {
+                    const float4 b = bp[e];
+                    s[2 * e] = __ffma2_rn(make_float2(__uint_as_float(raw[e / 8][e % 8 * 4]), __uint_as_float(raw[e / 8][e % 8 * 4 + 1])),
+                                          f2, make_float2(b.x, b.y));
+                    s[2 * e + 1] = __ffma2_rn(
+                        make_float2(__uint_as_float(raw[e / 8][e % 8 * 4 + 2]), __uint_as_float(raw[e / 8][e % 8 * 4 + 3])), f2,
+                        make_float2(b.z, b.w));
+                }
+            } else {
+                const float2 b2 = make_float2(far, far);
+#pragma unroll
+                for (int e = 0; e < kUmKeys / 2; ++e)
+                    s[e] = __ffma2_rn(make_float2(__uint_as_float(raw[e / 16][e % 16 * 2]), __uint_as_float(raw[e / 16][e % 16 * 2 + 1])),
+                                      f2, b2);
+            }
+#pragma unroll
+            for (int e = 0; e < kUmKeys / 2; ++e) mx[e % 4] = fmaxf(mx[e % 4], fmaxf(s[e].x, s[e].y));
+            const float top = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3]));
+            float alpha = 1.f;
+            if (top > m + kUmLazy) {  // (in the first block always: key 0 is visible to every row)
+                alpha = ex2(m - top);
+                m = top;
+            }
+            if (j > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+                // (the scores' barrier also says that the product before them is complete)
+#pragma unroll 1
+                for (uint32_t c = 0; c < a.vdim; c += 32) {
+                    uint32_t o[32];
+                    tmem_ld32(o_tmem + c, o);
+                    tmem_ld_wait();
+#pragma unroll
+                    for (int e = 0; e < 32; ++e) o[e] = __float_as_uint(__uint_as_float(o[e]) * alpha);
+                    tmem_store32(o_tmem + c, o);
+                }
+            }
+            float2 sum[2] = {make_float2(l * alpha, 0.f), make_float2(0.f, 0.f)};
+            const float2 m2 = make_float2(-m, -m);
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                uint32_t p[32];
+#pragma unroll
+                for (int e = 0; e < 32; ++e) {
+                    const float2 x = __fadd2_rn(s[32 * half + e], m2);
+                    const float2 w = make_float2(ex2(x.x), ex2(x.y));
+                    sum[e % 2] = __fadd2_rn(sum[e % 2], w);
+                    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(p[e]) : "f"(w.y), "f"(w.x));
+                }
+                tmem_store32(s_tmem + 32 * half, p);
+            }
+            l = (sum[0].x + sum[0].y) + (sum[1].x + sum[1].y);
+            asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            __syncwarp();
+            if (lane == 0) mbar_arrive(p_full + u);
+        }
+        if (me.n_blocks && ok) ok = mbar_wait(o_full + u, 0, abort_flag, wait_limit);
+        if (!ok) *abort_flag = 1;
+        if (me.n_blocks && ok) {
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            const float inv = 1.0f / l;
+            const uint32_t t = me.row0 + r;
+            uint16_t *dst = (uint16_t *)a.out + (size_t)t * a.out_stride + me.h * a.vdim;
+#pragma unroll 1
+            for (uint32_t c = 0; c < a.vdim; c += 32) {
+                uint32_t o[32];
+                tmem_ld32(o_tmem + c, o);
+                tmem_ld_wait();
+                if (t >= a.tokens) continue;
+#pragma unroll
+                for (int e = 0; e < 32; e += 8) {
+                    if (c + e >= a.vdim) break;
+                    uint32_t w[4];
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        w[i] = pack_bf16(__uint_as_float(o[e + 2 * i]) * inv, __uint_as_float(o[e + 2 * i + 1]) * inv);
+                    *reinterpret_cast<uint4 *>(dst + c + e) = make_uint4(w[0], w[1], w[2], w[3]);
+                }
+            }
+        }
+    }
+    __syncwarp();
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 8 && *abort_flag) {  // the copies still in flight
+        (void)mbar_wait(q_full, 0, never, kUmWaitDefault);
+        for (uint32_t j = fetched > kUmStages ? fetched - kUmStages : 0; j < fetched; ++j) {
+            (void)mbar_wait(k_full + j % kUmStages, (j / kUmStages) & 1, never, kUmWaitDefault);
+            (void)mbar_wait(v_full + j % kUmStages, (j / kUmStages) & 1, never, kUmWaitDefault);
+        }
+    }
+    if (warp == 9)
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(kUmTmemCols) : "memory");
+    if (threadIdx.x == 0 && *abort_flag) atomicOr(a.error, 1);
+}
+
 // ------------------------------------------------------------------ plain, float32 arithmetic
 // Grid (splits, query heads, rows).  Tiles of 128 keys: a thread scores one key, then owns value
 // channels threadIdx.x, + 128, ...
@@ -663,6 +1022,25 @@ qk_status enter(qk_ctx *ctx, const qk_grouped_call *d, qk_ctx **out, GroupedArgs
         (c)->launches++;                                                                                               \
     } while (0)
 
+qk_status launch_portion_umma(qk_ctx *c, const qk_grouped_call *d, const GroupedArgs &a) {
+    CUtensorMap qm, km, vm;
+    qk_status st;
+    const size_t n_keys = d->first_position + d->tokens;  // (rows behind them are filled with zeros)
+    const uint16_t *k = (const uint16_t *)d->cache_k + d->slot * d->kv_heads * d->s_max * d->dim_stride;
+    const uint16_t *v = (const uint16_t *)d->cache_v + d->slot * d->kv_heads * d->s_max * d->vdim_stride;
+    const cuuint64_t q_dims[2] = {d->proj_stride, d->tokens}, q_strides[1] = {d->proj_stride * 2};
+    const cuuint64_t k_dims[3] = {d->dim_stride, n_keys, d->kv_heads}, k_strides[2] = {d->dim_stride * 2, d->s_max * d->dim_stride * 2};
+    const cuuint64_t v_dims[3] = {d->vdim_stride, n_keys, d->kv_heads}, v_strides[2] = {d->vdim_stride * 2, d->s_max * d->vdim_stride * 2};
+    const cuuint32_t box[3] = {64, 128, 1};
+    if ((st = encode_bf16_map(d->proj, 2, q_dims, q_strides, box, &qm)) != QK_OK) return st;
+    if ((st = encode_bf16_map(k, 3, k_dims, k_strides, box, &km)) != QK_OK) return st;
+    if ((st = encode_bf16_map(v, 3, v_dims, v_strides, box, &vm)) != QK_OK) return st;
+    const uint32_t units = (a.heads / a.kv_heads) * (uint32_t)qk::ceil_div(d->tokens, kUmRows);
+    const dim3 grid(a.kv_heads, (units + 1) / 2), block(kUmThreads);
+    QK_GROUPED(c, grouped_portion_umma_kernel, grid, block, kUmSmem, qm, km, vm, a, c->wait_limit ? c->wait_limit : kUmWaitDefault);
+    return QK_OK;
+}
+
 qk_status launch_append(qk_ctx *c, const qk_grouped_call *d, const GroupedArgs &a) {
     const dim3 grid(a.tokens), block(256);
     if (d->proj_dtype == QK_F32 && d->cache_dtype == QK_F32) QK_GROUPED(c, (grouped_append_kernel<float, float>), grid, block, 0, a);
@@ -737,6 +1115,10 @@ qk_status qk_grouped_portion(qk_ctx *ctx, const qk_grouped_call *d) {
     if (d->out_stride % 2 || d->out_stride < d->heads * d->vdim_stride)
         return qk::fail(QK_ERR_VALUE, "qk_grouped_portion: output rows of %zu", d->out_stride);
     if (d->tokens == 0) return QK_OK;
+    auto aligned = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
+    if (a.dim >= 64 && a.vdim >= 64 && widest <= 128 && a.out_stride % 8 == 0 && aligned(d->proj) && aligned(d->out) &&
+        aligned(d->cache_k) && aligned(d->cache_v) && c->decode_attention_kernel != 0)
+        return launch_portion_umma(c, d, a);
     const dim3 grid((unsigned)qk::ceil_div(d->tokens, kPortQ), a.heads), block(128);
     if (widest <= 64) QK_GROUPED(c, grouped_portion_kernel<64>, grid, block, PortShape<64>::kSmem, a);
     else if (widest <= 128) QK_GROUPED(c, grouped_portion_kernel<128>, grid, block, PortShape<128>::kSmem, a);
