@@ -39,6 +39,11 @@ struct GroupedArgs {
 };
 // dim and vdim are strides: multiples of 16 with zeros behind the entries.
 
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ float query_scale(const GroupedArgs &a, int pos) {
     if (a.temp_every == 0.0) return a.scale;
     const float steps = (float)floor((double)(pos + 1) / a.temp_every);
@@ -153,12 +158,13 @@ template <int DM> struct RowShape {
     static constexpr size_t kSmem = kRing > kSums ? kRing : kSums;
 };
 // Grid (splits, key/value heads x groups of eight query heads, rows); four warps, each with key tiles of
-// its own.
-template <int DM>
+// its own.  FULL: both head strides are DM.
+template <int DM, bool FULL>
 __global__ void __launch_bounds__(128)
-grouped_rows_kernel(GroupedArgs a) {
+grouped_rows_kernel(const __grid_constant__ GroupedArgs a) {
     using S = RowShape<DM>;
     constexpr int kSteps = DM / 16, kKeyTiles = S::kKeys / 8;
+    const uint32_t dim = FULL ? (uint32_t)DM : a.dim, vdim = FULL ? (uint32_t)DM : a.vdim;
     qk::pdl_launch();
     extern __shared__ __align__(16) uint8_t row_smem[];
     const uint32_t t = blockIdx.z, warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane >> 2, c4 = lane & 3;
@@ -179,22 +185,31 @@ grouped_rows_kernel(GroupedArgs a) {
     const uint32_t cached = a.append ? n_keys - 1 - first : count;  // (the newest key is not in the cache yet)
     const uint32_t n_tiles = (count + S::kKeys - 1) / S::kKeys;
     const size_t head_row = ((size_t)a.slots[t] * a.kv_heads + kvh) * a.s_max;
-    const uint16_t *kb = (const uint16_t *)a.cache_k + (head_row + first) * a.dim;
-    const uint16_t *vb = (const uint16_t *)a.cache_v + (head_row + first) * a.vdim;
+    const uint16_t *kb = (const uint16_t *)a.cache_k + (head_row + first) * dim;
+    const uint16_t *vb = (const uint16_t *)a.cache_v + (head_row + first) * vdim;
     uint8_t *ring = row_smem + warp * S::kBufs * S::kTile;
+    // a lane copies one column piece of every kStride-th key
+    constexpr uint32_t kPieces = DM / 8, kStride = 32 / kPieces ? 32 / kPieces : 1;
+    const uint32_t piece = lane % kPieces * 8, key0 = lane / kPieces, end = min(cached, count);
+    const bool in_k = FULL || piece < dim, in_v = FULL || piece < vdim;
     auto fetch = [&](uint32_t i) {  // this warp's i-th tile
         const uint32_t k0 = (warp + 4 * i) * S::kKeys;
         if (k0 < count) {
-            uint8_t *kt = ring + (i % S::kBufs) * S::kTile, *vt = kt + S::kTile / 2;
-            const uint32_t end = min(cached, count);
+            uint8_t *kt = ring + (i % S::kBufs) * S::kTile + (key0 * S::kPitch + piece) * 2;
+            const uint16_t *ks = kb + (size_t)(k0 + key0) * dim + piece, *vs = vb + (size_t)(k0 + key0) * vdim + piece;
+            if (k0 + S::kKeys <= end) {
 #pragma unroll
-            for (int x = lane; x < S::kKeys * (DM / 8); x += 32) {
-                const uint32_t key = x / (DM / 8), c = x % (DM / 8) * 8;
-                const bool live = k0 + key < end;
-                if (c < a.dim)
-                    copy16(kt + (key * S::kPitch + c) * 2, live ? kb + (size_t)(k0 + key) * a.dim + c : kb, live ? 16u : 0u);
-                if (c < a.vdim)
-                    copy16(vt + (key * S::kPitch + c) * 2, live ? vb + (size_t)(k0 + key) * a.vdim + c : vb, live ? 16u : 0u);
+                for (int x = 0; x < S::kKeys; x += kStride) {
+                    if (in_k) copy16(kt + x * S::kPitch * 2, ks + x * dim, 16u);
+                    if (in_v) copy16(kt + S::kTile / 2 + x * S::kPitch * 2, vs + x * vdim, 16u);
+                }
+            } else {
+#pragma unroll 1
+                for (int x = 0; x < S::kKeys; x += kStride) {
+                    const bool live = k0 + key0 + x < end;
+                    if (in_k) copy16(kt + x * S::kPitch * 2, live ? ks + x * dim : kb, live ? 16u : 0u);
+                    if (in_v) copy16(kt + S::kTile / 2 + x * S::kPitch * 2, live ? vs + x * vdim : vb, live ? 16u : 0u);
+                }
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -256,7 +271,7 @@ grouped_rows_kernel(GroupedArgs a) {
         for (int n = 0; n < kKeyTiles; ++n) s[n][0] = s[n][1] = s[n][2] = s[n][3] = 0.f;
 #pragma unroll
         for (int ks = 0; ks < kSteps; ++ks) {
-            if (ks * 16 >= (int)a.dim) break;
+            if (ks * 16 >= (int)dim) break;
 #pragma unroll
             for (int pr = 0; pr < kKeyTiles / 2; ++pr) {
                 uint32_t b[4];
@@ -267,7 +282,7 @@ grouped_rows_kernel(GroupedArgs a) {
         }
         // scores of head g, keys k0 + 8 n + 2 c4 + e
         const uint32_t back0 = n_keys - 1 - first - k0;  // distance of the tile's first key
-        const bool all_far = back0 + 1 >= S::kKeys + last;
+        const bool near = bias && back0 + 1 < S::kKeys + last, ragged = k0 + S::kKeys > count;
         float x[kKeyTiles][2], mx = m;
 #pragma unroll
         for (int n = 0; n < kKeyTiles; ++n)
@@ -275,29 +290,32 @@ grouped_rows_kernel(GroupedArgs a) {
             for (int e = 0; e < 2; ++e) {
                 const uint32_t key = 8 * n + 2 * c4 + e;
                 float b = far;
-                if (bias && !all_far) b = __ldg(bias + (key <= back0 ? min(back0 - key, last) : 0u)) * kLog2E;
-                x[n][e] = k0 + key < count ? fmaf(s[n][e] + s[n][e + 2], factor, b) : -INFINITY;
+                if (near) b = __ldg(bias + max(min((int)back0 - (int)key, (int)last), 0)) * kLog2E;
+                x[n][e] = fmaf(s[n][e] + s[n][e + 2], factor, b);
+                if (ragged && k0 + key >= count) x[n][e] = -INFINITY;
                 mx = fmaxf(mx, x[n][e]);
             }
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));  // (a tile's first key is live: mx is finite)
-        const float alpha = exp2f(m - mx);
-        m = mx;
-        l *= alpha;
+        if (__any_sync(0xffffffffu, mx > m)) {
+            const float alpha = ex2(m - mx);
+            m = mx;
+            l *= alpha;
+#pragma unroll
+            for (int n = 0; n < DM / 8; ++n) {
+                o[n][0] *= alpha;
+                o[n][1] *= alpha;
+                o[n][2] *= alpha;
+                o[n][3] *= alpha;
+            }
+        }
 #pragma unroll
         for (int n = 0; n < kKeyTiles; ++n)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                x[n][e] = exp2f(x[n][e] - mx);
+                x[n][e] = ex2(x[n][e] - mx);
                 l += x[n][e];
             }
-#pragma unroll
-        for (int n = 0; n < DM / 8; ++n) {
-            o[n][0] *= alpha;
-            o[n][1] *= alpha;
-            o[n][2] *= alpha;
-            o[n][3] *= alpha;
-        }
 #pragma unroll
         for (int kk = 0; kk < kKeyTiles / 2; ++kk) {
             uint32_t p[4];
@@ -305,7 +323,7 @@ grouped_rows_kernel(GroupedArgs a) {
             split_bf16(x[2 * kk + 1][0], x[2 * kk + 1][1], p[2], p[3]);
 #pragma unroll
             for (int n = 0; n < DM / 8; n += 2) {
-                if (n * 8 >= (int)a.vdim) break;
+                if (n * 8 >= (int)vdim) break;
                 uint32_t b[4];
                 ldsm4_trans(b, vt + ((kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * S::kPitch + (n + (lane >> 4)) * 8) * 2);
                 mma16(o[n], p, b[0], b[1]);
@@ -549,11 +567,6 @@ constexpr float kUmLazy = 8.0f;
 constexpr uint32_t kUmWaitDefault = 1u << 22;
 static_assert(kUmSmem <= 227 * 1024, "the tiles must fit the shared memory of a CTA");
 
-__device__ __forceinline__ float ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 __device__ __forceinline__ void tmem_store32(uint32_t taddr, const uint32_t *v) {
     asm volatile(
         "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
@@ -1085,9 +1098,12 @@ qk_status qk_grouped_attention(qk_ctx *ctx, const qk_grouped_call *d) {
     const uint32_t widest = std::max(a.dim, a.vdim), group = a.heads / a.kv_heads;
     if (d->cache_dtype == QK_BF16 && widest <= 256 && c->decode_attention_kernel != 0) {
         const dim3 grid(a.n_splits, a.kv_heads * ((group + 7) / 8), a.tokens), block(128);
-        if (widest <= 64) QK_GROUPED(c, grouped_rows_kernel<64>, grid, block, RowShape<64>::kSmem, a);
-        else if (widest <= 128) QK_GROUPED(c, grouped_rows_kernel<128>, grid, block, RowShape<128>::kSmem, a);
-        else QK_GROUPED(c, grouped_rows_kernel<256>, grid, block, RowShape<256>::kSmem, a);
+        const bool full = a.dim == a.vdim;
+        if (widest == 64 && full) QK_GROUPED(c, (grouped_rows_kernel<64, true>), grid, block, RowShape<64>::kSmem, a);
+        else if (widest <= 64) QK_GROUPED(c, (grouped_rows_kernel<64, false>), grid, block, RowShape<64>::kSmem, a);
+        else if (widest == 128 && full) QK_GROUPED(c, (grouped_rows_kernel<128, true>), grid, block, RowShape<128>::kSmem, a);
+        else if (widest <= 128) QK_GROUPED(c, (grouped_rows_kernel<128, false>), grid, block, RowShape<128>::kSmem, a);
+        else QK_GROUPED(c, (grouped_rows_kernel<256, false>), grid, block, RowShape<256>::kSmem, a);
         return QK_OK;
     }
     if (d->vdim_stride > kPlainKeys * kPlainChannels || d->dim_stride > 8192)

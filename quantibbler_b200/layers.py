@@ -495,7 +495,7 @@ class GroupedAttention:
         """Key splits: about two blocks per SM, 64 keys or more each."""
         group = self.heads // self.kv_heads
         blocks = rows * (self.kv_heads * -(-group // 8) if self.tiled else self.heads)
-        return max(1, min(32, 296 // blocks, -(-max_seq // 64)))
+        return max(1, min(24, 296 // blocks, -(-max_seq // 64)))
 
     def _scratch(self, rows: Rows, n_splits: int):
         """Partial results and counters (zero between calls) for this number of rows and splits."""
