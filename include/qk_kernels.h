@@ -650,13 +650,13 @@ typedef struct {
     const int32_t *table, *places, *offsets, *tiles;
 } qk_dense_call;
 /* Sorts the choices of `tokens` rows by expert, for n_jobs tables at once (one launch).  tiles:
- * the number of tiles, then per tile its expert, first and last + 1 place, every tile at most
- * tile_rows (qk_route_tile_rows) places of one expert; room for ceil(tokens * top / tile_rows) +
- * experts tiles.  The launch lets no dependent kernel start early: a kernel after it may read
+ * the number of tiles, then per tile its expert, first and last + 1 place, the first tile and the
+ * number of tiles of its expert; a tile is at most tile_rows (qk_route_tile_rows) places of one
+ * expert; room for ceil(tokens * top / tile_rows) + experts tiles.  The launch lets no dependent kernel start early: a kernel after it may read
  * these before its own dependency wait. */
 typedef struct {
     const int32_t *table;                    /* [vocab][top] */
-    int32_t *places, *offsets, *tiles;       /* [tokens][top], [experts + 1], [1 + 3 * tiles] */
+    int32_t *places, *offsets, *tiles;       /* [tokens][top], [experts + 1], [1 + 5 * tiles] */
     uint64_t top, experts;
 } qk_route_job;
 qk_status qk_route(qk_ctx *ctx, const qk_route_job *device_jobs, size_t n_jobs, size_t max_experts, const int32_t *ids,

@@ -20,9 +20,10 @@
 namespace {
 
 constexpr int kVecThreads = 256, kVecWarps = kVecThreads / 32;
+constexpr int kRouteTile = 5;  // a tile of qk_route: expert, first and last + 1 place, the expert's first tile, its tiles
 constexpr int kVectorTokens = 4;
 constexpr int kNarrowTokens = 128;
-constexpr size_t kVecSmemMax = 200 * 1024;
+constexpr size_t kVecSmemMax = 200 * 1024, kVecSmemSm = 226 * 1024;  // of a block, of an SM
 
 // ------------------------------------------------------------------ vector form
 template <typename W> struct VecTraits;
@@ -77,26 +78,31 @@ __device__ __forceinline__ void vec_fma(float (&acc)[NT], const uint4 &w, const 
     }
 }
 
-// A warp (or `ksplit` warps that share out the k range) owns R weight rows; with a gated pair,
-// R / 2 gate rows and their up rows.
+// A warp (or `ksplit` warps that share out the k range) owns R weight rows at a time (with a gated
+// pair, R / 2 gate rows and their up rows).  As many blocks as stay resident walk over the rows, so
+// that each forms the input once; the next rows' first weights are requested while the last ones
+// of the present rows are multiplied.
 // (The blocks per SM matter more than a spilled register: they hide each other's prologues.)
+__host__ __device__ constexpr int vec_blocks(int nt, int r) { return nt == 4 && r == 4 ? 2 : r == 1 && nt <= 2 ? 4 : 3; }
+enum { kRowAny = 0, kRowNorm = 1, kRowPlain = 2 };  // how the input rows may be read
 template <typename W, int NT, int R>
-__global__ void __launch_bounds__(kVecThreads, NT == 4 && R == 4 ? 2 : R == 1 && NT <= 2 ? 4 : 3)
+__global__ void __launch_bounds__(kVecThreads, vec_blocks(NT, R))
 dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint32_t rows, uint32_t w_stride,
-                    uint32_t n_tokens, uint32_t ksplit, ChoiceArgs ch) {
+                    uint32_t n_tokens, uint32_t ksplit, ChoiceArgs ch, int row_kind) {
     using T = VecTraits<W>;
     constexpr int U = R >= 4 ? 2 : 4;  // steps in flight
     constexpr int HR = R >= 2 ? R / 2 : 1;
     qk::pdl_launch();
-    extern __shared__ __align__(16) float xs[];  // [NT][pitch]
+    extern __shared__ __align__(16) float xs[];  // [NT][pitch], staged norm weights [2][width]
     __shared__ float red[kVecWarps];
-    __shared__ float part_sum[kVecWarps][R * NT];
+    __shared__ float part_sum[2][kVecWarps][R * NT];
     const uint32_t warp = threadIdx.x / 32, lane = threadIdx.x % 32;
     const uint32_t k = in.k, pitch = (k + T::kStep - 1) / T::kStep * T::kStep, steps = pitch / T::kStep;
-    const uint32_t group = (blockIdx.x * kVecWarps + warp) / ksplit, part = warp % ksplit;
+    const uint32_t part = warp % ksplit, batches = (steps + U * ksplit - 1) / (U * ksplit);
     const bool pair = out.kind == QK_OUTPUT_GLU;
-    const W *row[R];
-    uint32_t r0 = group * R, t_in = 0, t_out = 0;  // first input and output row
+    const uint32_t per_block = kVecWarps / ksplit, per_group = pair ? HR : R;
+    const uint32_t groups = ((pair ? rows / 2 : rows) + per_group - 1) / per_group;
+    uint32_t t_in = 0, t_out = 0;  // first input and output row
     bool writer = blockIdx.x == 0;
     if (ch.table) {
         // one choice of one token per block row (NT is 1).  The token ids are written by copies and
@@ -107,97 +113,117 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
         t_in = ch.by_choice ? t_out : t;
         writer = writer && blockIdx.y % ch.top == 0;
     }
+    const W *row[R];   // the rows whose weights are requested next
+    bool any = false;
+    auto turn_to = [&](uint32_t group) {
+        any = group < groups;
 #pragma unroll
-    for (int r = 0; r < R; ++r) {
-        uint32_t n;
-        if (pair) n = pair_row(group * HR + r % HR) + (r >= HR ? 32 : 0);
-        else n = r0 + r;
-        row[r] = w + (size_t)min(n, rows - 1) * w_stride + lane * T::kPer;
-    }
+        for (int r = 0; r < R; ++r) {
+            const uint32_t n = pair ? pair_row(group * HR + r % HR) + (r >= HR ? 32 : 0) : group * R + r;
+            row[r] = w + (size_t)min(n, rows - 1) * w_stride + lane * T::kPer;
+        }
+    };
     uint4 cur[U][R];
     auto fetch = [&](uint32_t s, uint4 (&dst)[R]) {
-        const bool live = s < steps && s * T::kStep + lane * T::kPer < k;
+        const bool live = any && s < steps && s * T::kStep + lane * T::kPer < k;
 #pragma unroll
         for (int r = 0; r < R; ++r)
             dst[r] = live ? load_weights16(row[r] + (size_t)s * T::kStep) : make_uint4(0, 0, 0, 0);
     };
+    uint32_t group = blockIdx.x * per_block + warp / ksplit;
     // weights depend on no other kernel: the first ones are requested before the dependency wait
+    turn_to(group);
 #pragma unroll
     for (int u = 0; u < U; ++u) fetch(part + u * ksplit, cur[u]);
+    float *staged = xs + NT * pitch;
+    if (row_kind == kRowNorm) stage_norm_weights(in, staged);
     qk::pdl_wait();
 #pragma unroll 1
     for (uint32_t t = 0; t < (uint32_t)NT; ++t) {
         float *dst = xs + t * pitch;
         if (t < n_tokens) {
-            build_input(in, t_in + t, writer, [&](uint32_t i) -> float & { return dst[T::place(i)]; }, red);
+            auto at4 = [&](uint32_t p) -> float4 & { return *reinterpret_cast<float4 *>(dst + T::place(4 * p)); };
+            if (row_kind == kRowNorm) build_norm_row(in, t_in + t, writer, staged, at4, red);
+            else if (row_kind == kRowPlain) build_plain_row(in, t_in + t, at4);
+            else build_input(in, t_in + t, writer, [&](uint32_t i) -> float & { return dst[T::place(i)]; }, red);
         }
         // what lies between k and the pitch meets zero weights; it must only be finite
         for (uint32_t i = (t < n_tokens ? k : 0) + threadIdx.x; i < pitch; i += kVecThreads) dst[T::place(i)] = 0.f;
     }
     __syncthreads();
-    float acc[R][NT];
+    uint32_t turn = 0;
+#pragma unroll 1
+    for (uint32_t first = blockIdx.x * per_block; first < groups; first += gridDim.x * per_block, turn ^= 1) {
+        const uint32_t next = group + gridDim.x * per_block;
+        float acc[R][NT];
 #pragma unroll
-    for (int r = 0; r < R; ++r)
+        for (int r = 0; r < R; ++r)
 #pragma unroll
-        for (int t = 0; t < NT; ++t) acc[r][t] = 0.f;
-    for (uint32_t s = part; s < steps; s += U * ksplit) {
+            for (int t = 0; t < NT; ++t) acc[r][t] = 0.f;
+#pragma unroll 1
+        for (uint32_t b = 0; b < batches; ++b) {
+            const bool over = b + 1 == batches;
+            if (over) turn_to(next);
+            const uint32_t ahead = over ? part : part + (b + 1) * U * ksplit;
 #pragma unroll
-        for (int u = 0; u < U; ++u) {
-            uint4 now[R];
+            for (int u = 0; u < U; ++u) {
+                uint4 now[R];
 #pragma unroll
-            for (int r = 0; r < R; ++r) now[r] = cur[u][r];
-            const uint32_t at = s + u * ksplit;
-            fetch(at + U * ksplit, cur[u]);
-            if (at < steps) {
+                for (int r = 0; r < R; ++r) now[r] = cur[u][r];
+                const uint32_t at = part + (b * U + u) * ksplit;
+                fetch(ahead + u * ksplit, cur[u]);
+                if (at < steps) {
 #pragma unroll
-                for (int r = 0; r < R; ++r) vec_fma<W, NT>(acc[r], now[r], xs, pitch, at * T::kStep, lane);
+                    for (int r = 0; r < R; ++r) vec_fma<W, NT>(acc[r], now[r], xs, pitch, at * T::kStep, lane);
+                }
             }
         }
-    }
 #pragma unroll
-    for (int r = 0; r < R; ++r)
+        for (int r = 0; r < R; ++r)
 #pragma unroll
-        for (int t = 0; t < NT; ++t) {
-            float a = acc[r][t];
-            for (int off = 16; off > 0; off >>= 1) a += __shfl_xor_sync(0xffffffffu, a, off);
-            acc[r][t] = a;
+            for (int t = 0; t < NT; ++t) {
+                float a = acc[r][t];
+                for (int off = 16; off > 0; off >>= 1) a += __shfl_xor_sync(0xffffffffu, a, off);
+                acc[r][t] = a;
+            }
+        if (ksplit > 1) {  // (two buffers: the turn after the next finds this one read)
+            if (lane == 0) {
+#pragma unroll
+                for (int r = 0; r < R; ++r)
+#pragma unroll
+                    for (int t = 0; t < NT; ++t) part_sum[turn][warp][r * NT + t] = acc[r][t];
+            }
+            __syncthreads();
+            if (part == 0) {
+#pragma unroll
+                for (int r = 0; r < R; ++r)
+#pragma unroll
+                    for (int t = 0; t < NT; ++t)
+                        for (uint32_t p = 1; p < ksplit; ++p) acc[r][t] += part_sum[turn][warp + p][r * NT + t];
+            }
         }
-    if (ksplit > 1) {
-        if (lane == 0) {
-#pragma unroll
-            for (int r = 0; r < R; ++r)
-#pragma unroll
-                for (int t = 0; t < NT; ++t) part_sum[warp][r * NT + t] = acc[r][t];
-        }
-        __syncthreads();
         if (part == 0) {
+            if (pair) {
+                if constexpr (R >= 2) {
 #pragma unroll
-            for (int r = 0; r < R; ++r)
+                    for (int r = 0; r < R / 2; ++r)
 #pragma unroll
-                for (int t = 0; t < NT; ++t)
-                    for (uint32_t p = 1; p < ksplit; ++p) acc[r][t] += part_sum[warp + p][r * NT + t];
-        }
-    }
-    if (part == 0) {
-        if (pair) {
-            if constexpr (R >= 2) {
+                        for (int t = 0; t < NT; ++t) {
+                            const uint32_t j = group * (R / 2) + r;
+                            if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && j < rows / 2)
+                                finish_pair(out, t_out + t, j, acc[r][t], acc[r + R / 2][t]);
+                        }
+                }
+            } else {
 #pragma unroll
-                for (int r = 0; r < R / 2; ++r)
+                for (int r = 0; r < R; ++r)
 #pragma unroll
-                    for (int t = 0; t < NT; ++t) {
-                        const uint32_t j = group * (R / 2) + r;
-                        if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && j < rows / 2)
-                            finish_pair(out, t_out + t, j, acc[r][t], acc[r + R / 2][t]);
-                    }
+                    for (int t = 0; t < NT; ++t)
+                        if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && group * R + r < rows)
+                            finish(out, t_out + t, group * R + r, acc[r][t]);
             }
-        } else {
-#pragma unroll
-            for (int r = 0; r < R; ++r)
-#pragma unroll
-                for (int t = 0; t < NT; ++t)
-                    if (lane == (uint32_t)(r * NT + t) && (uint32_t)t < n_tokens && r0 + r < rows)
-                        finish(out, t_out + t, r0 + r, acc[r][t]);
         }
+        group = next;
     }
     if (in.append.src && blockIdx.x == gridDim.x - 1)
         for (uint32_t t = 0; t < n_tokens; ++t) append_latent(in, t, red);
@@ -242,7 +268,7 @@ dense_f32_kernel(const float *__restrict__ x, uint32_t x_stride, uint32_t k, con
     const uint32_t n0 = blockIdx.x * kFTile;
     if (tiles) {  // rows sorted by expert
         if (blockIdx.y >= (uint32_t)tiles[0]) return;
-        const int32_t *tile = tiles + 1 + 3 * blockIdx.y;
+        const int32_t *tile = tiles + 1 + kRouteTile * blockIdx.y;
         w += (size_t)tile[0] * rows * w_stride;
         t0 = (uint32_t)tile[1];
         n_tokens = (uint32_t)tile[2];
@@ -308,15 +334,21 @@ struct TcArgs {
     int *error;
     const int32_t *expert_tiles;  // rows sorted by expert: the token tiles (qk_route); null: one matrix
 };
-// Tile `tile` of the walk over token tiles (fastest) and weight tiles.
+// Tile `tile` of the walk over weight tiles and, fastest, the token tiles that share one; with experts
+// the walk goes from expert to expert.
 struct TcTile {
     uint32_t t0, t_end, n0, w0;  // rows of x, first output column, first row of W
 };
 template <int BN>
-__device__ __forceinline__ TcTile tc_tile(const TcArgs &g, uint32_t m_tiles, uint32_t tile) {
-    const uint32_t m = tile % m_tiles, n0 = (tile / m_tiles) * BN;
-    if (!g.expert_tiles) return {m * kTcM, g.n_tokens, n0, n0};
-    const int32_t *e = g.expert_tiles + 1 + 3 * m;
+__device__ __forceinline__ TcTile tc_tile(const TcArgs &g, uint32_t tile) {
+    if (!g.expert_tiles) {
+        const uint32_t n0 = (tile / g.m_tiles) * BN;
+        return {(tile % g.m_tiles) * kTcM, g.n_tokens, n0, n0};
+    }
+    const uint32_t per_row = (g.rows + BN - 1) / BN;
+    const int32_t *any = g.expert_tiles + 1 + kRouteTile * (tile / per_row);  // (a tile of the same expert)
+    const uint32_t first = (uint32_t)any[3], count = (uint32_t)any[4], at = tile - first * per_row, n0 = at / count * BN;
+    const int32_t *e = g.expert_tiles + 1 + kRouteTile * (first + at % count);
     return {(uint32_t)e[1], (uint32_t)e[2], n0, (uint32_t)e[0] * g.rows + n0};
 }
 __device__ __forceinline__ uint32_t tc_idesc(uint32_t bn) {
@@ -451,14 +483,13 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     qk::pdl_wait();
     const uint32_t tmem_base = *tmem_slot;
-    const uint32_t m_tiles = g.expert_tiles ? (uint32_t)g.expert_tiles[0] : g.m_tiles;
-    const uint32_t n_tiles = g.expert_tiles ? m_tiles * ((g.rows + BN - 1) / BN) : g.tiles;
+    const uint32_t n_tiles = g.expert_tiles ? (uint32_t)g.expert_tiles[0] * ((g.rows + BN - 1) / BN) : g.tiles;
 
     if (warp == 0) {
         uint32_t gc = 0;
         bool dead = false;
         for (uint32_t tile = blockIdx.x; tile < n_tiles && !dead; tile += gridDim.x) {
-            const TcTile at = tc_tile<BN>(g, m_tiles, tile);
+            const TcTile at = tc_tile<BN>(g, tile);
             for (uint32_t kc = 0; kc < g.k_chunks; ++kc, ++gc) {
                 const uint32_t s = gc % S::kStages;
                 if (!mbar_wait(&empty[s], ((gc / S::kStages) & 1) ^ 1, abort_flag, g.wait_limit)) {
@@ -534,7 +565,7 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
         uint32_t seg = 0;
         for (uint32_t tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, ++seg) {
             const uint32_t acc = seg & 1;
-            const TcTile at = tc_tile<BN>(g, m_tiles, tile);
+            const TcTile at = tc_tile<BN>(g, tile);
             const uint32_t t0 = at.t0 + quarter * 32, n0 = at.n0;
             float *stage = epi + (warp - 2) * 32 * kEpiPitch;
             if (!tc_epilogue_vote(mbar_wait(&acc_full[acc], (seg >> 1) & 1, abort_flag, g.wait_limit))) {
@@ -555,9 +586,12 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant
                     if (out.act == QK_ACT_RELU) {
 #pragma unroll
                         for (int j = 0; j < 32; ++j) v[j] = fmaxf(__uint_as_float(a[j]), 0.f) * __uint_as_float(b[j]);
+                    } else if (out.act == QK_ACT_SILU) {
+#pragma unroll
+                        for (int j = 0; j < 32; ++j) v[j] = silu_f(__uint_as_float(a[j])) * __uint_as_float(b[j]);
                     } else {
 #pragma unroll
-                        for (int j = 0; j < 32; ++j) v[j] = activate(out.act, __uint_as_float(a[j])) * __uint_as_float(b[j]);
+                        for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_f(__uint_as_float(a[j])) * __uint_as_float(b[j]);
                     }
                     tc_store_tile<KIND>(out, t0, at.t_end, (n0 + c) / 2, g.rows / 2, v, stage, lane, vec != 0);
                 } else {
@@ -939,6 +973,13 @@ qk_status encode_map(const void *base, size_t rows, size_t k, size_t stride, uin
     return encode_bf16_map(base, 2, dims, strides, box, out);
 }
 
+// Rows of x and of W as the matrix forms see them, and their row tiles.
+size_t input_rows(const qk_dense_call &d) { return d.experts ? d.tokens * d.top : d.tokens; }
+size_t weight_rows(const qk_dense_call &d) { return d.experts ? d.rows * d.experts : d.rows; }
+size_t row_tiles(const qk_dense_call &d, size_t tile) {
+    return qk::ceil_div(input_rows(d), tile) + (d.experts ? std::min(d.experts, input_rows(d)) : 0);
+}
+
 // Weight rows per tile: the width whose number of waves over the SMs costs least.
 int pick_tile(size_t m_tiles, size_t rows, size_t sms) {
     int best = 64;
@@ -949,13 +990,6 @@ int pick_tile(size_t m_tiles, size_t rows, size_t sms) {
         if (cost < best_cost) best = bn, best_cost = cost;
     }
     return best;
-}
-
-// Rows of x and of W as the matrix forms see them, and their row tiles.
-size_t input_rows(const qk_dense_call &d) { return d.experts ? d.tokens * d.top : d.tokens; }
-size_t weight_rows(const qk_dense_call &d) { return d.experts ? d.rows * d.experts : d.rows; }
-size_t row_tiles(const qk_dense_call &d, size_t tile) {
-    return qk::ceil_div(input_rows(d), tile) + (d.experts ? std::min(d.experts, input_rows(d)) : 0);
 }
 
 template <int BN, int KIND>
@@ -1048,21 +1082,39 @@ qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_ca
     }
 }
 
+// Which of the faster ways to read the input rows applies.
+int vector_row_kind(const InputArgs &a) {
+    auto aligned = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
+    if (a.width % 4 || a.k % 4 || a.x_stride % 4 || !aligned(a.x)) return kRowAny;
+    if (a.kind == QK_INPUT_PLAIN) return kRowPlain;
+    if (a.kind != QK_INPUT_NORM || a.width > 1024 * kNormPieces || !aligned(a.x_out)) return kRowAny;
+    if (a.norm != QK_NORM_NONE && !aligned(a.norm_weight)) return kRowAny;
+    if (a.pending && (a.pending_stride % 4 || !aligned(a.pending) || !aligned(a.pending_weight))) return kRowAny;
+    return kRowNorm;
+}
+
 template <typename W, int NT, int R>
 qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
                           size_t n_tokens, uint32_t ks) {
     const size_t step = VecTraits<W>::kStep;
-    const size_t smem = NT * qk::ceil_div(d.k, step) * step * 4;
+    int kind = vector_row_kind(in);
+    size_t smem = NT * qk::ceil_div(d.k, step) * step * 4;
+    if (kind == kRowNorm && smem + 8 * d.width > kVecSmemMax) kind = kRowAny;
+    if (kind == kRowNorm) smem += 8 * d.width;
     const size_t groups = d.output == QK_OUTPUT_GLU ? qk::ceil_div(d.rows / 2, R / 2 ? R / 2 : 1)
                                                     : qk::ceil_div(d.rows, R);
     QK_CUDA(cudaFuncSetAttribute(dense_vector_kernel<W, NT, R>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)std::max(smem, (size_t)48 * 1024)));
     ChoiceArgs ch{};
     if (d.experts) ch = ChoiceArgs{d.table, d.ids, (uint32_t)d.top, (uint32_t)d.vocab, d.by_choice ? 1u : 0u};
-    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>,
-                         dim3((unsigned)qk::ceil_div(groups * ks, kVecWarps), (unsigned)(d.experts ? input_rows(d) : 1)),
+    const size_t choices = d.experts ? input_rows(d) : 1;
+    // the blocks that stay resident, shared out evenly among the choices
+    const size_t per_sm = std::max<size_t>(1, std::min<size_t>(vec_blocks(NT, R), kVecSmemSm / (smem + 2048)));
+    const size_t resident = std::max<size_t>(1, per_sm * (size_t)c->sm_count / choices);
+    const size_t blocks = qk::ceil_div(groups * ks, kVecWarps), turns = qk::ceil_div(blocks, resident);
+    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>, dim3((unsigned)qk::ceil_div(blocks, turns), (unsigned)choices),
                          dim3(kVecThreads), smem, c->stream, in, out, (const W *)d.w, (uint32_t)d.rows,
-                         (uint32_t)d.w_stride, (uint32_t)n_tokens, ks, ch);
+                         (uint32_t)d.w_stride, (uint32_t)n_tokens, ks, ch, kind);
     QK_CUDA(cudaGetLastError());
     c->launches++;
     return QK_OK;
@@ -1233,10 +1285,12 @@ route_kernel(const qk_route_job *__restrict__ jobs, const int32_t *__restrict__ 
                 next[e] = first;
                 j.offsets[e] = (int32_t)first;
                 for (uint32_t k = 0; k < own; ++k) {
-                    int32_t *t = j.tiles + 1 + 3 * (tile0 + k);
+                    int32_t *t = j.tiles + 1 + kRouteTile * (tile0 + k);
                     t[0] = (int32_t)e;
                     t[1] = (int32_t)(first + k * tile_rows);
                     t[2] = (int32_t)min(first + (k + 1) * tile_rows, first + count);
+                    t[3] = (int32_t)tile0;
+                    t[4] = (int32_t)own;
                 }
             }
             places += __shfl_sync(0xffffffffu, p, 31);

@@ -14,8 +14,10 @@ namespace {
 
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float silu_f(float z) { return __fdividef(z, 1.0f + expf(-z)); }
+// 0.5 z (1 + tanh u) = z sigmoid(2 u)
 __device__ __forceinline__ float gelu_tanh_f(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return __fdividef(z, 1.0f + expf(-2.0f * u));
 }
 __device__ __forceinline__ float activate(int kind, float z) {
     return kind == QK_ACT_RELU ? fmaxf(z, 0.f) : kind == QK_ACT_SILU ? silu_f(z) : gelu_tanh_f(z);
@@ -172,6 +174,123 @@ __device__ __forceinline__ void build_input(const InputArgs &a, uint32_t t, bool
     } else {
         for (uint32_t i = n + threadIdx.x; i < a.k; i += blockDim.x) at(i) = 0.f;
     }
+    __syncthreads();
+}
+
+// The same for a normed row of up to 1024 kNormPieces aligned entries, for 256 threads: all loads of the
+// row go out together, the norms' weights have been staged by stage_norm_weights (which depends on no
+// other kernel).  `at4(p)` is the shared-memory place of entries 4 p .. 4 p + 3.
+constexpr int kNormPieces = 4;
+__device__ __forceinline__ void stage16(float *smem, const float *gmem) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem) : "memory");
+}
+// staged: [2][width] floats (every thread reads back only what it has copied itself)
+__device__ __forceinline__ void stage_norm_weights(const InputArgs &a, float *staged) {
+    for (uint32_t p = threadIdx.x; p < a.width / 4; p += 256) {
+        if (a.norm != QK_NORM_NONE) stage16(staged + 4 * p, a.norm_weight + 4 * p);
+        if (a.pending) stage16(staged + a.width + 4 * p, a.pending_weight + 4 * p);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+}
+template <typename At4>
+__device__ __forceinline__ void build_norm_row(const InputArgs &a, uint32_t t, bool writer, const float *staged, At4 &&at4,
+                                               float *red) {
+    const uint32_t n = a.width, pieces = n / 4;
+    const float4 *xr = reinterpret_cast<const float4 *>(a.x + (size_t)t * a.x_stride);
+    const float4 *nw = reinterpret_cast<const float4 *>(staged), *pw = nw + pieces;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 h[kNormPieces];
+#pragma unroll
+    for (int j = 0; j < kNormPieces; ++j) {
+        const uint32_t p = threadIdx.x + 256 * j;
+        h[j] = p < pieces ? xr[p] : zero;
+    }
+    if (a.pending) {
+        const uint32_t parts = a.pending_top ? a.pending_top : 1;
+        float4 y[kNormPieces];
+        for (uint32_t c = 0; c < parts; ++c) {
+            const float4 *pr = reinterpret_cast<const float4 *>(
+                a.pending_top ? pending_row(a, t, c) : a.pending + (size_t)t * a.pending_stride);
+#pragma unroll
+            for (int j = 0; j < kNormPieces; ++j) {
+                const uint32_t p = threadIdx.x + 256 * j;
+                const float4 v = p < pieces ? pr[p] : zero;
+                y[j] = c ? make_float4(y[j].x + v.x, y[j].y + v.y, y[j].z + v.z, y[j].w + v.w) : v;
+            }
+        }
+        const float share = a.pending_top ? a.pending_scale : 1.f;
+        float ps = 0.f;
+#pragma unroll
+        for (int j = 0; j < kNormPieces; ++j) {
+            y[j] = make_float4(y[j].x * share, y[j].y * share, y[j].z * share, y[j].w * share);
+            ps += y[j].x * y[j].x + y[j].y * y[j].y + y[j].z * y[j].z + y[j].w * y[j].w;
+        }
+        const float inv = 1.0f / sqrtf(in_block_sum(ps, red) / (float)n + a.pending_eps);
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        float4 *xo = writer && a.x_out ? reinterpret_cast<float4 *>(a.x_out + (size_t)t * a.x_stride) : nullptr;
+#pragma unroll
+        for (int j = 0; j < kNormPieces; ++j) {
+            const uint32_t p = threadIdx.x + 256 * j;
+            if (p >= pieces) continue;
+            const float4 w = pw[p];
+            h[j].x += y[j].x * inv * w.x;
+            h[j].y += y[j].y * inv * w.y;
+            h[j].z += y[j].z * inv * w.z;
+            h[j].w += y[j].w * inv * w.w;
+            if (xo) xo[p] = h[j];
+        }
+    } else if (writer && a.x_out) {
+        float4 *xo = reinterpret_cast<float4 *>(a.x_out + (size_t)t * a.x_stride);
+#pragma unroll
+        for (int j = 0; j < kNormPieces; ++j)
+            if (threadIdx.x + 256 * j < pieces) xo[threadIdx.x + 256 * j] = h[j];
+    }
+    float mean = 0.f, inv = 1.f;
+    if (a.norm == QK_NORM_LAYER) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < kNormPieces; ++j) s += h[j].x + h[j].y + h[j].z + h[j].w;
+        mean = in_block_sum(s, red) / (float)n;
+    }
+    if (a.norm != QK_NORM_NONE) {
+        float s = 0.f;
+#pragma unroll
+        for (int j = 0; j < kNormPieces; ++j) {
+            if (threadIdx.x + 256 * j >= pieces) continue;
+            const float b = h[j].x - mean, c = h[j].y - mean, d = h[j].z - mean, e = h[j].w - mean;
+            s += b * b + c * c + d * d + e * e;
+        }
+        inv = 1.0f / sqrtf(in_block_sum(s, red) / (float)n + a.norm_eps);
+    }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+#pragma unroll
+    for (int j = 0; j < kNormPieces; ++j) {
+        const uint32_t p = threadIdx.x + 256 * j;
+        if (p >= pieces) continue;
+        float4 v = h[j];
+        if (a.norm != QK_NORM_NONE) {
+            const float4 w = nw[p];
+            v = make_float4((v.x - mean) * inv * w.x, (v.y - mean) * inv * w.y, (v.z - mean) * inv * w.z, (v.w - mean) * inv * w.w);
+        }
+        at4(p) = v;
+    }
+    for (uint32_t p = pieces + threadIdx.x; p < a.k / 4; p += 256) at4(p) = zero;
+    __syncthreads();
+}
+// A plain row in aligned pieces.
+template <typename At4>
+__device__ __forceinline__ void build_plain_row(const InputArgs &a, uint32_t t, At4 &&at4) {
+    const uint32_t pieces = a.width / 4;
+    const float4 *xr = reinterpret_cast<const float4 *>(a.x + (size_t)t * a.x_stride);
+    for (uint32_t base = threadIdx.x; base < pieces; base += 8 * 256) {
+        float4 v[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = xr[min(base + 256 * j, pieces - 1)];
+#pragma unroll
+        for (int j = 0; j < 8; ++j)
+            if (base + 256 * j < pieces) at4(base + 256 * j) = v[j];
+    }
+    for (uint32_t p = pieces + threadIdx.x; p < a.k / 4; p += 256) at4(p) = make_float4(0.f, 0.f, 0.f, 0.f);
     __syncthreads();
 }
 

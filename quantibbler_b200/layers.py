@@ -314,7 +314,7 @@ class Route:
         n = cap * table.top
         self.places = torch.zeros(cap, table.top, **i32)
         self.offsets = torch.zeros(table.experts + 1, **i32)
-        self.tiles = torch.zeros(1 + 3 * (-(-n // 64) + table.experts), **i32)
+        self.tiles = torch.zeros(1 + 5 * (-(-n // 64) + table.experts), **i32)
 
 
 class RingCache:

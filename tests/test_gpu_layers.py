@@ -495,7 +495,8 @@ def test_experts(dev, tokens, experts, top, width, ff, serving, tol):
         assert r.offsets.tolist() == [0] + counts.cumsum(0).tolist()
         covered = []
         for n in range(int(r.tiles[0])):
-            e, first, end = r.tiles[1 + 3 * n:4 + 3 * n].tolist()
+            e, first, end, tile0, tiles = r.tiles[1 + 5 * n:6 + 5 * n].tolist()
+            assert tile0 <= n < tile0 + tiles and all(int(r.tiles[1 + 5 * i]) == e for i in range(tile0, tile0 + tiles))
             assert r.offsets[e] <= first < end <= r.offsets[e + 1] and end - first <= 128
             covered += range(first, end)
         assert covered == list(range(tokens * top))
