@@ -1654,7 +1654,7 @@ qk_status qk_argmax_first(qk_ctx *ctx, const float *logits, size_t n_tokens, siz
     if (n_tokens == 0) return QK_OK;
     // partial results live in the context's scratch; it is sized on the first call, so make
     // that call before any stream capture
-    const size_t parts = vocab >= 65536 ? 64 : vocab >= 4096 ? 16 : 1;
+    const size_t parts = vocab >= 16384 ? 64 : vocab >= 4096 ? 16 : 1;
     const size_t slice = qk::ceil_div(vocab, parts);
     if ((st = c->d_z.reserve(n_tokens * parts * 8)) != QK_OK) return st;
     float *part_val = (float *)c->d_z.ptr;

@@ -23,6 +23,7 @@ constexpr int kVecThreads = 256, kVecWarps = kVecThreads / 32;
 constexpr int kRouteTile = 5;  // a tile of qk_route: expert, first and last + 1 place, the expert's first tile, its tiles
 constexpr int kVectorTokens = 4;
 constexpr int kNarrowTokens = 128;
+enum { kRowAny = 0, kRowNorm = 1, kRowPlain = 2 };  // how input rows may be read
 constexpr size_t kVecSmemMax = 200 * 1024, kVecSmemSm = 226 * 1024;  // of a block, of an SM
 
 // ------------------------------------------------------------------ vector form
@@ -81,10 +82,11 @@ __device__ __forceinline__ void vec_fma(float (&acc)[NT], const uint4 &w, const 
 // A warp (or `ksplit` warps that share out the k range) owns R weight rows at a time (with a gated
 // pair, R / 2 gate rows and their up rows).  As many blocks as stay resident walk over the rows, so
 // that each forms the input once; the next rows' first weights are requested while the last ones
-// of the present rows are multiplied.
+// of the present rows are multiplied.  The rows are dealt out block by block before warp by warp:
+// every SM gets its share, wherever blocks that come in early (before the kernel in front has
+// left) find room.
 // (The blocks per SM matter more than a spilled register: they hide each other's prologues.)
 __host__ __device__ constexpr int vec_blocks(int nt, int r) { return nt == 4 && r == 4 ? 2 : r == 1 && nt <= 2 ? 4 : 3; }
-enum { kRowAny = 0, kRowNorm = 1, kRowPlain = 2 };  // how the input rows may be read
 template <typename W, int NT, int R>
 __global__ void __launch_bounds__(kVecThreads, vec_blocks(NT, R))
 dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint32_t rows, uint32_t w_stride,
@@ -130,7 +132,7 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
         for (int r = 0; r < R; ++r)
             dst[r] = live ? load_weights16(row[r] + (size_t)s * T::kStep) : make_uint4(0, 0, 0, 0);
     };
-    uint32_t group = blockIdx.x * per_block + warp / ksplit;
+    uint32_t group = warp / ksplit * gridDim.x + blockIdx.x;
     // weights depend on no other kernel: the first ones are requested before the dependency wait
     turn_to(group);
 #pragma unroll
@@ -153,7 +155,7 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
     __syncthreads();
     uint32_t turn = 0;
 #pragma unroll 1
-    for (uint32_t first = blockIdx.x * per_block; first < groups; first += gridDim.x * per_block, turn ^= 1) {
+    for (uint32_t first = blockIdx.x; first < groups; first += gridDim.x * per_block, turn ^= 1) {
         const uint32_t next = group + gridDim.x * per_block;
         float acc[R][NT];
 #pragma unroll
@@ -232,14 +234,19 @@ dense_vector_kernel(InputArgs in, OutputArgs out, const W *__restrict__ w, uint3
 // ------------------------------------------------------------------ input rows of the matrix forms
 template <typename A>
 __global__ void __launch_bounds__(256)
-dense_input_kernel(InputArgs in, A *__restrict__ dst) {
+dense_input_kernel(InputArgs in, A *__restrict__ dst, int row_kind) {
     qk::pdl_launch();
-    qk::pdl_wait();
-    extern __shared__ __align__(16) float row_smem[];
+    extern __shared__ __align__(16) float row_smem[];  // [k], staged norm weights [2][width]
     __shared__ float red[8];
     const uint32_t t = blockIdx.x;
+    if (row_kind == kRowNorm) stage_norm_weights(in, row_smem + in.k);
+    qk::pdl_wait();
     if (dst) {
-        build_input(in, t, true, [&](uint32_t i) -> float & { return row_smem[i]; }, red);
+        if (row_kind == kRowNorm)
+            build_norm_row(in, t, true, row_smem + in.k,
+                           [&](uint32_t p) -> float4 & { return *reinterpret_cast<float4 *>(row_smem + 4 * p); }, red);
+        else
+            build_input(in, t, true, [&](uint32_t i) -> float & { return row_smem[i]; }, red);
         for (uint32_t j = 0; j < (in.places ? in.top : 1u); ++j) {
             A *o = dst + (size_t)(in.places ? (uint32_t)in.places[t * in.top + j] : t) * in.k;
             if constexpr (sizeof(A) == 2) {
@@ -1083,7 +1090,7 @@ qk_status launch_tc(qk_ctx *c, const void *x, size_t x_stride, const qk_dense_ca
 }
 
 // Which of the faster ways to read the input rows applies.
-int vector_row_kind(const InputArgs &a) {
+int row_kind_of(const InputArgs &a) {
     auto aligned = [](const void *p) { return ((uintptr_t)p & 15) == 0; };
     if (a.width % 4 || a.k % 4 || a.x_stride % 4 || !aligned(a.x)) return kRowAny;
     if (a.kind == QK_INPUT_PLAIN) return kRowPlain;
@@ -1097,7 +1104,7 @@ template <typename W, int NT, int R>
 qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
                           size_t n_tokens, uint32_t ks) {
     const size_t step = VecTraits<W>::kStep;
-    int kind = vector_row_kind(in);
+    int kind = row_kind_of(in);
     size_t smem = NT * qk::ceil_div(d.k, step) * step * 4;
     if (kind == kRowNorm && smem + 8 * d.width > kVecSmemMax) kind = kRowAny;
     if (kind == kRowNorm) smem += 8 * d.width;
@@ -1111,8 +1118,7 @@ qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out,
     // the blocks that stay resident, shared out evenly among the choices
     const size_t per_sm = std::max<size_t>(1, std::min<size_t>(vec_blocks(NT, R), kVecSmemSm / (smem + 2048)));
     const size_t resident = std::max<size_t>(1, per_sm * (size_t)c->sm_count / choices);
-    const size_t blocks = qk::ceil_div(groups * ks, kVecWarps), turns = qk::ceil_div(blocks, resident);
-    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>, dim3((unsigned)qk::ceil_div(blocks, turns), (unsigned)choices),
+    (void)qk::launch_pdl(c->pdl, dense_vector_kernel<W, NT, R>, dim3((unsigned)std::min(groups, resident), (unsigned)choices),
                          dim3(kVecThreads), smem, c->stream, in, out, (const W *)d.w, (uint32_t)d.rows,
                          (uint32_t)d.w_stride, (uint32_t)n_tokens, ks, ch, kind);
     QK_CUDA(cudaGetLastError());
@@ -1122,13 +1128,32 @@ qk_status launch_vector_r(qk_ctx *c, const InputArgs &in, const OutputArgs &out,
 template <typename W, int NT>
 qk_status launch_vector(qk_ctx *c, const InputArgs &in, const OutputArgs &out, const qk_dense_call &d,
                         size_t n_tokens) {
-    // rows per warp and warps per row group: about two blocks per SM or more (one, where a block
-    // has a long vector to stage first)
-    const size_t share = d.experts ? input_rows(d) : 1;  // (every choice has blocks of its own)
-    const size_t want = qk::ceil_div((d.k > 8192 ? 1 : 2) * (size_t)c->sm_count * kVecWarps, share);
+    // rows per warp and warps per row group
     const size_t steps = qk::ceil_div(d.k, VecTraits<W>::kStep);
     const bool pair = d.output == QK_OUTPUT_GLU;
-    if (d.rows / 4 >= want) return launch_vector_r<W, NT, 4>(c, in, out, d, n_tokens, 1);
+    if (d.experts) {
+        // The blocks are shared out among the choices, so that a few turns over the rows are usual: what
+        // takes the fewest batches of four steps one after the other (a turn costs a little on its own).
+        const size_t choices = input_rows(d);
+        int best_r = 2;
+        uint32_t best_ks = 1;
+        size_t best_cost = ~(size_t)0;
+        for (int r = pair ? 2 : 1; r <= 2; ++r) {
+            const size_t warps = std::max<size_t>(1, (size_t)vec_blocks(NT, r) * (size_t)c->sm_count / choices) * kVecWarps;
+            const size_t groups = pair ? d.rows / 2 : qk::ceil_div(d.rows, r);
+            for (uint32_t ks = 1; ks <= (uint32_t)kVecWarps && (ks == 1 || ks * 2 <= steps); ks *= 2) {
+                const size_t turns = qk::ceil_div(groups * ks, warps), batches = qk::ceil_div(steps, 4 * ks);
+                const size_t cost = turns * (4 * batches + (ks > 1 ? 2 : 1));
+                if (cost < best_cost) best_r = r, best_ks = ks, best_cost = cost;
+            }
+        }
+        return best_r == 2 ? launch_vector_r<W, NT, 2>(c, in, out, d, n_tokens, best_ks)
+                           : launch_vector_r<W, NT, 1>(c, in, out, d, n_tokens, best_ks);
+    }
+    // one matrix: about two blocks per SM or more (one, where a block has a long vector to stage
+    // first); measured in a whole step, splitting the k range further costs more than it evens out
+    const size_t want = (d.k > 8192 ? 1 : 2) * (size_t)c->sm_count * kVecWarps;
+    if (NT > 1 && d.rows / 4 >= want) return launch_vector_r<W, NT, 4>(c, in, out, d, n_tokens, 1);
     if (d.rows / 2 >= want || pair) {
         uint32_t ks = 1;
         while (ks < kVecWarps && d.rows / 2 * ks < want && ks * 4 <= steps) ks *= 2;
@@ -1324,11 +1349,12 @@ qk_status launch_input(qk_ctx *c, const InputArgs &in, size_t tokens, A *dst) {
         c->launches++;
         return QK_OK;
     }
-    const size_t smem = dst ? (size_t)in.k * 4 : 0;
+    const int kind = dst && in.k % 4 == 0 && row_kind_of(in) == kRowNorm ? kRowNorm : kRowAny;
+    const size_t smem = dst ? (size_t)in.k * 4 + (kind == kRowNorm ? in.width * 8 : 0) : 0;
     if (smem > kVecSmemMax) return qk::fail(QK_ERR_VALUE, "qk_dense: an input vector of %u entries does not fit shared memory", in.k);
     QK_CUDA(cudaFuncSetAttribute(dense_input_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  (int)std::max(smem, (size_t)48 * 1024)));
-    (void)qk::launch_pdl(c->pdl, dense_input_kernel<A>, dim3((unsigned)tokens), dim3(256), smem, c->stream, in, dst);
+    (void)qk::launch_pdl(c->pdl, dense_input_kernel<A>, dim3((unsigned)tokens), dim3(256), smem, c->stream, in, dst, kind);
     QK_CUDA(cudaGetLastError());
     c->launches++;
     return QK_OK;
