@@ -10,6 +10,7 @@ Sizes and constants are parameters: nothing here belongs to one design.
 from __future__ import annotations
 
 import ctypes
+import functools
 import math
 from ctypes import c_double, c_float, c_int32, c_size_t, c_uint64, c_void_p
 from dataclasses import dataclass
@@ -443,7 +444,8 @@ class LatentAttention:
                                       self.vdim_stride, window, self.scale, c_void_p(att.data_ptr()), o_stride))
 
 
-def distance_buckets(rows: int, bias_max: float, most: int = 1 << 24) -> list:
+@functools.lru_cache(maxsize=64)
+def distance_buckets(rows: int, bias_max: float, most: int = 1 << 24) -> tuple:
     """The table row of every distance, up to the first one from which on it is the last row: the
     near half one by one, then logarithmic steps that reach the end at ``bias_max``."""
     half = rows // 2
@@ -456,7 +458,7 @@ def distance_buckets(rows: int, bias_max: float, most: int = 1 << 24) -> list:
         out.append(n if n < half else
                    min(rows - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (rows - half))))
         n += 1
-    return out
+    return tuple(out)
 
 
 class GroupedAttention:

@@ -401,7 +401,7 @@ def test_grouped_attention_of_a_batch(dev):
 @pytest.mark.parametrize("heads,kv_heads,dim,vdim,p0,tokens", [
     (1, 1, 16, 16, 0, 20), (4, 2, 32, 64, 3, 64), (6, 3, 48, 20, 100, 65), (3, 1, 64, 128, 10, 200), (2, 2, 128, 16, 0, 300),
     (4, 1, 128, 128, 500, 129), (3, 1, 80, 112, 0, 300), (6, 2, 96, 64, 130, 260), (1, 1, 112, 80, 1000, 17),
-    (9, 3, 64, 64, 7, 385), (2, 1, 160, 256, 33, 70), (2, 2, 250, 96, 70, 100), (8, 2, 128, 128, 0, 513)])
+    (9, 3, 64, 64, 7, 385), (4, 2, 128, 128, 3000, 150), (2, 1, 160, 256, 33, 70), (2, 2, 250, 96, 70, 100), (8, 2, 128, 128, 0, 513)])
 def test_grouped_attention_of_a_portion(dev, heads, kv_heads, dim, vdim, p0, tokens):
     """Portions that start and end anywhere between key tiles, with the append in front; cache rows
     behind the portion hold no numbers."""

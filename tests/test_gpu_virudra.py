@@ -18,6 +18,7 @@ from layered_checks import agree, assert_rows, decode_logits, greedy_oracle, pro
 
 pytestmark = pytest.mark.gpu
 both = pytest.mark.parametrize("serving", ["float32", "bfloat16"])
+kernels = pytest.mark.parametrize("dim", [16, 64])   # (head sizes of both kernels of a portion)
 
 
 def Limit(cfg, w, toks, want, serving):
@@ -135,11 +136,11 @@ def test_batches_of_unequal_requests_and_slots_used_again(gpu_ctx, serving, batc
         lengths = lengths[::-1]
 
 
-def needle_model(bias_rows=12, strength=1.0, **kw):
+def needle_model(bias_rows=12, strength=1.0, dim=16, **kw):
     """One attention layer in which every query looks for one token's key: channel 6 is the same
     for every token and makes the query, channel 5 marks the needle and makes its key; the needle's
     value stands out too."""
-    cfg = vm.config([vm.bare(vm.attention(heads=4, kv_heads=2, dim=16, vdim=16, scale=1.0, **kw))], width=48, vocab=40)
+    cfg = vm.config([vm.bare(vm.attention(heads=4, kv_heads=2, dim=dim, vdim=dim, scale=1.0, **kw))], width=48, vocab=40)
     w = vm.weights(cfg, 9, bias_rows)
     needle = 7
     w["embed"][:, 5] = 0.0
@@ -147,22 +148,23 @@ def needle_model(bias_rows=12, strength=1.0, **kw):
     w["embed"][needle, 5] = 6.0
     w["l0.norm1"][:] = 0.0
     w["l0.mix.q"][:] *= 0.1
-    w["l0.mix.q"][::16] = 0.0
-    w["l0.mix.q"][::16, 6] = 2.0 * strength
+    w["l0.mix.q"][::dim] = 0.0
+    w["l0.mix.q"][::dim, 6] = 2.0 * strength
     w["l0.mix.k"][:] *= 0.1
-    w["l0.mix.k"][::16] = 0.0
-    w["l0.mix.k"][::16, 5] = 1.0 * strength
+    w["l0.mix.k"][::dim] = 0.0
+    w["l0.mix.k"][::dim, 5] = 1.0 * strength
     w["l0.mix.v"][:, 5] = 1.5
     w["l0.mix.rel"][:] = 0.0
     return cfg, {n: vm.bf16(a) for n, a in w.items()}, needle
 
 
 @both
-def test_far_keys(gpu_ctx, serving):
+@kernels
+def test_far_keys(gpu_ctx, serving, dim):
     """One key among hundreds, at every distance from the rows behind it: the attention finds it as
     a prompt, in portions and decoded (it would drop out of the row if any split, tile or page edge
     lost it; checked on the restatement)."""
-    cfg, w, needle = needle_model(coef=0.0)
+    cfg, w, needle = needle_model(dim=dim, coef=0.0)
     base = [t if t != needle else 8 for t in vm.prompt(cfg, 400)]
     for at in (0, 1, 15, 16, 63, 64, 129):
         toks = list(base)
@@ -186,20 +188,21 @@ def test_far_keys(gpu_ctx, serving):
 def bucket_ranges(rows, bias_max):
     """{bucket: (first, last distance)}; the last one ends nowhere."""
     out = {}
-    for n in range(4 * bias_max):
+    for n in range(4 * bias_max if bias_max < 100 else bias_max + 5):
         b = ref.bucket(n, rows, bias_max)
         out[b] = (out.get(b, (n, n))[0], n)
     return out
 
 
 @both
-@pytest.mark.parametrize("rows,bias_max", [(12, 40), (7, 30), (32, 33), (2, 5)])
-def test_bias_bucket_edges(gpu_ctx, serving, rows, bias_max, monkeypatch):
+@kernels
+@pytest.mark.parametrize("rows,bias_max", [(12, 40), (7, 30), (32, 33), (2, 5), (9, 200)])
+def test_bias_bucket_edges(gpu_ctx, serving, rows, bias_max, dim, monkeypatch):
     """One bucket at a time draws all the attention.  A bucket that began or ended a token off
     would move the rows whose distance to the needle lies at its edges (checked on the
     restatement); rows far behind it see only the last bucket."""
-    cfg, w, needle = needle_model(rows, 0.0, bias_max=bias_max)
-    toks = [t if t != needle else 8 for t in vm.prompt(cfg, 40 + 3 * bias_max)]
+    cfg, w, needle = needle_model(rows, 0.0, dim=dim, bias_max=bias_max)
+    toks = [t if t != needle else 8 for t in vm.prompt(cfg, 40 + 3 * min(bias_max, 100))]
     at = 30
     toks[at] = needle
     ranges = bucket_ranges(rows, bias_max)
@@ -234,11 +237,12 @@ def decode_after(dec, toks, cut, n):
 
 
 @both
+@kernels
 @pytest.mark.parametrize("every,coef", [(1, 0.7), (16, 3.0), (50, 3.0), (7.5, 2.0)])
-def test_temperature_steps(gpu_ctx, serving, every, coef, monkeypatch):
+def test_temperature_steps(gpu_ctx, serving, every, coef, dim, monkeypatch):
     """The factor on the queries steps at positions every k - 1: a step one position off would move
     those rows (checked on the restatement)."""
-    cfg, w, needle = needle_model(strength=0.2, every=every, coef=coef)
+    cfg, w, needle = needle_model(strength=0.2, dim=dim, every=every, coef=coef)
     toks = vm.prompt(cfg, 130)
     toks[3] = needle
     want = ref.forward(cfg, w, toks)

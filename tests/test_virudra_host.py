@@ -26,7 +26,7 @@ def test_distance_buckets(rows, bias_max):
     for n in range(3 * bias_max + 100):
         assert got[min(n, len(got) - 1)] == ref.bucket(n, rows, bias_max), n
     half = rows // 2
-    assert got[:half] == list(range(half))
+    assert got[:half] == tuple(range(half))
     for n, b in enumerate(got[half:], half):
         k = b - half    # n >= half * (bias_max / half) ** (k / (rows - half))
         assert n >= half * (bias_max / half) ** (k / (rows - half)) * (1 - 1e-9)

@@ -90,6 +90,8 @@ MODELS = {
     "attention-large-group": (config([bare(attention(heads=22, kv_heads=2, dim=12, vdim=10))]), 9),
     "attention-wide": (config([bare(attention(heads=4, kv_heads=2, dim=144, vdim=200))], width=130), 13),
     "attention-wide-keys": (config([bare(attention(heads=2, kv_heads=1, dim=128, vdim=40))]), 13),
+    "attention-tensor-memory": (config([bare(attention(heads=6, kv_heads=2, dim=72, vdim=100))]), 13),
+    "attention-tensor-memory-odd-group": (config([dense(attention(heads=3, kv_heads=1, dim=64, vdim=64), 40)], loop=(0, 1, 2)), 13),
     "attention-too-wide-for-tiles": (config([bare(attention(heads=2, kv_heads=1, dim=264, vdim=300))]), 7),
     "two-buckets": (config([bare(attention(bias_max=2))]), 2),
     "bias-to-the-end": (config([bare(attention(bias_max=44))]), 80),
