@@ -42,7 +42,7 @@ def linear(h, w):
 
 
 def rms_norm(x, w, eps):
-    """``w`` is stored around zero."""
+    """``w`` is an offset from one."""
     return x / np.sqrt((x ** 2).mean(axis=-1, keepdims=True) + eps) * (1.0 + w)
 
 

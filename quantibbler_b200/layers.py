@@ -132,7 +132,7 @@ class Weights:
         return t.to(self.device, dtype or self.dtype).contiguous()
 
     def vector(self, t, offset: float = 0.0):
-        """In float32; ``offset``: what a weight stored around zero stands beside."""
+        """In float32, plus ``offset`` (1 for weights that are kept as offsets from one)."""
         v = self.to(t, self.torch.float32)
         return v + offset if offset else v
 

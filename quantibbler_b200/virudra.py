@@ -2,8 +2,8 @@
 
 A decoder-only model of layers with grouped attention over the whole sequence (no rotation: a query
 temperature and a learned distance bias carry the positions), feed-forwards that are dense or a
-mixture of experts chosen by a table of token ids, RMS norms before and behind every sublayer with
-weights stored around zero, optionally a block of layers that runs several times, and a soft cap on
+mixture of experts chosen by a table of token ids, RMS norms before and behind every sublayer whose
+weights are offsets from one, optionally a block of layers that runs several times, and a soft cap on
 the logits.  Sizes and constants come from config.json; what the design fixes is written here.
 """
 

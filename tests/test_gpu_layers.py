@@ -421,7 +421,7 @@ def test_grouped_attention_of_a_portion(dev, heads, kv_heads, dim, vdim, p0, tok
     out = torch.zeros(tokens, heads * vs, device="cuda", dtype=torch.bfloat16)
     pos = torch.arange(p0, p0 + tokens, dtype=torch.int32, device="cuda")
     slot = torch.ones(tokens, dtype=torch.int32, device="cuda")
-    scale, coef, every = 1.0 / dim ** 0.5, 0.3, 64.0
+    scale, coef, every = 1.0 / dim ** 0.5, 0.35, 48.0
     c = L.GroupedCall(tokens=tokens, positions=pos.data_ptr(), slots=slot.data_ptr(), heads=heads, kv_heads=kv_heads,
                       dim_stride=ds, vdim_stride=vs, s_max=s_max, n_slots=3, scale=scale, temp_coef=coef, temp_every=every,
                       bias=bias.data_ptr(), bias_len=bias.shape[1], proj=proj.data_ptr(), proj_dtype=QK_BF16,

@@ -64,9 +64,9 @@ def test_attention_row_by_row():
 
 
 def test_temperature_norm_cap_activations():
-    assert ref.query_temperature(0, 0.3, 64) == 1.0 and ref.query_temperature(62, 0.3, 64) == 1.0
-    assert ref.query_temperature(63, 0.3, 64) == 1 + 0.3 * np.log(2)
-    assert ref.query_temperature(127, 0.3, 64) == 1 + 0.3 * np.log(3)
+    assert ref.query_temperature(0, 0.7, 50) == 1.0 and ref.query_temperature(48, 0.7, 50) == 1.0
+    assert ref.query_temperature(49, 0.7, 50) == 1 + 0.7 * np.log(2)
+    assert ref.query_temperature(99, 0.7, 50) == 1 + 0.7 * np.log(3)
     assert ref.query_temperature(0, 2.0, 1) == 1 + 2 * np.log(2)
     x = np.array([[1.0, 2.0, 6.0]])
     np.testing.assert_allclose(ref.rms_norm(x, 0.25, 0.5), 1.25 * x / np.sqrt(41 / 3 + 0.5))
